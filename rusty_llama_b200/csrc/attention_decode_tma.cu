@@ -100,7 +100,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
                        const float* __restrict__ inv_freq, int rot, int interleaved,
                        unsigned int* __restrict__ counters, bf16* __restrict__ out, int out_stride,
                        const float* __restrict__ q_parts, int n_parts, long long part_stride, int test_role,
-                       uint32_t test_ns, const float* __restrict__ sink, int chunk, float softcap) {
+                       uint32_t test_ns, const float* __restrict__ sink, int chunk, float softcap, int maps) {
   // all shared memory is dynamic, so that the ring starts at the block's first byte (1024-byte
   // aligned, as the 128-byte swizzle needs)
   constexpr int STAGES = Shape<HD>::STAGES, STAGE_BYTES = Shape<HD>::STAGE_BYTES, BOXES = Shape<HD>::BOXES;
@@ -209,8 +209,10 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     // this block's queries: HEADS rows of HD values, 16 bytes per thread
     constexpr int PIECES = HD / 8;
     const int r = threadIdx.x / PIECES, piece = threadIdx.x % PIECES;  // 128 threads = 8 (or 16) rows x 16 (or 8) pieces
-    if (r < n_heads) {
-      const size_t at = (size_t)s * q_stride + (size_t)(h0 + r) * HD + piece * 8;
+    // (with two maps per head, query heads 2h and 2h + 1 are the halves of row h; the rest of their rows here stays zero)
+    const int qh = (h0 + r) / maps, q_half = (h0 + r) - qh * maps;
+    if (r < n_heads && (maps == 1 || piece / (PIECES / 2) == q_half)) {
+      const size_t at = (size_t)s * q_stride + (size_t)qh * HD + piece * 8;
       if (n_parts == 0) {
         *reinterpret_cast<uint4*>(q_s + (size_t)r * Q_STRIDE + piece * 8) = __ldcg(reinterpret_cast<const uint4*>(q + at));
       } else {
@@ -282,7 +284,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
 #pragma unroll
   for (int e = 0; e < DPL; ++e) new_k[e] = new_v[e] = 0.f;
   if (patch_here) {
-    const size_t k_at = (size_t)s * q_stride + (size_t)(H + kh) * HD + DPL * lane, v_at = k_at + (size_t)K * HD;
+    const size_t k_at = (size_t)s * q_stride + (size_t)(H / maps + kh) * HD + DPL * lane, v_at = k_at + (size_t)K * HD;
     if (n_parts == 0) {
       if (DPL == 4) {
         const uint2 kr = __ldcg(reinterpret_cast<const uint2*>(q + k_at)), vr = __ldcg(reinterpret_cast<const uint2*>(q + v_at));
@@ -575,6 +577,8 @@ RL_API int rl_attn_decode_tma_takes(int hd) { return hd == 64 || hd == 128; }
 // counters: null, or n_seqs * (K * groups of 8 heads) zeros in device memory: the splits are then added
 // up by the block that finishes last (no merge kernel is launched) and the counters are zeros again
 // when the kernel ends.
+// maps: 1, or 2: query heads 2h and 2h + 1 are the two halves of row h's hd numbers (and meet the same halves of the keys); the
+// second kernel then combines the pair, out[s][h] = o / sqrt(mean(o^2) + pair_eps) * pair_factor with o = a_2h - pair_lambda a_(2h+1).
 // wait_test_role, wait_test_ns: 0, 0 in normal use; a test names 51 or 52 and a limit in nanoseconds, and
 // that role's waits give up after that long instead of a second.
 template <int HD>
@@ -583,7 +587,8 @@ static int launch_decode_tma(const void* q, int q_stride, const void* k_pages, c
                              void* out, int out_stride, int n_seqs, int H, int K, int window, float scale, int n_splits,
                              int* status, int fuse, const float* inv_freq, int rot, int interleaved, unsigned int* counters,
                              const float* q_parts, int n_parts, long long part_stride, int wait_test_role,
-                             unsigned int wait_test_ns, const float* sink, int chunk, float softcap, cudaStream_t stream) {
+                             unsigned int wait_test_ns, const float* sink, int chunk, float softcap, int maps, float pair_lambda, float pair_eps,
+                             float pair_factor, cudaStream_t stream) {
   CUtensorMap map_k, map_v;
   if (make_page_map(&map_k, k_pages, n_pages, K, PAGE, HD, PAGE) || make_page_map(&map_v, v_pages, n_pages, K, PAGE, HD, PAGE))
     RL_REFUSE(10, "attn_decode_tma: cannot describe the cache pages to TMA");
@@ -597,7 +602,13 @@ static int launch_decode_tma(const void* q, int q_stride, const void* k_pages, c
                             table_width, seq_len, part_o, part_ml, H, K, window, scale * 1.4426950408889634f, n_splits, status,
                             fuse, (bf16*)const_cast<void*>(k_pages), (bf16*)const_cast<void*>(v_pages), inv_freq, fuse ? rot : 0,
                             interleaved, counters, (bf16*)out, out_stride, q_parts, n_parts, part_stride, wait_test_role,
-                            (uint32_t)wait_test_ns, sink, chunk, softcap));
+                            (uint32_t)wait_test_ns, sink, chunk, softcap, maps));
+  if (maps == 2) {
+    dim3 grid1(H / 2, n_seqs);
+    RL_LAUNCH_CHECK(rl_launch(attn_decode_merge_pair_kernel, grid1, HD, 0, stream, (const float*)part_o, (const float*)part_ml, (bf16*)out,
+                              out_stride, H, HD, n_splits, pair_lambda, pair_eps, pair_factor));
+    return 0;
+  }
   if (counters != nullptr) return 0;
   dim3 grid2(H, n_seqs);
   RL_LAUNCH_CHECK(rl_launch(attn_decode_merge_kernel, grid2, 128, 0, stream, (const float*)part_o, (const float*)part_ml,
@@ -611,7 +622,9 @@ RL_API int rl_attn_decode_tma(const void* q, int q_stride, const void* k_pages, 
                               float scale, int n_splits, int* status, int fuse, const float* inv_freq, int rot,
                               int interleaved, unsigned int* counters, const float* q_parts, int n_parts,
                               long long part_stride, int wait_test_role, unsigned int wait_test_ns, const float* sink,
-                              int chunk, float softcap, cudaStream_t stream) {
+                              int chunk, float softcap, int maps, float pair_lambda, float pair_eps, float pair_factor, cudaStream_t stream) {
+  if (maps < 1 || maps > 2 || H % maps || (maps == 2 && (counters != nullptr || rot != 0)))
+    RL_REFUSE(15, "attn_decode_tma: %d maps in %d heads (two maps: no rotation, no counters)", maps, H);
   if (n_seqs <= 0 || H <= 0 || K <= 0 || n_pages <= 0) RL_REFUSE(1, "attn_decode_tma: S=%d H=%d K=%d pages=%d", n_seqs, H, K, n_pages);
   if (!rl_attn_decode_tma_takes(hd)) RL_REFUSE(2, "attn_decode_tma: head size %d, this kernel is built for 64 and 128", hd);
   if (H % K) RL_REFUSE(3, "attn_decode_tma: %d query heads are not a multiple of %d kv heads", H, K);
@@ -625,11 +638,12 @@ RL_API int rl_attn_decode_tma(const void* q, int q_stride, const void* k_pages, 
     RL_REFUSE(12, "attn_decode_tma: fuse=%d with a rotary size of %d (a multiple of 8 up to the head size)%s", fuse, rot, inv_freq ? "" : " and no angles");
   if (n_parts < 0 || n_parts > 64 || (n_parts > 0 && (q_parts == nullptr || fuse == 0 || ((uintptr_t)q_parts & 15) || part_stride % 4 || q_stride % 4)))
     RL_REFUSE(14, "attn_decode_tma: %d partial sums need fuse > 0 and 16-byte aligned rows", n_parts);
-  if (fuse == 2 && q_stride < (H + 2 * K) * hd) RL_REFUSE(13, "attn_decode_tma: rows of %d hold no key and value behind %d query heads", q_stride, H);
+  if (fuse == 2 && q_stride < (H / maps + 2 * K) * hd) RL_REFUSE(13, "attn_decode_tma: rows of %d hold no key and value behind %d query heads", q_stride, H);
 #define RL_DECODE_TMA(HDV)                                                                                                  \
   return launch_decode_tma<HDV>(q, q_stride, k_pages, v_pages, n_pages, block_table, table_width, seq_len, part_o, part_ml, out, \
                                 out_stride, n_seqs, H, K, window, scale, n_splits, status, fuse, inv_freq, rot, interleaved,      \
-                                counters, q_parts, n_parts, part_stride, wait_test_role, wait_test_ns, sink, chunk, softcap, stream)
+                                counters, q_parts, n_parts, part_stride, wait_test_role, wait_test_ns, sink, chunk, softcap, maps, pair_lambda,    \
+                                pair_eps, pair_factor, stream)
   if (hd == 64) RL_DECODE_TMA(64);
   RL_DECODE_TMA(128);
 #undef RL_DECODE_TMA

@@ -13,7 +13,10 @@
 //     counted from the start of the sequence),
 //   - a cap on the scores, s <- cap tanh(s / cap), after the scale (and the mixing),
 //   - a sink per head: exp(sink_h) joins the softmax's denominator and nothing else,
-//   - a gate on the result, out *= sigmoid(gate), and a constant factor `out_scale`.
+//   - a gate on the result, out *= sigmoid(gate), and a constant factor `out_scale`,
+//   - two maps per head (`maps` 2): query heads 2h and 2h + 1 are the two halves of head h's query row of `kdim` numbers and meet
+//     the same halves of the keys, kdim / 2 numbers each; `map_combine` makes o_h = a_2h - lambda a_(2h+1) of their results,
+//     divided by its root mean square over the head's values, times a constant.
 //
 // Two kernels.  `qkv_prep` adds the biases, rotates q in place and writes the rotated k and v to the token's
 // place in its sequence's pages; with `v_src` the value that is stored is (1 - lambda) v + lambda v_src[t] (values that an
@@ -229,7 +232,7 @@ RL_API int rl_qkv_prep(void* qkv, int dtype, int row_stride, const float* bias, 
                        int vdim, int rot, int interleaved, int page_size, const void* v_src, int v_src_stride, const float* v_lambda,
                        cudaStream_t stream) {
   if (v_src != nullptr && (v_lambda == nullptr || v_src_stride < K * vdim)) RL_REFUSE(8, "qkv_prep: values to mix in need a factor and rows of %d numbers", K * vdim);
-  if (n_tokens <= 0 || H <= 0 || K <= 0 || kdim <= 0 || vdim <= 0 || page_size <= 0 || table_width <= 0)
+  if (n_tokens <= 0 || H < 0 || K <= 0 || kdim <= 0 || vdim <= 0 || page_size <= 0 || table_width <= 0)  // (H 0: rows that hold keys and values only)
     RL_REFUSE(1, "qkv_prep: T=%d H=%d K=%d kdim=%d vdim=%d page=%d", n_tokens, H, K, kdim, vdim, page_size);
   if (rot < 0 || rot > kdim || (rot & 1)) RL_REFUSE(2, "qkv_prep: %d rotated dimensions do not fit a head of %d", rot, kdim);
   if (row_stride < (H + K) * kdim + K * vdim) RL_REFUSE(3, "qkv_prep: row stride %d too small", row_stride);
@@ -268,7 +271,7 @@ __global__ void attn_ext_kernel(const T* __restrict__ q, int q_stride, const T* 
                                 const int* __restrict__ block_table, int table_width, const int* __restrict__ tok_seq,
                                 const int* __restrict__ tok_pos, const float* __restrict__ sink, const float* __restrict__ mix,
                                 const T* __restrict__ gate, int gate_stride, float out_scale, T* __restrict__ out, int out_stride,
-                                int H, int K, int kdim, int vdim, int page_size, int window, float scale, int chunk, float softcap) {
+                                int H, int K, int kdim, int vdim, int page_size, int window, float scale, int chunk, float softcap, int maps) {
   extern __shared__ float smem[];  // q of the block's heads [HB][kdim], then (with mix) scores [HB][32]
   const int lane = threadIdx.x;
   const int hb = threadIdx.y, HB = blockDim.y;
@@ -278,8 +281,9 @@ __global__ void attn_ext_kernel(const T* __restrict__ q, int q_stride, const T* 
   const int* table = block_table + (size_t)tok_seq[t] * table_width;
   float* q_s = smem + (size_t)hb * kdim;
   float* sc = smem + (size_t)HB * kdim;
-  const T* qh = q + (size_t)t * q_stride + (size_t)h * kdim;
-  for (int i = lane; i < kdim; i += 32) q_s[i] = to_f32(qh[i]);
+  const T* qh = q + (size_t)t * q_stride + (size_t)(h / maps) * kdim;
+  const int i_lo = (h % maps) * (kdim / maps), i_hi = i_lo + kdim / maps;  // the numbers of query and key that make this head's score
+  for (int i = i_lo + lane; i < i_hi; i += 32) q_s[i] = to_f32(qh[i]);
   __syncwarp();
 
   int first = (window != 0 && pos + 1 > window) ? pos + 1 - window : 0;
@@ -301,7 +305,7 @@ __global__ void attn_ext_kernel(const T* __restrict__ q, int q_stride, const T* 
       const int page = table[key / page_size];
       const T* kr = k_pages + (((size_t)page * K + kh) * page_size + key % page_size) * kdim;
       float dot = 0.f;
-      for (int i = 0; i < kdim; ++i) dot += q_s[i] * to_f32(kr[i]);
+      for (int i = i_lo; i < i_hi; ++i) dot += q_s[i] * to_f32(kr[i]);
       s = dot * scale;
     }
     if (mix != nullptr) {
@@ -351,7 +355,8 @@ __global__ void attn_ext_kernel(const T* __restrict__ q, int q_stride, const T* 
 RL_API int rl_attn_ext(const void* q, int dtype, int q_stride, const void* k_pages, const void* v_pages, const int* block_table,
                        int table_width, const int* tok_seq, const int* tok_pos, const float* sink, const float* mix,
                        const void* gate, int gate_stride, float out_scale, void* out, int out_stride, int n_tokens, int H, int K,
-                       int kdim, int vdim, int page_size, int window, float scale, int chunk, float softcap, cudaStream_t stream) {
+                       int kdim, int vdim, int page_size, int window, float scale, int chunk, float softcap, int maps, cudaStream_t stream) {
+  if (maps < 1 || maps > 2 || H % maps || kdim % maps || (maps > 1 && mix != nullptr)) RL_REFUSE(9, "attn_ext: %d maps in %d heads of %d numbers%s", maps, H, kdim, mix ? " whose scores are mixed" : "");
   if (n_tokens <= 0 || H <= 0 || K <= 0 || kdim <= 0 || vdim <= 0 || page_size <= 0)
     RL_REFUSE(1, "attn_ext: T=%d H=%d K=%d kdim=%d vdim=%d page=%d", n_tokens, H, K, kdim, vdim, page_size);
   if (H % K) RL_REFUSE(2, "attn_ext: %d query heads are not a multiple of %d kv heads", H, K);
@@ -367,13 +372,82 @@ RL_API int rl_attn_ext(const void* q, int dtype, int q_stride, const void* k_pag
     attn_ext_kernel<bf16><<<grid, block, smem, stream>>>((const bf16*)q, q_stride, (const bf16*)k_pages, (const bf16*)v_pages,
                                                          block_table, table_width, tok_seq, tok_pos, sink, mix, (const bf16*)gate,
                                                          gate_stride, out_scale, (bf16*)out, out_stride, H, K, kdim, vdim, page_size,
-                                                         window, scale, chunk, softcap);
+                                                         window, scale, chunk, softcap, maps);
   else if (dtype == RL_F32)
     attn_ext_kernel<float><<<grid, block, smem, stream>>>((const float*)q, q_stride, (const float*)k_pages, (const float*)v_pages,
                                                           block_table, table_width, tok_seq, tok_pos, sink, mix, (const float*)gate,
                                                           gate_stride, out_scale, (float*)out, out_stride, H, K, kdim, vdim, page_size,
-                                                          window, scale, chunk, softcap);
+                                                          window, scale, chunk, softcap, maps);
   else
     RL_REFUSE(8, "attn_ext: unknown dtype %d", dtype);
   RL_LAUNCH_RESULT();
+}
+
+// ---------------------------------------------------------------- two maps into one head
+// One warp per (token, head): a1 = a[t][2h], a2 = a[t][2h + 1] (vdim numbers each), o = a1 - lambda a2, out[t][h] = o / sqrt(mean(o^2) + eps) * factor.
+// All of it 32-bit.  U: neighbouring numbers a lane takes at a time.
+template <typename T, int U>
+__global__ void map_combine_kernel(const T* __restrict__ a, int a_stride, float lambda, float eps, float factor, T* __restrict__ out, int out_stride,
+                                   int n_rows, int H, int vdim) {
+  pdl_trigger();
+  pdl_wait();
+  const int lane = threadIdx.x & 31;
+  const int pair = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (pair >= n_rows * H) return;
+  const int t = pair / H, h = pair - t * H;
+  const T* a1 = a + (size_t)t * a_stride + (size_t)(2 * h) * vdim;
+  const T* a2 = a1 + vdim;
+  constexpr int N = 256 / (32 * U);  // value sizes up to 256
+  float v[N][U];
+  float ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < N; ++c) {
+    const int i = (lane + 32 * c) * U;
+    if (i < vdim) {
+      float x[U], y[U];
+      if (U == 4) {
+        load4_g<T>(a1 + i, x);
+        load4_g<T>(a2 + i, y);
+      } else {
+        x[0] = to_f32(__ldcg(a1 + i));
+        y[0] = to_f32(__ldcg(a2 + i));
+      }
+#pragma unroll
+      for (int e = 0; e < U; ++e) {
+        v[c][e] = x[e] - lambda * y[e];
+        ss += v[c][e] * v[c][e];
+      }
+    }
+  }
+  const float inv = factor / sqrtf(warp_sum(ss) / (float)vdim + eps);
+  T* o = out + (size_t)t * out_stride + (size_t)h * vdim;
+#pragma unroll
+  for (int c = 0; c < N; ++c) {
+    const int i = (lane + 32 * c) * U;
+    if (i < vdim) {
+#pragma unroll
+      for (int e = 0; e < U; ++e) v[c][e] *= inv;
+      if (U == 4) store4<T>(o + i, v[c]);
+      else o[i] = from_f32<T>(v[c][0]);
+    }
+  }
+}
+
+RL_API int rl_map_combine(const void* a, int dtype, int a_stride, float lambda, float eps, float factor, void* out, int out_stride, int n_rows,
+                          int H, int vdim, cudaStream_t stream) {
+  if (n_rows <= 0 || H <= 0 || vdim <= 0 || vdim > 256) RL_REFUSE(1, "map_combine: rows=%d H=%d values=%d (at most 256)", n_rows, H, vdim);
+  if (a_stride < 2 * H * vdim || out_stride < H * vdim) RL_REFUSE(2, "map_combine: rows too short");
+  if ((long long)n_rows * H > 0x7ffffff0LL) RL_REFUSE(3, "map_combine: %d rows of %d heads are too many", n_rows, H);
+  const int blocks = (int)(((long long)n_rows * H + 3) / 4);
+  const size_t bytes = dtype == RL_BF16 ? 8 : 16;
+  const bool vec = vdim % 4 == 0 && a_stride % 4 == 0 && out_stride % 4 == 0 && (((uintptr_t)a | (uintptr_t)out) % bytes) == 0;
+#define RL_MC(T, U) \
+  RL_LAUNCH_CHECK(rl_launch(map_combine_kernel<T, U>, blocks, 128, 0, stream, (const T*)a, a_stride, lambda, eps, factor, (T*)out, out_stride, n_rows, H, vdim))
+  if (dtype == RL_BF16 && vec) RL_MC(bf16, 4);
+  else if (dtype == RL_BF16) RL_MC(bf16, 1);
+  else if (dtype == RL_F32 && vec) RL_MC(float, 4);
+  else if (dtype == RL_F32) RL_MC(float, 1);
+  else RL_REFUSE(4, "map_combine: unknown dtype %d", dtype);
+#undef RL_MC
+  return 0;
 }

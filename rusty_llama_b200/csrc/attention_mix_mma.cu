@@ -58,13 +58,19 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 // One block per token: the token's rotated queries (32-bit) and the mixing matrix in shared memory; a warp makes one
 // (head, kv head) part at a time, its lanes the dimensions.
 __global__ void __launch_bounds__(256)
-fold_queries_kernel(const bf16* __restrict__ q, int q_stride, const float* __restrict__ mix, bf16* __restrict__ out, int H, int K, int kdim) {
+fold_queries_kernel(const bf16* __restrict__ q, int q_stride, const float* __restrict__ mix, bf16* __restrict__ out, int H, int K, int kdim, int maps) {
   extern __shared__ float fq_s[];  // q [H][kdim], mix [H][H]
   float* q_s = fq_s;
   float* m_s = fq_s + H * kdim;
   const int t = blockIdx.x, rep = H / K;
   const bf16* row = q + (size_t)t * q_stride;
-  if (((H * kdim) & 7) == 0 && (((uintptr_t)row) & 15) == 0) {  // sixteen bytes a load, all of a thread's loads in flight at once
+  if (maps > 1) {  // query head h is half h % 2 of row h / 2, zeros elsewhere
+    const int part = kdim / maps;
+    for (int i = threadIdx.x; i < H * kdim; i += blockDim.x) {
+      const int h = i / kdim, d = i - h * kdim;
+      q_s[i] = d / part == h % maps ? __bfloat162float(row[(size_t)(h / maps) * kdim + d]) : 0.f;
+    }
+  } else if (((H * kdim) & 7) == 0 && (((uintptr_t)row) & 15) == 0) {  // sixteen bytes a load, all of a thread's loads in flight at once
 #pragma unroll 4
     for (int i = threadIdx.x * 8; i < H * kdim; i += blockDim.x * 8) {
       const uint4 raw = __ldg(reinterpret_cast<const uint4*>(row + i));
@@ -95,12 +101,13 @@ fold_queries_kernel(const bf16* __restrict__ q, int q_stride, const float* __res
 }
 
 RL_API int rl_fold_queries(const void* q, int q_stride, const float* mix, void* out, int n_tokens, int H, int K, int kdim,
-                           cudaStream_t stream) {
+                           int maps, cudaStream_t stream) {
+  if (maps < 1 || maps > 2 || H % maps || kdim % maps) RL_REFUSE(3, "fold_queries: %d maps in %d heads of %d numbers", maps, H, kdim);
   if (n_tokens <= 0 || H <= 0 || K <= 0 || kdim <= 0 || H % K || !q || !mix || !out) RL_REFUSE(1, "fold_queries: T=%d H=%d K=%d kdim=%d", n_tokens, H, K, kdim);
   const size_t smem = ((size_t)H * kdim + (size_t)H * H) * sizeof(float);
   if (smem > 48 * 1024) RL_REFUSE(2, "fold_queries: %d heads of %d numbers do not fit shared memory", H, kdim);
   dim3 grid(n_tokens, n_tokens >= 64 ? 1 : 8);
-  fold_queries_kernel<<<grid, 256, smem, stream>>>((const bf16*)q, q_stride, mix, (bf16*)out, H, K, kdim);
+  fold_queries_kernel<<<grid, 256, smem, stream>>>((const bf16*)q, q_stride, mix, (bf16*)out, H, K, kdim, maps);
   RL_LAUNCH_RESULT();
 }
 
@@ -121,7 +128,7 @@ flash_mix_kernel(const bf16* __restrict__ q, long long q_row_stride, int q_head_
                  const bf16* __restrict__ v_pages, const int* __restrict__ block_table, int table_width,
                  const int* __restrict__ seq_start, const int* __restrict__ seq_pos0, const float* __restrict__ sink,
                  const bf16* __restrict__ gate, int gate_stride, float out_scale, bf16* __restrict__ out, int out_stride, int H, int K,
-                 int kdim, int vdim, int window, float scale_log2, int chunk, float softcap) {
+                 int kdim, int vdim, int window, float scale_log2, int chunk, float softcap, int maps) {
   constexpr int STRIDE = HD + 8;  // 16 bytes of padding per row keep ldmatrix free of bank conflicts
   constexpr int KSTEPS = HD / 16;
   constexpr int NTHREADS = BM * 2;  // a warp per 16 query rows
@@ -148,9 +155,14 @@ flash_mix_kernel(const bf16* __restrict__ q, long long q_row_stride, int q_head_
     for (int i = tid; i < n16; i += NTHREADS) p[i] = z;
   }
   __syncthreads();
-  for (int p = 0; p < parts; ++p)
-    load_rows<NTHREADS>(q_s + (size_t)p * BM * STRIDE, q + (size_t)(tok0 + row0) * q_row_stride + (size_t)h * q_head_stride + (size_t)p * kdim,
-              (size_t)q_row_stride, rows_here, kdim, STRIDE);
+  if (maps > 1) {  // half h % 2 of the row of head h / 2; the other half stays zero
+    const int part = kdim / maps, at = (h % maps) * part;
+    load_rows<NTHREADS>(q_s + at, q + (size_t)(tok0 + row0) * q_row_stride + (size_t)(h / maps) * q_head_stride + at, (size_t)q_row_stride, rows_here, part, STRIDE);
+  } else {
+    for (int p = 0; p < parts; ++p)
+      load_rows<NTHREADS>(q_s + (size_t)p * BM * STRIDE, q + (size_t)(tok0 + row0) * q_row_stride + (size_t)h * q_head_stride + (size_t)p * kdim,
+                          (size_t)q_row_stride, rows_here, kdim, STRIDE);
+  }
   const int* table = block_table + (size_t)s * table_width;
   const int last_pos = pos0 + row0 + rows_here - 1;
   const int first_pos = pos0 + row0;
@@ -311,7 +323,7 @@ template <int HD, int BM>
 static int launch_mix_rows(const bf16* q, long long q_row_stride, int q_head_stride, int parts, const bf16* k_pages, const bf16* v_pages,
                       const int* block_table, int table_width, const int* seq_start, const int* seq_pos0, const float* sink,
                       const bf16* gate, int gate_stride, float out_scale, bf16* out, int out_stride, int n_seqs, int max_q_len, int H, int K,
-                      int kdim, int vdim, int window, float scale, int chunk, float softcap, cudaStream_t stream) {
+                      int kdim, int vdim, int window, float scale, int chunk, float softcap, int maps, cudaStream_t stream) {
   const size_t smem = (size_t)(NBUF * BN + parts * BM) * (HD + 8) * sizeof(bf16);
   auto kern = flash_mix_kernel<HD, BM>;
   if (smem > 227 * 1024) RL_REFUSE(8, "flash_mix: %zu bytes of shared memory for %d query parts exceed the SM's", smem, parts);
@@ -322,7 +334,7 @@ static int launch_mix_rows(const bf16* q, long long q_row_stride, int q_head_str
   dim3 grid(H * n_seqs, (max_q_len + BM - 1) / BM);
   kern<<<grid, BM * 2, smem, stream>>>(q, q_row_stride, q_head_stride, parts, k_pages, v_pages, block_table, table_width, seq_start,
                                          seq_pos0, sink, gate, gate_stride, out_scale, out, out_stride, H, K, kdim, vdim, window,
-                                         scale * 1.4426950408889634f, chunk, softcap);
+                                         scale * 1.4426950408889634f, chunk, softcap, maps);
   RL_LAUNCH_RESULT();
 }
 
@@ -330,7 +342,7 @@ template <int HD>
 static int launch_mix(const bf16* q, long long q_row_stride, int q_head_stride, int parts, const bf16* k_pages, const bf16* v_pages,
                       const int* block_table, int table_width, const int* seq_start, const int* seq_pos0, const float* sink,
                       const bf16* gate, int gate_stride, float out_scale, bf16* out, int out_stride, int n_seqs, int max_q_len, int H, int K,
-                      int kdim, int vdim, int window, float scale, int chunk, float softcap, cudaStream_t stream) {
+                      int kdim, int vdim, int window, float scale, int chunk, float softcap, int maps, cudaStream_t stream) {
   // 128 rows to a block where several query parts would leave one block of 64 rows alone on its SM anyway and the step has
   // the rows to fill it
   const size_t smem128 = (size_t)(NBUF * BN + parts * 128) * (HD + 8) * sizeof(bf16);
@@ -338,17 +350,19 @@ static int launch_mix(const bf16* q, long long q_row_stride, int q_head_stride, 
   if (HD <= 128 && parts > 1 && max_q_len > 64 && smem128 <= 227 * 1024 && 2 * smem64 > 227 * 1024)
     return launch_mix_rows<HD, 128>(q, q_row_stride, q_head_stride, parts, k_pages, v_pages, block_table, table_width, seq_start, seq_pos0,
                                     sink, gate, gate_stride, out_scale, out, out_stride, n_seqs, max_q_len, H, K, kdim, vdim, window, scale,
-                                    chunk, softcap, stream);
+                                    chunk, softcap, maps, stream);
   return launch_mix_rows<HD, 64>(q, q_row_stride, q_head_stride, parts, k_pages, v_pages, block_table, table_width, seq_start, seq_pos0, sink,
-                                 gate, gate_stride, out_scale, out, out_stride, n_seqs, max_q_len, H, K, kdim, vdim, window, scale, chunk, softcap, stream);
+                                 gate, gate_stride, out_scale, out, out_stride, n_seqs, max_q_len, H, K, kdim, vdim, window, scale, chunk, softcap, maps, stream);
 }
 
 // q: the queries [T][..], row stride q_row_stride, head h at h * q_head_stride, part p of a head at + p * kdim.
 // parts: 1 (a head reads its own kv head's keys) or K (folded queries: part c goes against the keys of kv head c).
+// maps: 1, or 2 (with one part): query heads 2h and 2h + 1 are the halves of the row of kdim numbers at h * q_head_stride.
 RL_API int rl_flash_mix(const void* q, long long q_row_stride, int q_head_stride, int parts, const void* k_pages, const void* v_pages,
                         const int* block_table, int table_width, const int* seq_start, const int* seq_pos0, const float* sink,
                         const void* gate, int gate_stride, float out_scale, void* out, int out_stride, int n_seqs, int max_q_len, int H,
-                        int K, int kdim, int vdim, int page_size, int window, float scale, int chunk, float softcap, cudaStream_t stream) {
+                        int K, int kdim, int vdim, int page_size, int window, float scale, int chunk, float softcap, int maps, cudaStream_t stream) {
+  if (maps < 1 || maps > 2 || H % maps || kdim % (8 * maps) || (maps > 1 && parts > 1)) RL_REFUSE(10, "flash_mix: %d maps in %d heads of %d numbers", maps, H, kdim);
   if (n_seqs <= 0 || max_q_len <= 0 || H <= 0 || K <= 0 || kdim <= 0 || vdim <= 0)
     RL_REFUSE(1, "flash_mix: S=%d max_q=%d H=%d K=%d kdim=%d vdim=%d", n_seqs, max_q_len, H, K, kdim, vdim);
   if (H % K) RL_REFUSE(2, "flash_mix: %d query heads are not a multiple of %d kv heads", H, K);
@@ -364,7 +378,7 @@ RL_API int rl_flash_mix(const void* q, long long q_row_stride, int q_head_stride
 #define RL_MIX(HDV)                                                                                                                   \
   return launch_mix<HDV>((const bf16*)q, q_row_stride, q_head_stride, parts, (const bf16*)k_pages, (const bf16*)v_pages, block_table,  \
                          table_width, seq_start, seq_pos0, sink, (const bf16*)gate, gate_stride, out_scale, (bf16*)out, out_stride,      \
-                         n_seqs, max_q_len, H, K, kdim, vdim, window, scale, chunk, softcap, stream)
+                         n_seqs, max_q_len, H, K, kdim, vdim, window, scale, chunk, softcap, maps, stream)
   if (hd <= 32) RL_MIX(32);
   if (hd <= 64) RL_MIX(64);
   if (hd <= 128) RL_MIX(128);

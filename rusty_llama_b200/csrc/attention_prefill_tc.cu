@@ -95,11 +95,12 @@ __device__ __forceinline__ float exp2_fast(float x) {
 // The MMAs of S = Q K^T for one key tile (a k step is 16 dims; Q and K lie in sub-tiles of 64 dims: 16 KB and 8 KB
 // apart, in the descriptors' units of 16 bytes 1024 and 512), their commit, and a question about another barrier asked
 // first and read last.  Returns 1 if that barrier's phase `peek_parity` is complete.
-template <int HD>
+// KD: how many dims take part (HD, or half of them where a head has two maps: the descriptors then start at the map's half).
+template <int KD>
 __device__ __forceinline__ uint32_t qk_block(uint32_t tmem_s, uint64_t q_desc, uint64_t k_desc, uint32_t idesc, uint32_t commit_bar,
                                              uint32_t peek_bar, uint32_t peek_parity) {
   uint32_t ready;
-  if (HD == 128) {
+  if (KD == 128) {
     asm volatile(
         "{\n"
         ".reg .pred t, f, q;\n"
@@ -129,6 +130,24 @@ __device__ __forceinline__ uint32_t qk_block(uint32_t tmem_s, uint64_t q_desc, u
         "tcgen05.mma.cta_group::1.kind::f16 [%1], a5, b5, %4, t;\n"
         "tcgen05.mma.cta_group::1.kind::f16 [%1], a6, b6, %4, t;\n"
         "tcgen05.mma.cta_group::1.kind::f16 [%1], a7, b7, %4, t;\n"
+        "tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%5];\n"
+        "selp.u32 %0, 1, 0, q;\n"
+        "}\n"
+        : "=r"(ready)
+        : "r"(tmem_s), "l"(q_desc), "l"(k_desc), "r"(idesc), "r"(commit_bar), "r"(peek_bar), "r"(peek_parity)
+        : "memory");
+  } else if (KD == 32) {
+    asm volatile(
+        "{\n"
+        ".reg .pred t, f, q;\n"
+        ".reg .b64 a1, b1;\n"
+        "mbarrier.test_wait.parity.shared::cta.b64 q, [%6], %7;\n"
+        "setp.eq.b32 t, 0, 0;\n"
+        "setp.ne.b32 f, 0, 0;\n"
+        "add.u64 a1, %2, 2;\n"
+        "add.u64 b1, %3, 2;\n"
+        "tcgen05.mma.cta_group::1.kind::f16 [%1], %2, %3, %4, f;\n"
+        "tcgen05.mma.cta_group::1.kind::f16 [%1], a1, b1, %4, t;\n"
         "tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%5];\n"
         "selp.u32 %0, 1, 0, q;\n"
         "}\n"
@@ -195,7 +214,9 @@ __device__ __forceinline__ uint32_t pv_block(uint32_t tmem_o, uint32_t tmem_p, u
   return ready;
 }
 
-template <int HD>
+// MAPS 2: query heads 2h and 2h + 1 are the two halves of the HD numbers of row h (the values are the same for both); the row's
+// tile is loaded whole and a block's scores use its half of it and of the keys.
+template <int HD, int MAPS>
 __global__ void __launch_bounds__(NUM_THREADS, 2)
 flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                         const __grid_constant__ CUtensorMap map_v, const int* __restrict__ block_table, int table_width,
@@ -272,7 +293,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     if (lane == 0) {
       mbar_expect_tx(&q_full, Q_BYTES);
 #pragma unroll
-      for (int b = 0; b < SUBS; ++b) tma_load_2d(q_s + b * SUBQ_BYTES, &map_q, &q_full, h * HD + 64 * b, tok0 + row0);
+      for (int b = 0; b < SUBS; ++b) tma_load_2d(q_s + b * SUBQ_BYTES, &map_q, &q_full, (h / MAPS) * HD + 64 * b, tok0 + row0);
       const int* table = block_table + (size_t)s * table_width;
       for (int j = 0; j < n_tiles; ++j) {
         const int st = j % KV_STAGES;
@@ -322,7 +343,10 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       // data that is needed later (mbarrier.test_wait, before its MMAs, read after them); the answers are NOT used
       // to skip the waits below: the tensor-core GEMM's issuer, built the same way, gave up on a stage about once in
       // 10^5 launches when it skipped its wait after a yes, and until that is understood every tile is waited for.
-      const uint64_t q_desc = make_smem_desc(q_addr);
+      // (a map's half starts at the second sub-tile of 64 dims, or 64 bytes into the only one)
+      constexpr uint64_t HALF_Q = HD == 128 ? SUBQ_BYTES / 16 : 4, HALF_K = HD == 128 ? SUBK_BYTES / 16 : 4;
+      const uint64_t q_desc = make_smem_desc(q_addr) + (MAPS > 1 ? (h % MAPS) * HALF_Q : 0);
+      const uint64_t k_half = MAPS > 1 ? (h % MAPS) * HALF_K : 0;
       uint32_t v_ready = 0, k_ready = 0;  // the answers: value tile j, key tile j + 2 (for the S after next) have landed
       auto wait_for = [&](uint64_t* bar, uint32_t parity, int code) -> bool {
         if (mbar_wait_role(bar, parity, ctl, code)) return true;
@@ -334,7 +358,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       auto issue_qk = [&](int j, int jv) {
         const int st = j % KV_STAGES;
         tc_fence_after();
-        v_ready = qk_block<HD>(tmem_base + (uint32_t)((j & 1) * BNK), q_desc, make_smem_desc(smem_u32(k_s + (size_t)st * KV_BYTES)), idesc_qk,
+        v_ready = qk_block<HD / MAPS>(tmem_base + (uint32_t)((j & 1) * BNK), q_desc, make_smem_desc(smem_u32(k_s + (size_t)st * KV_BYTES)) + k_half, idesc_qk,
                                smem_u32(&s_full[j & 1]), smem_u32(&v_full[jv % KV_STAGES]), (uint32_t)((jv / KV_STAGES) & 1));
       };
       if (ok) ok = wait_for(&k_full[0], 0, 14);
@@ -375,6 +399,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     const int r = warp * 32 + lane;
     const int qpos = first_pos + r;
     const int qlow = rl_first_key(qpos, window, chunk);
+    const int last_low = rl_first_key(last_pos, window, chunk);
     // with a cap c the scores become tanh(raw * scale / c) first, and c log2(e) takes the scale's place from there on
     const float exp_scale = softcap != 0.f ? softcap * 1.4426950408889634f : scale_log2;
     const float cap_in = softcap != 0.f ? scale_log2 / exp_scale : 0.f;
@@ -404,8 +429,8 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       }
       tc_fence_after();
       const int key0 = (tile_lo + j) * BNK;
-      // (a chunk's start cuts into a tile only where the tile begins before the chunk of the block's last row)
-      const bool need_mask = key0 + BNK - 1 > first_pos || window != 0 || (chunk != 0 && key0 < rl_first_key(last_pos, 0, chunk));
+      // (a window's or a chunk's start cuts into a tile only where the tile begins before the first key of the block's last row)
+      const bool need_mask = key0 + BNK - 1 > first_pos || key0 < last_low;
       const uint32_t s_addr = lane_addr + (uint32_t)((j & 1) * BNK);
       // this thread's row of S in one round trip
       uint32_t v[BNK];
@@ -520,7 +545,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
 // Head sizes this kernel is built for: 64 and 128 (1 if `hd` is one of them).
 RL_API int rl_flash_prefill_tc_takes(int hd) { return hd == 64 || hd == 128; }
 
-template <int HD>
+template <int HD, int MAPS>
 static int launch_flash_tc(const void* q, int q_stride, int n_tokens, const void* k_pages, const void* v_pages, int n_pages,
                            const int* block_table, int table_width, const int* seq_start, const int* seq_pos0, void* out,
                            int out_stride, int n_seqs, int max_q_len, int H, int K, int window, float scale, int* status,
@@ -531,7 +556,7 @@ static int launch_flash_tc(const void* q, int q_stride, int n_tokens, const void
   if (make_page_map(&map_k, k_pages, n_pages, K, PAGE, HD, PAGE) || make_page_map(&map_v, v_pages, n_pages, K, PAGE, HD, PAGE))
     RL_REFUSE(11, "flash_prefill_tc: cannot describe the cache pages to TMA");
   const size_t smem = SMEM_BYTES_OF(HD);
-  auto kern = flash_prefill_tc_kernel<HD>;
+  auto kern = flash_prefill_tc_kernel<HD, MAPS>;
   if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
     RL_REFUSE(12, "flash_prefill_tc: cannot get %zu bytes of shared memory", smem);
   dim3 grid(H * n_seqs, (max_q_len + BMQ - 1) / BMQ);
@@ -551,7 +576,8 @@ RL_API int rl_flash_prefill_tc(const void* q, int q_stride, int n_tokens, const 
                                int n_pages, const int* block_table, int table_width, const int* seq_start,
                                const int* seq_pos0, void* out, int out_stride, int n_seqs, int max_q_len, int H, int K,
                                int hd, int page_size, int window, float scale, int* status, int wait_test_role,
-                               unsigned int wait_test_ns, const float* sink, int chunk, float softcap, cudaStream_t stream) {
+                               unsigned int wait_test_ns, const float* sink, int chunk, float softcap, int maps, cudaStream_t stream) {
+  if (maps < 1 || maps > 2 || H % maps) RL_REFUSE(9, "flash_prefill_tc: %d maps in %d heads", maps, H);
   if (n_seqs <= 0 || max_q_len <= 0 || H <= 0 || K <= 0 || n_tokens <= 0 || n_pages <= 0)
     RL_REFUSE(1, "flash_prefill_tc: S=%d max_q=%d H=%d K=%d T=%d pages=%d", n_seqs, max_q_len, H, K, n_tokens, n_pages);
   if (!rl_flash_prefill_tc_takes(hd)) RL_REFUSE(2, "flash_prefill_tc: head size %d, this kernel is built for 64 and 128", hd);
@@ -563,9 +589,13 @@ RL_API int rl_flash_prefill_tc(const void* q, int q_stride, int n_tokens, const 
     RL_REFUSE(7, "flash_prefill_tc: H=%d x S=%d blocks or %d query rows exceed the grid", H, n_seqs, max_q_len);
   if (window < 0 || chunk < 0 || softcap < 0.f || status == nullptr || !(scale > 0.f))
     RL_REFUSE(8, "flash_prefill_tc: bad window, chunk, cap or scale, or no status word");
-  if (hd == 64)
-    return launch_flash_tc<64>(q, q_stride, n_tokens, k_pages, v_pages, n_pages, block_table, table_width, seq_start, seq_pos0, out,
-                               out_stride, n_seqs, max_q_len, H, K, window, scale, status, wait_test_role, wait_test_ns, sink, chunk, softcap, stream);
-  return launch_flash_tc<128>(q, q_stride, n_tokens, k_pages, v_pages, n_pages, block_table, table_width, seq_start, seq_pos0, out,
-                              out_stride, n_seqs, max_q_len, H, K, window, scale, status, wait_test_role, wait_test_ns, sink, chunk, softcap, stream);
+#define RL_FTC(HDV, MAPSV)                                                                                                                  \
+  return launch_flash_tc<HDV, MAPSV>(q, q_stride, n_tokens, k_pages, v_pages, n_pages, block_table, table_width, seq_start, seq_pos0, out,  \
+                                     out_stride, n_seqs, max_q_len, H, K, window, scale, status, wait_test_role, wait_test_ns, sink, chunk, \
+                                     softcap, stream)
+  if (hd == 64 && maps == 2) RL_FTC(64, 2);
+  if (hd == 64) RL_FTC(64, 1);
+  if (maps == 2) RL_FTC(128, 2);
+  RL_FTC(128, 1);
+#undef RL_FTC
 }

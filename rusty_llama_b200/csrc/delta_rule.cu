@@ -6,9 +6,10 @@
 //
 // in this order, so the read-out sees the token's own write.  Three kernels and a helper:
 //
-//   short_conv        a causal convolution over time per channel, y_t = act(sum_i w[i][c] x_(t - taps + 1 + i)), through a
+//   short_conv        a causal convolution over time per channel, y_t = act(b[c] + sum_i w[i][c] x_(t - taps + 1 + i)), through a
 //                     record of the last taps - 1 inputs per sequence (zeros before a sequence's start); a second small
-//                     kernel moves the record on after the outputs are made
+//                     kernel moves the record on after the outputs are made.  Where every sequence brings one token
+//                     (a decode step) one kernel does both
 //   delta_prep        per token: q and k heads made unit vectors, x / sqrt(sum(x^2) + eps), q times a constant; k . q per
 //                     head; beta = logistic(b); g = exp(-exp(A_log) softplus(a + dt_bias)): all 32-bit, written as float32
 //   delta_rule        the recurrence, token by token: a block owns 32 columns of one head's state of one sequence, a
@@ -29,7 +30,8 @@ __device__ __forceinline__ float dr_silu(float z) { return z / (1.0f + expf(-z))
 // One thread per (token, channel).  x: [T, >= C] rows; w: [taps][C] (tap i of every channel side by side, the last row the
 // current token's); state: [slots][taps - 1][C], entry j the input at (first position of the step) - (taps - 1) + j.
 template <typename T>
-__global__ void short_conv_kernel(const T* __restrict__ x, int x_stride, const float* __restrict__ w, const float* __restrict__ state,
+__global__ void short_conv_kernel(const T* __restrict__ x, int x_stride, const float* __restrict__ w, const float* __restrict__ bias,
+                                  const float* __restrict__ state,
                                   const int* __restrict__ slot_ids, const int* __restrict__ seq_start, const int* __restrict__ tok_seq,
                                   T* __restrict__ out, int out_stride, int n_tokens, int C, int taps, int silu) {
   const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -39,7 +41,7 @@ __global__ void short_conv_kernel(const T* __restrict__ x, int x_stride, const f
   const int start = seq_start[s];
   const int local = t - start;
   const float* rec = state + (size_t)slot_ids[s] * (taps - 1) * C;
-  float acc = 0.f;
+  float acc = bias ? bias[c] : 0.f;
   for (int i = 0; i < taps; ++i) {
     const int src = local - (taps - 1) + i;
     const float v = src >= 0 ? to_f32(x[(size_t)(start + src) * x_stride + c]) : rec[(size_t)(taps - 1 + src) * C + c];
@@ -50,7 +52,8 @@ __global__ void short_conv_kernel(const T* __restrict__ x, int x_stride, const f
 
 // The same for bfloat16 rows of a multiple of 8 channels that start on 16 bytes: a thread takes 8 neighbouring channels of a token,
 // sixteen bytes a load (32 from the record), the same sums in the same order.
-__global__ void short_conv_rows8_kernel(const bf16* __restrict__ x, int x_stride, const float* __restrict__ w, const float* __restrict__ state,
+__global__ void short_conv_rows8_kernel(const bf16* __restrict__ x, int x_stride, const float* __restrict__ w, const float* __restrict__ bias,
+                                        const float* __restrict__ state,
                                         const int* __restrict__ slot_ids, const int* __restrict__ seq_start, const int* __restrict__ tok_seq,
                                         bf16* __restrict__ out, int out_stride, int n_tokens, int C, int taps, int silu) {
   const int c8s = C >> 3;
@@ -62,6 +65,10 @@ __global__ void short_conv_rows8_kernel(const bf16* __restrict__ x, int x_stride
   const int local = t - start;
   const float* rec = state + (size_t)slot_ids[s] * (taps - 1) * C;
   float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+  if (bias) {
+    load4<float>(bias + c, acc);
+    load4<float>(bias + c + 4, acc + 4);
+  }
   for (int i = 0; i < taps; ++i) {
     const int src = local - (taps - 1) + i;
     float v[8];
@@ -101,29 +108,71 @@ __global__ void short_conv_state_kernel(const T* __restrict__ x, int x_stride, f
   for (int j = 0; j < taps - 1; ++j) rec[(size_t)j * C + c] = keep[j];
 }
 
-RL_API int rl_short_conv(const void* x, int dtype, int x_stride, const float* w, float* state, const int* slot_ids, const int* seq_start,
+// Every sequence brings one token: one thread per (sequence, channel) makes the output (the same sum in the same order as above) and
+// moves the record on.
+template <typename T>
+__global__ void short_conv_step_kernel(const T* __restrict__ x, int x_stride, const float* __restrict__ w, const float* __restrict__ bias,
+                                       float* __restrict__ state, const int* __restrict__ slot_ids, T* __restrict__ out, int out_stride,
+                                       int n_seqs, int C, int taps, int silu) {
+  pdl_trigger();
+  pdl_wait();
+  const int idx = blockIdx.x * blockDim.x + threadIdx.x;
+  if (idx >= n_seqs * C) return;
+  const int s = idx / C, c = idx - s * C;
+  float* rec = state + (size_t)slot_ids[s] * (taps - 1) * C + c;
+  float v[CONV_MAX_TAPS];
+#pragma unroll
+  for (int i = 0; i < CONV_MAX_TAPS; ++i)
+    if (i < taps - 1) v[i] = __ldcg(rec + (size_t)i * C);
+  const float now = to_f32(__ldcg(x + (size_t)s * x_stride + c));
+  float acc = bias ? bias[c] : 0.f;
+#pragma unroll
+  for (int i = 0; i < CONV_MAX_TAPS; ++i)
+    if (i < taps - 1) acc += w[(size_t)i * C + c] * v[i];
+  acc += w[(size_t)(taps - 1) * C + c] * now;
+#pragma unroll
+  for (int i = 0; i < CONV_MAX_TAPS; ++i)
+    if (i < taps - 1) rec[(size_t)i * C] = i + 1 < taps - 1 ? v[(i + 1) & (CONV_MAX_TAPS - 1)] : now;
+  out[(size_t)s * out_stride + c] = from_f32<T>(silu ? dr_silu(acc) : acc);
+}
+
+// single: the host knows that every sequence brings exactly one token.
+RL_API int rl_short_conv(const void* x, int dtype, int x_stride, const float* w, const float* bias, float* state, const int* slot_ids, const int* seq_start,
                          const int* tok_seq, void* out, int out_stride, int n_tokens, int n_seqs, int C, int taps, int silu,
-                         cudaStream_t stream) {
+                         int single, cudaStream_t stream) {
   if (n_tokens <= 0 || n_seqs <= 0 || C <= 0) RL_REFUSE(1, "short_conv: T=%d S=%d C=%d", n_tokens, n_seqs, C);
   if (taps < 1 || taps > CONV_MAX_TAPS) RL_REFUSE(2, "short_conv: %d taps (1 to %d)", taps, CONV_MAX_TAPS);
   if (x_stride < C || out_stride < C) RL_REFUSE(3, "short_conv: rows shorter than %d channels", C);
   if (taps > 1 && state == nullptr) RL_REFUSE(4, "short_conv: no record of earlier inputs");
+  if (single && n_tokens != n_seqs) RL_REFUSE(6, "short_conv: %d tokens of %d sequences are not one each", n_tokens, n_seqs);
   const int threads = 256;
   const long long total = (long long)n_tokens * C, total_s = (long long)n_seqs * C;
+  if (single && total <= 0x7fffff00LL) {
+    const int blocks1 = (int)((total + 127) / 128);
+    if (dtype == RL_BF16)
+      RL_LAUNCH_CHECK(rl_launch(short_conv_step_kernel<bf16>, blocks1, 128, 0, stream, (const bf16*)x, x_stride, w, bias, state, slot_ids, (bf16*)out,
+                                out_stride, n_seqs, C, taps, silu));
+    else if (dtype == RL_F32)
+      RL_LAUNCH_CHECK(rl_launch(short_conv_step_kernel<float>, blocks1, 128, 0, stream, (const float*)x, x_stride, w, bias, state, slot_ids,
+                                (float*)out, out_stride, n_seqs, C, taps, silu));
+    else
+      RL_REFUSE(5, "short_conv: unknown dtype %d", dtype);
+    return 0;
+  }
   const int blocks = (int)((total + threads - 1) / threads), blocks_s = (int)((total_s + threads - 1) / threads);
   if (dtype == RL_BF16) {
     // (which of the two kernels runs depends on sizes and addresses only, never on the batch)
-    const bool rows8 = C % 8 == 0 && x_stride % 8 == 0 && out_stride % 8 == 0 && ((((uintptr_t)x | (uintptr_t)out | (uintptr_t)state | (uintptr_t)w) & 15) == 0);
+    const bool rows8 = C % 8 == 0 && x_stride % 8 == 0 && out_stride % 8 == 0 && ((((uintptr_t)x | (uintptr_t)out | (uintptr_t)state | (uintptr_t)w | (uintptr_t)bias) & 15) == 0);
     if (rows8)
-      short_conv_rows8_kernel<<<(int)((total / 8 + threads - 1) / threads), threads, 0, stream>>>((const bf16*)x, x_stride, w, state, slot_ids, seq_start,
+      short_conv_rows8_kernel<<<(int)((total / 8 + threads - 1) / threads), threads, 0, stream>>>((const bf16*)x, x_stride, w, bias, state, slot_ids, seq_start,
                                                                                                    tok_seq, (bf16*)out, out_stride, n_tokens, C, taps, silu);
     else
-      short_conv_kernel<bf16><<<blocks, threads, 0, stream>>>((const bf16*)x, x_stride, w, state, slot_ids, seq_start, tok_seq, (bf16*)out,
+      short_conv_kernel<bf16><<<blocks, threads, 0, stream>>>((const bf16*)x, x_stride, w, bias, state, slot_ids, seq_start, tok_seq, (bf16*)out,
                                                               out_stride, n_tokens, C, taps, silu);
     if (taps > 1)
       short_conv_state_kernel<bf16><<<blocks_s, threads, 0, stream>>>((const bf16*)x, x_stride, state, slot_ids, seq_start, n_seqs, C, taps);
   } else if (dtype == RL_F32) {
-    short_conv_kernel<float><<<blocks, threads, 0, stream>>>((const float*)x, x_stride, w, state, slot_ids, seq_start, tok_seq, (float*)out,
+    short_conv_kernel<float><<<blocks, threads, 0, stream>>>((const float*)x, x_stride, w, bias, state, slot_ids, seq_start, tok_seq, (float*)out,
                                                              out_stride, n_tokens, C, taps, silu);
     if (taps > 1)
       short_conv_state_kernel<float><<<blocks_s, threads, 0, stream>>>((const float*)x, x_stride, state, slot_ids, seq_start, n_seqs, C, taps);

@@ -545,3 +545,154 @@ RL_API int rl_normed_add_rmsnorm(float* x, const void* delta, int delta_dtype, i
 #undef RL_NN
   RL_REFUSE(5, "normed_add_rmsnorm: unsupported dtypes act=%d w=%d delta=%d", act_dtype, w_dtype, delta_dtype);
 }
+
+// ---------------------------------------------------------------- a gated sublayer result, the residual sum, a norm in groups
+// For output row r (stream row t = rows ? rows[r] : r):
+//   s = delta[0][t] + delta[1][t] + ...                                       (32-bit, in this order)
+//   v = x[t] + s * logistic(z[t] + bias)        (without a gate: x[t] + s)    x[t] = v
+//   if w: the row cut into `groups` equal consecutive parts, out[r] = v / sqrt(mean(v^2 over its part) + eps) * w
+// One block per row, the row in registers.  A unit is U neighbouring values (four where the sizes allow); every unit leaves its
+// sum of squares in shared memory, a warp per part adds them up in an order that depends on the sizes alone.  So a row's bits
+// depend neither on the number of rows nor on how many threads work it: the launcher takes few threads with several units each
+// for the many rows of a prompt step and a thread per unit for the few rows of a decode step.
+template <typename TA, typename TW, typename TD, int U, int UNITS>
+__global__ void __launch_bounds__(UNITS == 4 ? 256 : 1024)
+gated_add_rmsnorm_kernel(float* __restrict__ x, const TD* __restrict__ delta, int n_parts, long long part_stride,
+                         const TA* __restrict__ z, int z_stride, const float* __restrict__ gate_bias, const TW* __restrict__ w,
+                         TA* __restrict__ out, const int* __restrict__ rows, int d, int groups, float eps, int write_x) {
+  extern __shared__ __align__(16) float unit_ss[];  // [d / U], then 1 / rms of the parts [groups]
+  pdl_trigger();
+  pdl_wait();
+  const int r = blockIdx.x;
+  const int t = rows ? rows[r] : r;
+  const int n_units = d / U, per_group = n_units / groups;
+  float* inv_rms = unit_ss + n_units;
+  float* xr = x + (size_t)t * d;
+  float v[UNITS][U], wv[UNITS][U];
+#pragma unroll
+  for (int c = 0; c < UNITS; ++c) {
+    const int u = threadIdx.x + c * blockDim.x, i = u * U;
+    if (u >= n_units) continue;
+    float s[U], zv[U];
+#pragma unroll
+    for (int e = 0; e < U; ++e) s[e] = 0.f;
+    if (U == 4) {
+      load4_g<float>(xr + i, v[c]);
+      if (w != nullptr) load4_g<TW>(w + i, wv[c]);
+      if (z != nullptr) load4_g<TA>(z + (size_t)t * z_stride + i, zv);
+    } else {
+      v[c][0] = xr[i];
+      if (w != nullptr) wv[c][0] = to_f32(w[i]);
+      if (z != nullptr) zv[0] = to_f32(z[(size_t)t * z_stride + i]);
+    }
+    for (int p = 0; p < n_parts; ++p) {
+      float dv[U];
+      const TD* dp = delta + (size_t)p * part_stride + (size_t)t * d + i;
+      if (U == 4) load4_g<TD>(dp, dv);
+      else dv[0] = to_f32(dp[0]);
+#pragma unroll
+      for (int e = 0; e < U; ++e) s[e] += dv[e];
+    }
+    if (z != nullptr) {
+#pragma unroll
+      for (int e = 0; e < U; ++e) s[e] *= 1.0f / (1.0f + expf(-(zv[e] + gate_bias[i + e])));
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < U; ++e) {
+      v[c][e] += s[e];
+      ss += v[c][e] * v[c][e];
+    }
+    if (write_x) {
+      if (U == 4) store4<float>(xr + i, v[c]);
+      else xr[i] = v[c][0];
+    }
+    unit_ss[u] = ss;
+  }
+  if (w == nullptr) return;
+  __syncthreads();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
+  for (int g = warp; g < groups; g += nwarps) {
+    float ss = 0.f;
+    for (int u = lane; u < per_group; u += 32) ss += unit_ss[g * per_group + u];
+    ss = warp_sum(ss);
+    if (lane == 0) inv_rms[g] = 1.0f / sqrtf(ss / (float)(per_group * U) + eps);
+  }
+  __syncthreads();
+  TA* o = out + (size_t)r * d;
+#pragma unroll
+  for (int c = 0; c < UNITS; ++c) {
+    const int u = threadIdx.x + c * blockDim.x, i = u * U;
+    if (u >= n_units) continue;
+    const float inv = inv_rms[u / per_group];
+    float y[U];
+#pragma unroll
+    for (int e = 0; e < U; ++e) y[e] = v[c][e] * inv * wv[c][e];
+    if (U == 4) store4<TA>(o + i, y);
+    else o[i] = from_f32<TA>(y[0]);
+  }
+}
+
+template <typename TA, typename TW, typename TD>
+static int launch_gated_add_rmsnorm(float* x, const void* delta, int n_parts, long long part_stride, const void* z, int z_stride,
+                                    const float* gate_bias, const void* w, void* out, const int* rows, int n_rows, int d, int groups,
+                                    float eps, int write_x, cudaStream_t stream) {
+  // (which body runs depends on sizes and addresses only)
+  const bool vec = (d / groups) % 4 == 0 && z_stride % 4 == 0 && part_stride % 4 == 0 &&
+                   (((uintptr_t)x | (uintptr_t)delta | (uintptr_t)z | (uintptr_t)w | (uintptr_t)out) % 16 == 0);
+  const int n_units = vec ? d / 4 : d;
+  const size_t smem = (size_t)(n_units + groups) * sizeof(float);
+  if (n_units > 8 * 1024 || smem > 48 * 1024) RL_REFUSE(3, "gated_add_rmsnorm: a row of %d values (%d parts) is too long", d, groups);
+  const int full = n_units >= 1024 ? 1024 : ((n_units + 31) / 32) * 32;
+#define RL_GAR(U, UNITS, TH, EARLY)                                                                                                    \
+  do {                                                                                                                                 \
+    RL_LAUNCH_CHECK(rl_launch<EARLY>(gated_add_rmsnorm_kernel<TA, TW, TD, U, UNITS>, n_rows, TH, smem, stream, x, (const TD*)delta, n_parts, \
+                                     part_stride, (const TA*)z, z_stride, gate_bias, (const TW*)w, (TA*)out, rows, d, groups, eps, write_x)); \
+    return 0;                                                                                                                          \
+  } while (0)
+  if (vec) {
+    if (n_rows >= ROWS_KERNEL_MIN_ROWS && n_units > 256 && n_units <= 1024) RL_GAR(4, 4, 256, true);
+    if (n_units <= 1024) RL_GAR(4, 1, full, true);
+    RL_GAR(4, 8, 1024, true);
+  }
+  if (n_units <= 1024) RL_GAR(1, 1, full, false);
+  RL_GAR(1, 8, 1024, false);
+#undef RL_GAR
+}
+
+RL_API int rl_gated_add_rmsnorm(float* x, const void* delta, int delta_dtype, int n_parts, long long part_stride, const void* z, int z_stride,
+                                const float* gate_bias, const void* w, int w_dtype, void* out, int act_dtype, const int* rows, int n_rows,
+                                int d, int groups, float eps, int write_x, cudaStream_t stream) {
+  if (n_rows <= 0 || d <= 0 || n_parts < 0 || groups <= 0 || d % groups) RL_REFUSE(1, "gated_add_rmsnorm: n_rows=%d d=%d n_parts=%d groups=%d", n_rows, d, n_parts, groups);
+  if (n_parts > 0 && delta == nullptr) RL_REFUSE(2, "gated_add_rmsnorm: %d parts but no delta", n_parts);
+  if ((w != nullptr && out == nullptr) || (z != nullptr && gate_bias == nullptr)) RL_REFUSE(2, "gated_add_rmsnorm: a weight without an output or a gate without its bias");
+  if (n_parts == 0) delta_dtype = act_dtype;
+#define RL_GN(TA, TW, TD) \
+  return launch_gated_add_rmsnorm<TA, TW, TD>(x, delta, n_parts, part_stride, z, z_stride, gate_bias, w, out, rows, n_rows, d, groups, eps, write_x, stream)
+  if (act_dtype == RL_BF16 && w_dtype == RL_F32 && delta_dtype == RL_BF16) RL_GN(bf16, float, bf16);
+  if (act_dtype == RL_BF16 && w_dtype == RL_F32 && delta_dtype == RL_F32) RL_GN(bf16, float, float);
+  if (act_dtype == RL_BF16 && w_dtype == RL_BF16 && delta_dtype == RL_BF16) RL_GN(bf16, bf16, bf16);
+  if (act_dtype == RL_BF16 && w_dtype == RL_BF16 && delta_dtype == RL_F32) RL_GN(bf16, bf16, float);
+  if (act_dtype == RL_F32 && w_dtype == RL_F32 && delta_dtype == RL_F32) RL_GN(float, float, float);
+#undef RL_GN
+  RL_REFUSE(5, "gated_add_rmsnorm: unsupported dtypes act=%d w=%d delta=%d", act_dtype, w_dtype, delta_dtype);
+}
+
+// ---------------------------------------------------------------- logits: a constant factor and a cap
+// y <- y * scale, then y <- cap tanh(y / cap) where cap > 0; in place, 32-bit.
+__global__ void scale_softcap_kernel(float* __restrict__ y, long long total, float scale, float cap) {
+  pdl_trigger();
+  pdl_wait();
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const float v = __ldcg(y + i) * scale;
+    y[i] = cap > 0.f ? cap * tanhf(v / cap) : v;
+  }
+}
+
+RL_API int rl_scale_softcap(float* y, long long total, float scale, float cap, cudaStream_t stream) {
+  if (total <= 0 || cap < 0.f) RL_REFUSE(1, "scale_softcap: %lld numbers, cap %g", total, (double)cap);
+  long long blocks = (total + 255) / 256;
+  if (blocks > 148 * 8) blocks = 148 * 8;
+  RL_LAUNCH_CHECK(rl_launch(scale_softcap_kernel, (int)blocks, 256, 0, stream, y, total, scale, cap));
+  return 0;
+}

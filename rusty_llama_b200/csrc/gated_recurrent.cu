@@ -3,10 +3,11 @@
 //   S_t = diag(a_t) S_(t-1) + b_t k_t v_t^T,   o_t = S_t^T (c q_t)        per head; S is [dim, vcols]
 //
 // a_t = exp(log_decay_t) is one number per key channel (a row of `dim`) or one per head; b_t is one number per head or 1;
-// c is a constant.  With `ext` the state has one more column that is fed with v = 1: it carries n_t = a_t n_(t-1) + b_t k_t,
-// and the output's last column is n_t . q_t, the normaliser of a matrix memory.  Two designs use it:
+// c is a constant.  q and k may have fewer heads than v (`qk_heads`: head h reads q/k head h / (H / qk_heads)).  With `ext` the state has one more column that is fed with v = 1: it carries n_t = a_t n_(t-1) + b_t k_t,
+// and the output's last column is n_t . q_t, the normaliser of a matrix memory.  Three kinds of layer use it:
 //
 //   gated linear attention   a_t = sigmoid(z_t)^(1/tau) per channel (`gla_log_decay` makes log a_t), b = 1
+//   state-space layer        a_t = exp(-rate_h dt_t), b_t = dt_t per head, q and k shared by groups of heads (csrc/state_space.cu)
 //   matrix memory (mLSTM)    log gates i_t, f_t per head with a running maximum m_t = max(f_t + m_(t-1), i_t):
 //                            a_t = exp(f_t + m_(t-1) - m_t), b_t = exp(i_t - m_t) (`mlstm_gates`), `ext` column,
 //                            o_t / (max(|n_t . q_t|, exp(-m_t)) + c_den) in `head_norm_gate`
@@ -198,12 +199,12 @@ template <typename T>
 __global__ void gated_attn_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, int in_stride,
                                   const float* __restrict__ log_decay, int per_channel, const float* __restrict__ in_scale, float q_scale,
                                   float* __restrict__ state, const int* __restrict__ slot_ids, const int* __restrict__ seq_start,
-                                  float* __restrict__ out, int out_stride, int H, int dim, int vdim, int ext) {
+                                  float* __restrict__ out, int out_stride, int H, int QH, int dim, int vdim, int ext) {
   extern __shared__ float sm[];
   pdl_trigger();
   pdl_wait();
   const int lane = threadIdx.x & 31, w = threadIdx.x >> 5, nw = blockDim.x >> 5;
-  const int s = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * 32;
+  const int s = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * 32, qh = h / (H / QH);
   const int vcols = vdim + ext;
   const int col = col0 + lane;
   const bool col_ok = col < vcols;
@@ -225,7 +226,7 @@ __global__ void gated_attn_kernel(const T* __restrict__ q, const T* __restrict__
     for (int idx = threadIdx.x; idx < n * dim; idx += blockDim.x) {
       const int j = idx / dim, i = idx - j * dim;
       const int t = base + j;
-      const size_t at = (size_t)t * in_stride + (size_t)h * dim + i;
+      const size_t at = (size_t)t * in_stride + (size_t)qh * dim + i;
       const float b = in_scale ? in_scale[(size_t)t * H + h] : 1.f;
       q_s[idx] = to_f32(q[at]) * q_scale;
       k_s[idx] = to_f32(k[at]) * b;
@@ -274,7 +275,8 @@ __global__ void gated_attn_kernel(const T* __restrict__ q, const T* __restrict__
 
 RL_API int rl_gated_attn(const void* q, const void* k, const void* v, int dtype, int in_stride, const float* log_decay, int per_channel,
                          const float* in_scale, float q_scale, float* state, const int* slot_ids, const int* seq_start, float* out,
-                         int out_stride, int n_seqs, int H, int dim, int vdim, int ext, cudaStream_t stream) {
+                         int out_stride, int n_seqs, int H, int QH, int dim, int vdim, int ext, cudaStream_t stream) {
+  if (QH <= 0 || H % QH) RL_REFUSE(6, "gated_attn: %d heads are not a multiple of %d q/k heads", H, QH);
   if (n_seqs <= 0 || H <= 0 || dim <= 0 || vdim <= 0 || (ext != 0 && ext != 1) || !log_decay)
     RL_REFUSE(1, "gated_attn: S=%d H=%d dim=%d vdim=%d ext=%d", n_seqs, H, dim, vdim, ext);
   if (dim > 1024) RL_REFUSE(2, "gated_attn: key size %d exceeds 1024", dim);
@@ -291,8 +293,8 @@ RL_API int rl_gated_attn(const void* q, const void* k, const void* v, int dtype,
       if (e != cudaSuccess) RL_REFUSE(4, "gated_attn: %zu bytes of shared memory refused", smem);                                  \
     }                                                                                                                              \
     RL_LAUNCH_CHECK(rl_launch(gated_attn_kernel<T>, grid, nw * 32, smem, stream, (const T*)q, (const T*)k, (const T*)v, in_stride,  \
-                              log_decay, per_channel, in_scale, q_scale, state, slot_ids, seq_start, out, out_stride, H, dim, vdim, \
-                              ext));                                                                                               \
+                              log_decay, per_channel, in_scale, q_scale, state, slot_ids, seq_start, out, out_stride, H, QH, dim,   \
+                              vdim, ext));                                                                                               \
   } while (0)
   if (dtype == RL_BF16) RL_GA(bf16);
   else if (dtype == RL_F32) RL_GA(float);
@@ -336,11 +338,11 @@ template <typename T>
 __global__ void __launch_bounds__(256)
 gated_chunk_state_kernel(const T* __restrict__ k, const T* __restrict__ v, int in_stride, const float* __restrict__ log_decay,
                          int per_channel, const float* __restrict__ in_scale, const int* __restrict__ seq_start,
-                         float* __restrict__ scratch, float* __restrict__ chunk_decay, int max_chunks, int H, int dim, int vdim, int ext) {
+                         float* __restrict__ scratch, float* __restrict__ chunk_decay, int max_chunks, int H, int QH, int dim, int vdim, int ext) {
   extern __shared__ float sm[];
   pdl_trigger();
   pdl_wait();
-  const int s = blockIdx.x / H, h = blockIdx.x % H, c = blockIdx.y, col0 = blockIdx.z * GC_COLS;
+  const int s = blockIdx.x / H, h = blockIdx.x % H, c = blockIdx.y, col0 = blockIdx.z * GC_COLS, qh = h / (H / QH);
   const int vcols = vdim + ext;
   const int t0 = seq_start[s] + c * GC;
   const int n = min(GC, seq_start[s + 1] - t0);
@@ -381,7 +383,7 @@ gated_chunk_state_kernel(const T* __restrict__ k, const T* __restrict__ v, int i
   for (int idx = threadIdx.x; idx < n * dim; idx += 256) {
     const int i = idx / dim, r = idx - i * dim;
     const float b = in_scale ? in_scale[(size_t)(t0 + i) * H + h] : 1.f;
-    k_s[idx] = to_f32(k[(size_t)(t0 + i) * in_stride + (size_t)h * dim + r]) * b * gr_exp2(k_s[idx]);
+    k_s[idx] = to_f32(k[(size_t)(t0 + i) * in_stride + (size_t)qh * dim + r]) * b * gr_exp2(k_s[idx]);
   }
   __syncthreads();
   const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
@@ -468,11 +470,11 @@ __global__ void __launch_bounds__(256)
 gated_chunk_out_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, int in_stride,
                        const float* __restrict__ log_decay, int per_channel, const float* __restrict__ in_scale, float q_scale,
                        const int* __restrict__ seq_start, const float* __restrict__ scratch, int max_chunks, float* __restrict__ out,
-                       int out_stride, int H, int dim, int vdim, int ext) {
+                       int out_stride, int H, int QH, int dim, int vdim, int ext) {
   extern __shared__ float sm[];
   pdl_trigger();
   pdl_wait();
-  const int s = blockIdx.x / H, h = blockIdx.x % H, c = blockIdx.y;
+  const int s = blockIdx.x / H, h = blockIdx.x % H, c = blockIdx.y, qh = h / (H / QH);
   const int vcols = vdim + ext;
   const int t0 = seq_start[s] + c * GC;
   const int n = min(GC, seq_start[s + 1] - t0);
@@ -494,7 +496,7 @@ gated_chunk_out_kernel(const T* __restrict__ q, const T* __restrict__ k, const T
     const int i = idx / dim, r = idx - i * dim;
     float qv = 0.f, kv = 0.f, la = 0.f;
     if (i < n) {
-      const size_t at = (size_t)(t0 + i) * in_stride + (size_t)h * dim + r;
+      const size_t at = (size_t)(t0 + i) * in_stride + (size_t)qh * dim + r;
       const size_t th = (size_t)(t0 + i) * H + h;
       qv = to_f32(q[at]) * q_scale;
       kv = to_f32(k[at]) * (in_scale ? in_scale[th] : 1.f);
@@ -667,7 +669,8 @@ RL_API int rl_gated_attn_chunked_takes(int dim) { return dim > 0 && gated_chunk_
 RL_API int rl_gated_attn_chunked(const void* q, const void* k, const void* v, int dtype, int in_stride, const float* log_decay,
                                  int per_channel, const float* in_scale, float q_scale, float* state, const int* slot_ids,
                                  const int* seq_start, float* scratch, float* out, int out_stride, int n_seqs, int max_q_len, int H,
-                                 int dim, int vdim, int ext, cudaStream_t stream) {
+                                 int QH, int dim, int vdim, int ext, cudaStream_t stream) {
+  if (QH <= 0 || H % QH) RL_REFUSE(6, "gated_attn_chunked: %d heads are not a multiple of %d q/k heads", H, QH);
   if (n_seqs <= 0 || max_q_len <= 0 || H <= 0 || dim <= 0 || vdim <= 0 || (ext != 0 && ext != 1) || !log_decay || !scratch)
     RL_REFUSE(1, "gated_attn_chunked: S=%d max_q=%d H=%d dim=%d vdim=%d ext=%d", n_seqs, max_q_len, H, dim, vdim, ext);
   if (!rl_gated_attn_chunked_takes(dim)) RL_REFUSE(2, "gated_attn_chunked: key size %d needs more shared memory than an SM has", dim);
@@ -685,12 +688,12 @@ RL_API int rl_gated_attn_chunked(const void* q, const void* k, const void* v, in
         cudaFuncSetAttribute(gated_chunk_out_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem3) != cudaSuccess)     \
       RL_REFUSE(4, "gated_attn_chunked: %zu bytes of shared memory refused", smem3);                                                 \
     RL_LAUNCH_CHECK(rl_launch(gated_chunk_state_kernel<T>, grid, 256, smem1, stream, (const T*)k, (const T*)v, in_stride, log_decay,  \
-                              per_channel, in_scale, seq_start, scratch, chunk_decay, max_chunks, H, dim, vdim, ext));               \
+                              per_channel, in_scale, seq_start, scratch, chunk_decay, max_chunks, H, QH, dim, vdim, ext));           \
     RL_LAUNCH_CHECK(rl_launch(gated_chunk_scan_kernel, grid2, 256, 0, stream, state, slot_ids, seq_start, scratch,                   \
                               (const float*)chunk_decay, max_chunks, H, dim, vcols));                                                \
     RL_LAUNCH_CHECK(rl_launch(gated_chunk_out_kernel<T>, grid3, 256, smem3, stream, (const T*)q, (const T*)k, (const T*)v, in_stride,  \
                               log_decay, per_channel, in_scale, q_scale, seq_start, (const float*)scratch, max_chunks, out,          \
-                              out_stride, H, dim, vdim, ext));                                                                       \
+                              out_stride, H, QH, dim, vdim, ext));                                                                   \
   } while (0)
   if (dtype == RL_BF16) RL_GC(bf16);
   else if (dtype == RL_F32) RL_GC(float);

@@ -11,7 +11,9 @@
 //
 //   latent_prep    per token: RMS-norm of the latent, rotation of the shared key part, both stored into the
 //                  token's place in the paged cache; rotation of every head's rotated query part into the
-//                  tail of the head's row of q_cat[T, H, rank + rot]
+//                  tail of the head's row of q_cat[T, H, rank + rot]; RMS-norm of the queries' own latent where the
+//                  queries are made from one (each of the three is optional: queries that are made from a latent exist
+//                  only after the product that follows its norm)
 //   head_linear    out[t,h,:] = W[h] x[t,h,:], one small product per head (the two absorbed maps), optionally
 //                  times sigmoid(gate[t,h,:]) (the mixer's output gate)
 //   latent_attn    softmax attention with a sink over the cached rows; any sizes, both element types, keys
@@ -25,21 +27,51 @@
 RL_DEFINE_ERROR_TEXT()
 
 // ---------------------------------------------------------------- norm, rotation, cache write
-// Pair i of a rotated part, dimensions (2i, 2i+1), turns by pos * freq[i]; cos and sin are multiplied by
-// `mag`; pairs from n_pairs on pass unchanged.  Everything in 32-bit, rounded once when stored.
+// Pair i of a rotated part, dimensions (2i, 2i+1) or, not `interleaved`, (i, i + n_pairs), turns by pos * freq[i]; cos and sin are
+// multiplied by `mag`; dimensions from 2 n_pairs on pass unchanged.  Everything in 32-bit, rounded once when stored.
+template <typename T>
+__device__ __forceinline__ void turn_pair(const T* __restrict__ src, T* __restrict__ dst, int i, int n_pairs, int interleaved, int pos,
+                                          const float* __restrict__ freq, float mag) {
+  const bool halves = !interleaved && i < n_pairs;
+  const int d0 = halves ? i : 2 * i, d1 = halves ? i + n_pairs : 2 * i + 1;
+  float u = to_f32(src[d0]), v = to_f32(src[d1]);
+  if (i < n_pairs) {
+    float s, c;
+    sincosf((float)pos * freq[i], &s, &c);
+    s *= mag;
+    c *= mag;
+    const float a = u * c - v * s, b = v * c + u * s;
+    u = a;
+    v = b;
+  }
+  dst[d0] = from_f32<T>(u);
+  dst[d1] = from_f32<T>(v);
+}
+
 template <typename T>
 __global__ void latent_prep_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ kv, int ldkv,
                                    const float* __restrict__ norm_w, float eps, const float* __restrict__ freq,
-                                   int n_pairs, float mag, const int* __restrict__ tok_pos,
+                                   int n_pairs, int interleaved, float mag, const int* __restrict__ tok_pos,
                                    const int* __restrict__ tok_seq, const int* __restrict__ block_table,
                                    int table_width, T* __restrict__ pages, int page_size, T* __restrict__ q_cat,
-                                   int H, int dim, int rot, int rank) {
+                                   int H, int dim, int rot, int rank, const T* __restrict__ ql, int ldql, int q_rank,
+                                   const float* __restrict__ q_norm_w, T* __restrict__ ql_out) {
   __shared__ float red[32];
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x;
   const int pos = tok_pos[t];
   const int Dk = rank + rot;
+  if (ql != nullptr) {
+    const T* row = ql + (size_t)t * ldql;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < q_rank; i += blockDim.x) {
+      const float v = to_f32(row[i]);
+      ss += v * v;
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)q_rank + eps);
+    for (int i = threadIdx.x; i < q_rank; i += blockDim.x) ql_out[(size_t)t * q_rank + i] = from_f32<T>(to_f32(row[i]) * inv * q_norm_w[i]);
+  }
   if (kv != nullptr) {
     const T* row = kv + (size_t)t * ldkv;
     const int page = block_table[(size_t)tok_seq[t] * table_width + pos / page_size];
@@ -51,62 +83,42 @@ __global__ void latent_prep_kernel(const T* __restrict__ q, int ldq, const T* __
     }
     const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)rank + eps);
     for (int i = threadIdx.x; i < rank; i += blockDim.x) dst[i] = from_f32<T>(to_f32(row[i]) * inv * norm_w[i]);
-    for (int i = threadIdx.x; i < rot / 2; i += blockDim.x) {
-      float u = to_f32(row[rank + 2 * i]), v = to_f32(row[rank + 2 * i + 1]);
-      if (i < n_pairs) {
-        float s, c;
-        sincosf((float)pos * freq[i], &s, &c);
-        s *= mag;
-        c *= mag;
-        const float a = u * c - v * s, b = v * c + u * s;
-        u = a;
-        v = b;
-      }
-      dst[rank + 2 * i] = from_f32<T>(u);
-      dst[rank + 2 * i + 1] = from_f32<T>(v);
-    }
+    for (int i = threadIdx.x; i < rot / 2; i += blockDim.x) turn_pair(row + rank, dst + rank, i, n_pairs, interleaved, pos, freq, mag);
     if ((rot & 1) && threadIdx.x == 0) dst[rank + rot - 1] = row[rank + rot - 1];
   }
+  if (q == nullptr) return;
   const int half = rot / 2;
   for (int idx = threadIdx.x; idx < H * half; idx += blockDim.x) {
     const int h = idx / half, i = idx % half;
-    const T* src = q + (size_t)t * ldq + (size_t)h * (dim + rot) + dim;
-    float u = to_f32(src[2 * i]), v = to_f32(src[2 * i + 1]);
-    if (i < n_pairs) {
-      float s, c;
-      sincosf((float)pos * freq[i], &s, &c);
-      s *= mag;
-      c *= mag;
-      const float a = u * c - v * s, b = v * c + u * s;
-      u = a;
-      v = b;
-    }
-    T* dst = q_cat + ((size_t)t * H + h) * Dk + rank;
-    dst[2 * i] = from_f32<T>(u);
-    dst[2 * i + 1] = from_f32<T>(v);
+    turn_pair(q + (size_t)t * ldq + (size_t)h * (dim + rot) + dim, q_cat + ((size_t)t * H + h) * Dk + rank, i, n_pairs, interleaved, pos, freq, mag);
   }
   if (rot & 1)
     for (int h = threadIdx.x; h < H; h += blockDim.x)
       q_cat[((size_t)t * H + h) * Dk + rank + rot - 1] = q[(size_t)t * ldq + (size_t)h * (dim + rot) + dim + rot - 1];
 }
 
+// q, kv, ql: each may be null, its part of the work is then left out.  ql: [T, >= q_rank] rows, the queries' latent; ql_out: [T, q_rank].
 RL_API int rl_latent_prep(const void* q, int ldq, const void* kv, int ldkv, int dtype, const float* norm_w, float eps,
-                          const float* freq, int n_pairs, float mag, const int* tok_pos, const int* tok_seq,
+                          const float* freq, int n_pairs, int interleaved, float mag, const int* tok_pos, const int* tok_seq,
                           const int* block_table, int table_width, void* pages, int page_size, void* q_cat,
-                          int n_tokens, int H, int dim, int rot, int rank, cudaStream_t stream) {
+                          int n_tokens, int H, int dim, int rot, int rank, const void* ql, int ldql, int q_rank, const float* q_norm_w,
+                          void* ql_out, cudaStream_t stream) {
   if (n_tokens <= 0 || H <= 0 || dim < 0 || rot < 0 || rank <= 0 || page_size <= 0)
     RL_REFUSE(1, "latent_prep: T=%d H=%d dim=%d rot=%d rank=%d page=%d", n_tokens, H, dim, rot, rank, page_size);
   if (2 * n_pairs > rot) RL_REFUSE(2, "latent_prep: %d rotated pairs do not fit %d dimensions", n_pairs, rot);
   if (kv != nullptr && (pages == nullptr || block_table == nullptr || norm_w == nullptr))
     RL_REFUSE(3, "latent_prep: a latent row to store, but no pages, page table or norm weight");
+  if (ql != nullptr && (q_rank <= 0 || ldql < q_rank || q_norm_w == nullptr || ql_out == nullptr))
+    RL_REFUSE(5, "latent_prep: a query latent of %d in rows of %d needs a norm weight and an output", q_rank, ldql);
+  if (q != nullptr && q_cat == nullptr) RL_REFUSE(6, "latent_prep: queries to turn, but nowhere to put them");
   if (dtype == RL_BF16)
     RL_LAUNCH_CHECK(rl_launch<false>(latent_prep_kernel<bf16>, n_tokens, 128, 0, stream, (const bf16*)q, ldq, (const bf16*)kv, ldkv,
-                              norm_w, eps, freq, n_pairs, mag, tok_pos, tok_seq, block_table, table_width, (bf16*)pages,
-                              page_size, (bf16*)q_cat, H, dim, rot, rank));
+                              norm_w, eps, freq, n_pairs, interleaved, mag, tok_pos, tok_seq, block_table, table_width, (bf16*)pages,
+                              page_size, (bf16*)q_cat, H, dim, rot, rank, (const bf16*)ql, ldql, q_rank, q_norm_w, (bf16*)ql_out));
   else if (dtype == RL_F32)
     RL_LAUNCH_CHECK(rl_launch<false>(latent_prep_kernel<float>, n_tokens, 128, 0, stream, (const float*)q, ldq, (const float*)kv,
-                              ldkv, norm_w, eps, freq, n_pairs, mag, tok_pos, tok_seq, block_table, table_width,
-                              (float*)pages, page_size, (float*)q_cat, H, dim, rot, rank));
+                              ldkv, norm_w, eps, freq, n_pairs, interleaved, mag, tok_pos, tok_seq, block_table, table_width,
+                              (float*)pages, page_size, (float*)q_cat, H, dim, rot, rank, (const float*)ql, ldql, q_rank, q_norm_w, (float*)ql_out));
   else
     RL_REFUSE(4, "latent_prep: unknown dtype %d", dtype);
   return 0;

@@ -319,9 +319,13 @@ def attn_decode(
     n_splits: int, scratch: torch.Tensor, window: int = 0, scale: Optional[float] = None,
     out: Optional[torch.Tensor] = None, impl: str = "auto", fuse: int = 0,
     inv_freq: Optional[torch.Tensor] = None, rotary_dim: int = 0, interleaved: bool = False,
-    counters: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0,
+    counters: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0, pair=None,
 ) -> torch.Tensor:
     """One query token per sequence over keys 0..seq_len-1, the key range cut into `n_splits`.
+
+    pair (the "tma" kernel only): None, or (lambda, eps, factor): query heads 2h and 2h + 1 are two maps, the two halves of row h's
+    head_dim numbers (q's rows hold H / 2 such rows, k and v follow them with fuse = 2) against the same halves of the keys, and the
+    result [S, H / 2 head_dim] is o / sqrt(mean(o^2) + eps) * factor per head with o = a_2h - lambda a_(2h+1).
 
     sink: None, or float32 [H]: exp(sink_h) joins the softmax's denominator of head h and nothing else.
     chunk, softcap (the "tma" kernel only): 0, or the size of the chunks of positions outside of which the query sees nothing,
@@ -352,7 +356,9 @@ def attn_decode(
         _cuda(q, "attn_decode q", contiguous=False)
         qs, act = _rows(q, "attn_decode q"), q.dtype
         S, q_cols = q.shape
-    _need(q_cols >= num_heads * head_dim, "attn_decode: q rows too short")
+    maps = 1 if pair is None else 2
+    _need(pair is None or (num_heads % 2 == 0 and rotary_dim == 0 and counters is None), "attn_decode: two maps per head take neither a rotation nor counters")
+    _need(q_cols >= num_heads // maps * head_dim, "attn_decode: q rows too short")
     _need(q.data_ptr() % 16 == 0, "attn_decode: q is not 16-byte aligned")
     _check_pages(k_pages, v_pages, act, num_kv_heads, head_dim, "attn_decode")
     _cuda(block_table, "attn_decode block_table", torch.int32)
@@ -362,9 +368,9 @@ def attn_decode(
     need = attn_decode_scratch_floats(S, num_heads, head_dim, n_splits)
     _need(scratch.numel() >= need, f"attn_decode: scratch holds {scratch.numel()} floats, {need} needed")
     if out is None:
-        out = torch.empty((S, num_heads * head_dim), dtype=act, device=q.device)
+        out = torch.empty((S, num_heads // maps * head_dim), dtype=act, device=q.device)
     _cuda(out, "attn_decode out", act, contiguous=False)
-    _need(_rows(out, "attn_decode out") >= num_heads * head_dim and tuple(out.shape) == (S, num_heads * head_dim), "attn_decode: out must be [S, H head_dim] rows")
+    _need(_rows(out, "attn_decode out") >= out.shape[1] and tuple(out.shape) == (S, num_heads // maps * head_dim), "attn_decode: out must be [S, H head_dim] rows")
     if scale is None:
         scale = 1.0 / math.sqrt(head_dim)
     n_o = S * num_heads * n_splits * head_dim
@@ -380,7 +386,7 @@ def attn_decode(
             _cuda(inv_freq, "attn_decode inv_freq", torch.float32)
             _need(inv_freq.numel() >= rotary_dim // 2, "attn_decode: too few angles for the rotary size")
         if fuse == 2:
-            _need(q_cols >= (num_heads + 2 * num_kv_heads) * head_dim, "attn_decode: q rows hold no key and value")
+            _need(q_cols >= (num_heads // maps + 2 * num_kv_heads) * head_dim, "attn_decode: q rows hold no key and value")
     if counters is not None:
         _need(impl == "tma", "attn_decode: only the TMA kernel adds the splits up itself")
         _cuda(counters, "attn_decode counters", torch.int32)
@@ -399,11 +405,12 @@ def attn_decode(
             c_int(n_splits), _p(status), c_int(fuse), _p(inv_freq) if (fuse and rotary_dim) else c_void_p(0), c_int(rotary_dim if fuse else 0),
             c_int(1 if interleaved else 0), _p(counters) if counters is not None else c_void_p(0),
             _p(q_parts) if q_parts is not None else c_void_p(0), c_int(0 if q_parts is None else q_parts.shape[0]),
-            c_ll(0 if q_parts is None else q_parts.stride(0)), *_wt(), _p(sink), c_int(chunk), c_float(softcap), _stream(),
+            c_ll(0 if q_parts is None else q_parts.stride(0)), *_wt(), _p(sink), c_int(chunk), c_float(softcap), c_int(maps),
+            *(c_float(x) for x in (pair or (0.0, 0.0, 0.0))), _stream(),
         )
         _check(lib, rc, "attn_decode_tma", kernels=1 if counters is not None else 2)
         return out
-    _need(chunk == 0 and softcap == 0.0, "attn_decode: only the TMA kernel takes chunks and capped scores")
+    _need(chunk == 0 and softcap == 0.0 and pair is None, "attn_decode: only the TMA kernel takes chunks, capped scores and two maps per head")
     lib = build.load("attention_decode")
     rc = lib.rl_attn_decode_sink(
         _p(q), c_int(_dt(q, "attn_decode")), c_int(qs), _p(k_pages), _p(v_pages), _p(block_table),
@@ -454,16 +461,18 @@ FLASH_TC_HEAD_DIMS = (64, 128)  # head sizes the tcgen05 prompt attention is bui
 def flash_prefill_tc(
     q: torch.Tensor, k_pages, v_pages, block_table, seq_start, seq_pos0, max_q_len: int, num_heads: int,
     num_kv_heads: int, head_dim: int, window: int = 0, scale: Optional[float] = None,
-    out: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0,
+    out: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0, maps: int = 1,
 ) -> torch.Tensor:
     """`flash_prefill` on the tcgen05 tensor cores (TMA-fed, S and P V in tensor memory); head sizes 64 and 128.
     chunk: 0, or the size of the chunks of positions (counted from 0) outside of which a query sees nothing; softcap: 0, or the
-    cap c of s <- c tanh(s / c) on the scaled scores."""
+    cap c of s <- c tanh(s / c) on the scaled scores.
+    maps: 1, or 2: query heads 2h and 2h + 1 are the two halves of row h's head_dim numbers, against the same halves of the keys."""
+    _need(maps in (1, 2) and num_heads % maps == 0, f"flash_prefill_tc: {maps} maps in {num_heads} heads")
     _need(head_dim in FLASH_TC_HEAD_DIMS, f"flash_prefill_tc: head size {head_dim}, this kernel is built for {FLASH_TC_HEAD_DIMS}")
     _cuda(q, "flash_prefill_tc q", torch.bfloat16, contiguous=False)
     qs = _rows(q, "flash_prefill_tc q")
     T = q.shape[0]
-    _need(q.shape[1] >= num_heads * head_dim, "flash_prefill_tc: q rows too short")
+    _need(q.shape[1] >= num_heads // maps * head_dim, "flash_prefill_tc: q rows too short")
     _check_pages(k_pages, v_pages, torch.bfloat16, num_kv_heads, head_dim, "flash_prefill_tc")
     _need(k_pages.shape[0] == v_pages.shape[0], "flash_prefill_tc: k and v have different page counts")
     _cuda(block_table, "flash_prefill_tc block_table", torch.int32)
@@ -484,7 +493,7 @@ def flash_prefill_tc(
         _p(q), c_int(qs), c_int(T), _p(k_pages), _p(v_pages), c_int(k_pages.shape[0]), _p(block_table),
         c_int(block_table.shape[1]), _p(seq_start), _p(seq_pos0), _p(out), c_int(out.stride(0)), c_int(S), c_int(max_q_len),
         c_int(num_heads), c_int(num_kv_heads), c_int(head_dim), c_int(PAGE_SIZE), c_int(window), c_float(scale), _p(status), *_wt(), _p(sink),
-        c_int(chunk), c_float(softcap), _stream(),
+        c_int(chunk), c_float(softcap), c_int(maps), _stream(),
     )
     _check(lib, rc, "flash_prefill_tc")
     return out
@@ -955,6 +964,66 @@ def normed_add_rmsnorm(
     return out
 
 
+def gated_add_rmsnorm(
+    x: torch.Tensor, delta: Optional[torch.Tensor], gate, weight: Optional[torch.Tensor], eps: float, groups: int, act_dtype: torch.dtype,
+    rows: Optional[torch.Tensor] = None, write_x: bool = True,
+) -> Optional[torch.Tensor]:
+    """x (float32 [T, d]) += (sum of delta parts) * logistic(z + bias) with gate = (z [T, d] rows of `act_dtype`, bias float32 [d]),
+    or without the factor (gate None); returns x / rms * weight in `act_dtype`, the root mean square taken in each of `groups`
+    equal consecutive parts of a row on its own (None without a weight).  delta: None, [T, d] or [parts, T, d], in `act_dtype` or float32."""
+    _cuda(x, "gated_add_rmsnorm x", torch.float32)
+    _need(x.dim() == 2, "gated_add_rmsnorm: x must be [T, d]")
+    T, d = x.shape
+    _need(groups >= 1 and d % groups == 0, f"gated_add_rmsnorm: {groups} groups do not divide a row of {d}")
+    n_parts, part_stride, delta_dt = 0, 0, _DT[act_dtype]
+    if delta is not None:
+        _cuda(delta, "gated_add_rmsnorm delta")
+        _need(delta.dtype in (act_dtype, torch.float32), f"gated_add_rmsnorm: delta is {delta.dtype} in a run of {act_dtype}")
+        delta_dt = _DT[delta.dtype]
+        _need(tuple(delta.shape[-2:]) == (T, d) and delta.dim() in (2, 3), f"gated_add_rmsnorm: delta {tuple(delta.shape)} does not match x {(T, d)}")
+        n_parts, part_stride = (1, 0) if delta.dim() == 2 else (delta.shape[0], T * d)
+    z = bias = None
+    zs = 0
+    if gate is not None:
+        z, bias = gate
+        _need(delta is not None, "gated_add_rmsnorm: a gate but nothing to gate")
+        _cuda(z, "gated_add_rmsnorm gate", act_dtype, contiguous=False)
+        zs = _rows(z, "gated_add_rmsnorm gate")
+        _need(tuple(z.shape) == (T, d), f"gated_add_rmsnorm: gate {tuple(z.shape)} does not match x {(T, d)}")
+        _cuda(bias, "gated_add_rmsnorm bias", torch.float32)
+        _need(tuple(bias.shape) == (d,), "gated_add_rmsnorm: bias does not match d")
+    n_rows = T if rows is None else rows.numel()
+    out, w_dt = None, _F32
+    if weight is not None:
+        _cuda(weight, "gated_add_rmsnorm weight")
+        _need(tuple(weight.shape) == (d,), "gated_add_rmsnorm: weight does not match d")
+        w_dt = _dt(weight, "gated_add_rmsnorm weight")
+        out = torch.empty((n_rows, d), dtype=act_dtype, device=x.device)
+    else:
+        _need(delta is not None, "gated_add_rmsnorm: neither a delta nor a weight, nothing to do")
+    if rows is not None:
+        _cuda(rows, "gated_add_rmsnorm rows", torch.int32)
+    if n_rows == 0:
+        return out
+    lib = build.load("elementwise")
+    rc = lib.rl_gated_add_rmsnorm(
+        _p(x), _p(delta), c_int(delta_dt), c_int(n_parts), c_ll(part_stride), _p(z), c_int(zs), _p(bias), _p(weight), c_int(w_dt), _p(out),
+        c_int(_DT[act_dtype]), _p(rows), c_int(n_rows), c_int(d), c_int(groups), c_float(eps), c_int(1 if write_x else 0), _stream(),
+    )
+    _check(lib, rc, "gated_add_rmsnorm")
+    return out
+
+
+def scale_softcap(y: torch.Tensor, scale: float, cap: float = 0.0) -> torch.Tensor:
+    """y <- y * scale, then y <- cap tanh(y / cap) if cap > 0; in place, float32 (dense)."""
+    _cuda(y, "scale_softcap y", torch.float32)
+    if y.numel():
+        lib = build.load("elementwise")
+        rc = lib.rl_scale_softcap(_p(y), c_ll(y.numel()), c_float(scale), c_float(cap), _stream())
+        _check(lib, rc, "scale_softcap")
+    return y
+
+
 def gated_glu(gate_up: torch.Tensor, act) -> torch.Tensor:
     """h[t, i] = act(gate_up[t, i], gate_up[t, ff + i]) for the activations of a gate/up product (None: silu(gate) * up,
     (alpha, limit): the clamped form, "gelu_tanh": gelu(gate) * up), as a pass of its own behind a plain product."""
@@ -976,28 +1045,35 @@ def clamped_glu(gate_up: torch.Tensor, alpha: float, limit: float) -> torch.Tens
 
 # ------------------------------------------------------------------ latent attention
 def latent_prep(
-    q: torch.Tensor, kv: Optional[torch.Tensor], norm_w: Optional[torch.Tensor], eps: float, freq: Optional[torch.Tensor], n_pairs: int,
+    q: Optional[torch.Tensor], kv: Optional[torch.Tensor], norm_w: Optional[torch.Tensor], eps: float, freq: Optional[torch.Tensor], n_pairs: int,
     magnitude: float, tok_pos: torch.Tensor, tok_seq: torch.Tensor, block_table: Optional[torch.Tensor], pages: Optional[torch.Tensor],
-    q_cat: torch.Tensor, num_heads: int, dim: int, rot: int, rank: int,
-) -> None:
+    q_cat: Optional[torch.Tensor], num_heads: int, dim: int, rot: int, rank: int, interleaved: bool = True,
+    q_latent: Optional[torch.Tensor] = None, q_norm: Optional[torch.Tensor] = None,
+) -> Optional[torch.Tensor]:
     """Per token: kv's first `rank` values RMS-normed (weight norm_w) and its last `rot` values rotated go into the token's
     place in `pages` [pages, 1, PAGE_SIZE, rank + rot] (kv None: nothing is stored); the rotated part of every head of
-    q [T, >= H (dim + rot)] is rotated into q_cat[T, H, rank:]."""
-    _cuda(q, "latent_prep q", contiguous=False)
-    ldq = _rows(q, "latent_prep q")
-    T = q.shape[0]
-    _need(q.shape[1] >= num_heads * (dim + rot), "latent_prep: q rows too short")
-    _cuda(q_cat, "latent_prep q_cat", q.dtype)
-    _need(tuple(q_cat.shape) == (T, num_heads, rank + rot), "latent_prep: q_cat has the wrong shape")
+    q [T, >= H (dim + rot)] is rotated into q_cat[T, H, rank:] (q None: left out); the rows q_latent [T, q_rank] are RMS-normed
+    (weight q_norm float32 [q_rank], the same eps) and returned (q_latent None: nothing is returned).
+    interleaved: whether a rotated pair is (2i, 2i + 1) or (i, i + n_pairs)."""
+    some = q if q is not None else (kv if kv is not None else q_latent)
+    _need(some is not None, "latent_prep: nothing to do")
+    T, dt = some.shape[0], some.dtype
+    ldq = 0
+    if q is not None:
+        _cuda(q, "latent_prep q", contiguous=False)
+        ldq = _rows(q, "latent_prep q")
+        _need(q.shape[1] >= num_heads * (dim + rot), "latent_prep: q rows too short")
+        _cuda(q_cat, "latent_prep q_cat", dt)
+        _need(tuple(q_cat.shape) == (T, num_heads, rank + rot), "latent_prep: q_cat has the wrong shape")
     _cuda(tok_pos, "latent_prep tok_pos", torch.int32)
     _cuda(tok_seq, "latent_prep tok_seq", torch.int32)
     _need(tok_pos.numel() == T and tok_seq.numel() == T, "latent_prep: one position and one sequence index per token")
     ldkv, width = 0, 0
     if kv is not None:
-        _cuda(kv, "latent_prep kv", q.dtype, contiguous=False)
+        _cuda(kv, "latent_prep kv", dt, contiguous=False)
         ldkv = _rows(kv, "latent_prep kv")
         _need(kv.shape[0] == T and kv.shape[1] >= rank + rot, "latent_prep: kv rows do not fit")
-        _cuda(pages, "latent_prep pages", q.dtype)
+        _cuda(pages, "latent_prep pages", dt)
         _need(pages.dim() == 4 and tuple(pages.shape[1:]) == (1, PAGE_SIZE, rank + rot), f"latent_prep: pages {tuple(pages.shape)}")
         _cuda(block_table, "latent_prep block_table", torch.int32)
         _need(block_table.dim() == 2, "latent_prep: block_table must be [S, width]")
@@ -1007,14 +1083,22 @@ def latent_prep(
     if n_pairs:
         _cuda(freq, "latent_prep freq", torch.float32)
         _need(freq.numel() >= n_pairs, "latent_prep: too few angles")
+    ql_out, ldql, q_rank = None, 0, 0
+    if q_latent is not None:
+        _cuda(q_latent, "latent_prep q_latent", dt, contiguous=False)
+        ldql, q_rank = _rows(q_latent, "latent_prep q_latent"), q_latent.shape[1]
+        _cuda(q_norm, "latent_prep q_norm", torch.float32)
+        _need(q_latent.shape[0] == T and q_norm.numel() == q_rank, "latent_prep: the query latent's rows or norm weight do not fit")
+        ql_out = torch.empty((T, q_rank), dtype=dt, device=q_latent.device)
     lib = build.load("latent_attention")
     rc = lib.rl_latent_prep(
-        _p(q), c_int(ldq), _p(kv), c_int(ldkv), c_int(_dt(q, "latent_prep")), _p(norm_w), c_float(eps), _p(freq), c_int(n_pairs),
-        c_float(magnitude), _p(tok_pos), _p(tok_seq), _p(block_table) if kv is not None else c_void_p(0), c_int(width),
-        _p(pages) if kv is not None else c_void_p(0), c_int(PAGE_SIZE), _p(q_cat), c_int(T), c_int(num_heads), c_int(dim), c_int(rot),
-        c_int(rank), _stream(),
+        _p(q), c_int(ldq), _p(kv), c_int(ldkv), c_int(_dt(some, "latent_prep")), _p(norm_w), c_float(eps), _p(freq), c_int(n_pairs),
+        c_int(1 if interleaved else 0), c_float(magnitude), _p(tok_pos), _p(tok_seq), _p(block_table) if kv is not None else c_void_p(0), c_int(width),
+        _p(pages) if kv is not None else c_void_p(0), c_int(PAGE_SIZE), _p(q_cat) if q is not None else c_void_p(0), c_int(T), c_int(num_heads),
+        c_int(dim), c_int(rot), c_int(rank), _p(q_latent), c_int(ldql), c_int(q_rank), _p(q_norm), _p(ql_out), _stream(),
     )
     _check(lib, rc, "latent_prep")
+    return ql_out
 
 
 def head_linear(
@@ -1346,8 +1430,12 @@ def attn_ext(
     q: torch.Tensor, k_pages, v_pages, block_table, tok_seq, tok_pos, num_heads: int, num_kv_heads: int, kdim: int, vdim: int,
     scale: float, window: int = 0, sink: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None,
     gate: Optional[torch.Tensor] = None, out_scale: float = 1.0, out: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0,
+    maps: int = 1,
 ) -> torch.Tensor:
     """Attention of each token over its sequence's cached keys, both element types, prompts and decoding.
+
+    maps: 1, or 2: query heads 2h and 2h + 1 are the two halves of row h's kdim numbers, against the same halves of the keys (the
+    values are whole; `map_combine` makes one head of the two results).
 
     window: 0, or how many of the last positions a query sees.  chunk: 0, or the size of the chunks (counted from position 0)
     outside of which a query sees nothing.  softcap: 0, or the cap c of s <- c tanh(s / c) on the scaled scores.
@@ -1358,7 +1446,8 @@ def attn_ext(
     _cuda(q, "attn_ext q", contiguous=False)
     qs = _rows(q, "attn_ext q")
     T = q.shape[0]
-    _need(q.shape[1] >= num_heads * kdim, "attn_ext: q rows too short")
+    _need(maps in (1, 2) and num_heads % maps == 0 and kdim % maps == 0, f"attn_ext: {maps} maps in {num_heads} heads of {kdim}")
+    _need(q.shape[1] >= num_heads // maps * kdim, "attn_ext: q rows too short")
     _check_kv_pages(k_pages, v_pages, q.dtype, num_kv_heads, kdim, vdim, "attn_ext")
     _cuda(block_table, "attn_ext block_table", torch.int32)
     _cuda(tok_seq, "attn_ext tok_seq", torch.int32)
@@ -1383,9 +1472,26 @@ def attn_ext(
     rc = lib.rl_attn_ext(
         _p(q), c_int(_dt(q, "attn_ext")), c_int(qs), _p(k_pages), _p(v_pages), _p(block_table), c_int(block_table.shape[1]), _p(tok_seq),
         _p(tok_pos), _p(sink), _p(mix), _p(gate), c_int(gs), c_float(out_scale), _p(out), c_int(out.stride(0)), c_int(T), c_int(num_heads),
-        c_int(num_kv_heads), c_int(kdim), c_int(vdim), c_int(PAGE_SIZE), c_int(window), c_float(scale), c_int(chunk), c_float(softcap), _stream(),
+        c_int(num_kv_heads), c_int(kdim), c_int(vdim), c_int(PAGE_SIZE), c_int(window), c_float(scale), c_int(chunk), c_float(softcap), c_int(maps), _stream(),
     )
     _check(lib, rc, "attn_ext")
+    return out
+
+
+def map_combine(a: torch.Tensor, num_heads: int, vdim: int, lam: float, eps: float, factor: float, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """a [T, >= 2 H vdim] rows, the results of two maps per head side by side -> [T, H vdim]: per head o = a_2h - lam a_(2h+1),
+    o / sqrt(mean(o^2) + eps) * factor; 32-bit arithmetic, both element types."""
+    _cuda(a, "map_combine a", contiguous=False)
+    T = a.shape[0]
+    _need(a.shape[1] >= 2 * num_heads * vdim, "map_combine: rows too short")
+    if out is None:
+        out = torch.empty((T, num_heads * vdim), dtype=a.dtype, device=a.device)
+    _cuda(out, "map_combine out", a.dtype, contiguous=False)
+    _need(tuple(out.shape) == (T, num_heads * vdim), "map_combine: out must be [T, H vdim]")
+    lib = build.load("attention_ext")
+    rc = lib.rl_map_combine(_p(a), c_int(_dt(a, "map_combine")), c_int(_rows(a, "map_combine a")), c_float(lam), c_float(eps), c_float(factor), _p(out),
+                            c_int(_rows(out, "map_combine out")), c_int(T), c_int(num_heads), c_int(vdim), _stream())
+    _check(lib, rc, "map_combine")
     return out
 
 
@@ -1671,13 +1777,18 @@ def mlstm_gates(
 def gated_attn(
     q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_decay: torch.Tensor, in_scale: Optional[torch.Tensor], state: torch.Tensor,
     slot_ids: torch.Tensor, seq_start: torch.Tensor, num_heads: int, dim: int, vdim: int, q_scale: float = 1.0, ext: bool = False,
+    qk_heads: int = 0,
 ) -> torch.Tensor:
     """S_t = diag(a_t) S_(t-1) + b_t k_t v_t^T, o_t = S_t^T (q_scale q_t) through the sequences' states, token by token.
+
+    qk_heads: 0 (as many as `num_heads`), or how many heads q and k have ([T, qk_heads dim]); head h reads number h // (H / qk_heads).
 
     q, k: [T, H dim], v: [T, H vdim], views of one projection's rows.  log_decay: float32 [T, H dim] (a per key channel) or [T, H]
     (a per head), a = exp(log_decay).  in_scale: float32 [T, H] (b) or None (1).  ext: the state has one more column, fed with
     v = 1, and so has the result.  state: float32 [slots, H, dim, vdim (+1)].  Returns float32 [T, H (vdim (+1))]."""
-    for name, t, n in (("q", q, num_heads * dim), ("k", k, num_heads * dim), ("v", v, num_heads * vdim)):
+    qk_heads = qk_heads or num_heads
+    _need(num_heads % qk_heads == 0, f"gated_attn: {num_heads} heads are not a multiple of {qk_heads} q/k heads")
+    for name, t, n in (("q", q, qk_heads * dim), ("k", k, qk_heads * dim), ("v", v, num_heads * vdim)):
         _cuda(t, f"gated_attn {name}", q.dtype, contiguous=False)
         _need(_rows(t, f"gated_attn {name}") == q.stride(0) and t.shape[1] == n and t.shape[0] == q.shape[0], f"gated_attn: {name} has the wrong shape or stride")
     T = q.shape[0]
@@ -1698,8 +1809,8 @@ def gated_attn(
     lib = build.load("gated_recurrent")
     rc = lib.rl_gated_attn(
         _p(q), _p(k), _p(v), c_int(_dt(q, "gated_attn")), c_int(q.stride(0)), _p(log_decay), c_int(1 if per_channel else 0), _p(in_scale),
-        c_float(q_scale), _p(state), _p(slot_ids), _p(seq_start), _p(out), c_int(out.stride(0)), c_int(S), c_int(num_heads), c_int(dim),
-        c_int(vdim), c_int(1 if ext else 0), _stream(),
+        c_float(q_scale), _p(state), _p(slot_ids), _p(seq_start), _p(out), c_int(out.stride(0)), c_int(S), c_int(num_heads), c_int(qk_heads),
+        c_int(dim), c_int(vdim), c_int(1 if ext else 0), _stream(),
     )
     _check(lib, rc, "gated_attn")
     return out
@@ -1722,11 +1833,13 @@ def gated_attn_chunked_scratch_floats(n_seqs: int, max_q_len: int, num_heads: in
 def gated_attn_chunked(
     q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_decay: torch.Tensor, in_scale: Optional[torch.Tensor], state: torch.Tensor,
     slot_ids: torch.Tensor, seq_start: torch.Tensor, num_heads: int, dim: int, vdim: int, max_q_len: int, scratch: torch.Tensor,
-    q_scale: float = 1.0, ext: bool = False,
+    q_scale: float = 1.0, ext: bool = False, qk_heads: int = 0,
 ) -> torch.Tensor:
     """`gated_attn` chunk by chunk (64 tokens, all chunks side by side, 32-bit arithmetic): equal within rounding, for prompts.
     max_q_len: the most tokens a sequence of the step brings; scratch: float32, at least `gated_attn_chunked_scratch_floats(...)`."""
-    for name, t, n in (("q", q, num_heads * dim), ("k", k, num_heads * dim), ("v", v, num_heads * vdim)):
+    qk_heads = qk_heads or num_heads
+    _need(num_heads % qk_heads == 0, f"gated_attn_chunked: {num_heads} heads are not a multiple of {qk_heads} q/k heads")
+    for name, t, n in (("q", q, qk_heads * dim), ("k", k, qk_heads * dim), ("v", v, num_heads * vdim)):
         _cuda(t, f"gated_attn_chunked {name}", q.dtype, contiguous=False)
         _need(_rows(t, f"gated_attn_chunked {name}") == q.stride(0) and t.shape[1] == n and t.shape[0] == q.shape[0], f"gated_attn_chunked: {name} has the wrong shape or stride")
     T = q.shape[0]
@@ -1751,7 +1864,7 @@ def gated_attn_chunked(
     rc = lib.rl_gated_attn_chunked(
         _p(q), _p(k), _p(v), c_int(_dt(q, "gated_attn_chunked")), c_int(q.stride(0)), _p(log_decay), c_int(1 if per_channel else 0), _p(in_scale),
         c_float(q_scale), _p(state), _p(slot_ids), _p(seq_start), _p(scratch), _p(out), c_int(out.stride(0)), c_int(S), c_int(max_q_len),
-        c_int(num_heads), c_int(dim), c_int(vdim), c_int(1 if ext else 0), _stream(),
+        c_int(num_heads), c_int(qk_heads), c_int(dim), c_int(vdim), c_int(1 if ext else 0), _stream(),
     )
     _check(lib, rc, "gated_attn_chunked", kernels=3)
     return out
@@ -1808,9 +1921,11 @@ DELTA_RULE_MAX_DIM = 256
 
 def short_conv(
     x: torch.Tensor, w: torch.Tensor, state: Optional[torch.Tensor], slot_ids: torch.Tensor, seq_start: torch.Tensor, tok_seq: torch.Tensor,
-    silu: bool = True,
+    silu: bool = True, bias: Optional[torch.Tensor] = None, single: bool = False,
 ) -> torch.Tensor:
-    """y[t, c] = act(sum_i w[i, c] x[t - taps + 1 + i, c]) over each sequence's tokens, a causal convolution over time per channel.
+    """y[t, c] = act(bias[c] + sum_i w[i, c] x[t - taps + 1 + i, c]) over each sequence's tokens, a causal convolution over time per channel.
+
+    bias: float32 [C] or None.  single: every sequence brings exactly one token (one kernel instead of two).
 
     x: [T, C] rows (a view of a projection's rows is taken as it is).  w: float32 [taps, C] (tap i of every channel side by side,
     so that neighbouring channels read neighbouring weights), the last row the current token's.
@@ -1831,13 +1946,17 @@ def short_conv(
     if taps > 1:
         _cuda(state, "short_conv state", torch.float32)
         _need(state.dim() == 3 and tuple(state.shape[1:]) == (taps - 1, C), f"short_conv: state {tuple(state.shape)} is not [slots, {taps - 1}, {C}]")
+    if bias is not None:
+        _cuda(bias, "short_conv bias", torch.float32)
+        _need(bias.numel() == C, "short_conv: one bias per channel")
+    _need(not single or T == S, f"short_conv: {T} tokens of {S} sequences are not one each")
     out = torch.empty((T, C), dtype=x.dtype, device=x.device)
     lib = build.load("delta_rule")
     rc = lib.rl_short_conv(
-        _p(x), c_int(_dt(x, "short_conv")), c_int(xs), _p(w), _p(state if taps > 1 else None), _p(slot_ids), _p(seq_start), _p(tok_seq), _p(out),
-        c_int(out.stride(0)), c_int(T), c_int(S), c_int(C), c_int(taps), c_int(1 if silu else 0), _stream(),
+        _p(x), c_int(_dt(x, "short_conv")), c_int(xs), _p(w), _p(bias), _p(state if taps > 1 else None), _p(slot_ids), _p(seq_start), _p(tok_seq), _p(out),
+        c_int(out.stride(0)), c_int(T), c_int(S), c_int(C), c_int(taps), c_int(1 if silu else 0), c_int(1 if single else 0), _stream(),
     )
-    _check(lib, rc, "short_conv", kernels=2 if taps > 1 else 1)
+    _check(lib, rc, "short_conv", kernels=2 if taps > 1 and not single else 1)
     return out
 
 
@@ -1899,6 +2018,100 @@ def delta_rule(
     return out
 
 
+# ------------------------------------------------------------------ state-space layer (csrc/state_space.cu)
+def ssm_gates(raw: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor):
+    """raw [T, H] rows of the run's type -> (log_a = -exp(a_log) dt, dt = softplus(raw + dt_bias)), float32 [T, H] each."""
+    _cuda(raw, "ssm_gates raw", contiguous=False)
+    T, H = raw.shape
+    for name, t in (("a_log", a_log), ("dt_bias", dt_bias)):
+        _cuda(t, f"ssm_gates {name}", torch.float32)
+        _need(t.numel() == H, f"ssm_gates: one {name} per head")
+    log_a, dt = (torch.empty((T, H), dtype=torch.float32, device=raw.device) for _ in range(2))
+    lib = build.load("state_space")
+    rc = lib.rl_ssm_gates(_p(raw), c_int(_dt(raw, "ssm_gates")), c_int(_rows(raw, "ssm_gates raw")), _p(a_log), _p(dt_bias), _p(log_a), _p(dt), c_int(T), c_int(H), _stream())
+    _check(lib, rc, "ssm_gates")
+    return log_a, dt
+
+
+def ssm_gate_norm(
+    y: torch.Tensor, x: torch.Tensor, skip: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, eps: float, groups: int, act_dtype: torch.dtype,
+    out_scale: float = 1.0, out: Optional[torch.Tensor] = None,
+) -> torch.Tensor:
+    """v = (y + skip[head] x) * silu(z) over rows of n numbers; each of `groups` equal parts of a row divided by its own root mean
+    square (eps inside the root), times weight and `out_scale`.  y: float32 [T, n]; x, z: [T, n] rows of `act_dtype`; skip: float32 [H]."""
+    _cuda(y, "ssm_gate_norm y", torch.float32, contiguous=False)
+    T, n = y.shape
+    for name, t in (("x", x), ("z", z)):
+        _cuda(t, f"ssm_gate_norm {name}", act_dtype, contiguous=False)
+        _need(tuple(t.shape) == (T, n), f"ssm_gate_norm: {name} {tuple(t.shape)} does not match y {(T, n)}")
+    _cuda(skip, "ssm_gate_norm skip", torch.float32)
+    _cuda(weight, "ssm_gate_norm weight", torch.float32)
+    H = skip.numel()
+    _need(n % H == 0 and n % groups == 0 and weight.numel() == n, f"ssm_gate_norm: {H} heads, {groups} parts and {weight.numel()} weights for a row of {n}")
+    if out is None:
+        out = torch.empty((T, n), dtype=act_dtype, device=y.device)
+    _cuda(out, "ssm_gate_norm out", act_dtype, contiguous=False)
+    _need(tuple(out.shape) == (T, n), "ssm_gate_norm: out must be [T, n]")
+    lib = build.load("state_space")
+    rc = lib.rl_ssm_gate_norm(
+        _p(y), c_int(_rows(y, "ssm_gate_norm y")), _p(x), c_int(_rows(x, "ssm_gate_norm x")), _p(skip), c_int(n // H), _p(z), c_int(_rows(z, "ssm_gate_norm z")),
+        _p(weight), c_float(eps), c_int(groups), _p(out), c_int(_rows(out, "ssm_gate_norm out")), c_int(_DT[act_dtype]), c_int(T), c_int(n),
+        c_float(out_scale), _stream(),
+    )
+    _check(lib, rc, "ssm_gate_norm")
+    return out
+
+
+SCALAR_DECAY_CHUNK = 64  # tokens per chunk
+SCALAR_DECAY_MAX_DIM = 128
+
+
+def scalar_decay_chunked_takes(dim: int, vdim: int) -> bool:
+    """Whether the tensor-core form of a recurrence with one decay per head and token is built for these sizes (bfloat16 only)."""
+    return 0 < dim <= SCALAR_DECAY_MAX_DIM and 0 < vdim <= SCALAR_DECAY_MAX_DIM
+
+
+def scalar_decay_chunked_scratch_floats(n_seqs: int, max_q_len: int, num_heads: int, dim: int, vdim: int) -> int:
+    return n_seqs * num_heads * ((max_q_len + SCALAR_DECAY_CHUNK - 1) // SCALAR_DECAY_CHUNK) * (dim * vdim + 1)
+
+
+def scalar_decay_chunked(
+    q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_decay: torch.Tensor, in_scale: Optional[torch.Tensor], state: torch.Tensor,
+    slot_ids: torch.Tensor, seq_start: torch.Tensor, num_heads: int, dim: int, vdim: int, max_q_len: int, scratch: torch.Tensor, qk_heads: int = 0,
+) -> torch.Tensor:
+    """`gated_attn` with one decay per head (log_decay float32 [T, H]) chunk by chunk on the tensor cores, bfloat16 q, k, v, key and
+    value sizes up to 128: equal within rounding, for prompts.  max_q_len: the most tokens a sequence of the step brings; scratch:
+    float32, `scalar_decay_chunked_scratch_floats(...)` numbers.  Returns float32 [T, H vdim]."""
+    qk_heads = qk_heads or num_heads
+    _need(num_heads % qk_heads == 0, f"scalar_decay_chunked: {num_heads} heads are not a multiple of {qk_heads} q/k heads")
+    for name, t, n in (("q", q, qk_heads * dim), ("k", k, qk_heads * dim), ("v", v, num_heads * vdim)):
+        _cuda(t, f"scalar_decay_chunked {name}", torch.bfloat16, contiguous=False)
+        _need(_rows(t, f"scalar_decay_chunked {name}") == q.stride(0) and t.shape[1] == n and t.shape[0] == q.shape[0], f"scalar_decay_chunked: {name} has the wrong shape or stride")
+    T = q.shape[0]
+    _need(scalar_decay_chunked_takes(dim, vdim), f"scalar_decay_chunked: sizes {dim} x {vdim} are not built")
+    _cuda(log_decay, "scalar_decay_chunked log_decay", torch.float32)
+    _need(log_decay.numel() == T * num_heads, f"scalar_decay_chunked: log_decay {tuple(log_decay.shape)} is not [T, H]")
+    if in_scale is not None:
+        _cuda(in_scale, "scalar_decay_chunked in_scale", torch.float32)
+        _need(in_scale.numel() == T * num_heads, "scalar_decay_chunked: in_scale must be [T, H]")
+    _cuda(state, "scalar_decay_chunked state", torch.float32)
+    _need(state.dim() == 4 and tuple(state.shape[1:]) == (num_heads, dim, vdim), f"scalar_decay_chunked: state {tuple(state.shape)} is not [slots, {num_heads}, {dim}, {vdim}]")
+    _cuda(slot_ids, "scalar_decay_chunked slot_ids", torch.int32)
+    _cuda(seq_start, "scalar_decay_chunked seq_start", torch.int32)
+    S = slot_ids.numel()
+    _need(seq_start.numel() == S + 1, "scalar_decay_chunked: seq_start must hold one more entry than there are sequences")
+    _cuda(scratch, "scalar_decay_chunked scratch", torch.float32)
+    _need(max_q_len >= 1 and scratch.numel() >= scalar_decay_chunked_scratch_floats(S, max_q_len, num_heads, dim, vdim), "scalar_decay_chunked: scratch too small")
+    out = torch.empty((T, num_heads * vdim), dtype=torch.float32, device=q.device)
+    lib = build.load("state_space")
+    rc = lib.rl_scalar_decay_chunked(
+        _p(q), _p(k), _p(v), c_int(q.stride(0)), _p(log_decay), _p(in_scale), _p(state), _p(slot_ids), _p(seq_start), _p(scratch), _p(out),
+        c_int(out.stride(0)), c_int(S), c_int(max_q_len), c_int(num_heads), c_int(qk_heads), c_int(dim), c_int(vdim), _stream(),
+    )
+    _check(lib, rc, "scalar_decay_chunked", kernels=3)
+    return out
+
+
 ACT_RELU2 = 1  # relu(x)^2
 
 
@@ -1927,18 +2140,19 @@ def flash_mix_takes(kdim: int, vdim: int, parts: int) -> bool:
     return (3 * 64 + parts * 64) * (hd + 8) * 2 <= FLASH_MIX_SMEM_LIMIT
 
 
-def fold_queries(q: torch.Tensor, mix: torch.Tensor, num_heads: int, num_kv_heads: int, kdim: int) -> torch.Tensor:
+def fold_queries(q: torch.Tensor, mix: torch.Tensor, num_heads: int, num_kv_heads: int, kdim: int, maps: int = 1) -> torch.Tensor:
     """out[t, h, c, :] = sum over the heads g of kv head c of mix[h, g] * q[t, g, :] (32-bit sums, bfloat16 result): the queries
-    with which head h's mixed score is one product against the keys of all kv heads side by side."""
+    with which head h's mixed score is one product against the keys of all kv heads side by side.
+    maps: as in `attn_ext` (the half of a row that is not the head's reads zero)."""
     _cuda(q, "fold_queries q", torch.bfloat16, contiguous=False)
     qs = _rows(q, "fold_queries q")
-    _need(q.shape[1] >= num_heads * kdim, "fold_queries: q rows too short")
+    _need(q.shape[1] >= num_heads // maps * kdim, "fold_queries: q rows too short")
     _cuda(mix, "fold_queries mix", torch.float32)
     _need(tuple(mix.shape) == (num_heads, num_heads), "fold_queries: the mixing matrix must be [H, H]")
     T = q.shape[0]
     out = torch.empty((T, num_heads * num_kv_heads * kdim), dtype=torch.bfloat16, device=q.device)
     lib = build.load("attention_mix_mma")
-    rc = lib.rl_fold_queries(_p(q), c_int(qs), _p(mix), _p(out), c_int(T), c_int(num_heads), c_int(num_kv_heads), c_int(kdim), _stream())
+    rc = lib.rl_fold_queries(_p(q), c_int(qs), _p(mix), _p(out), c_int(T), c_int(num_heads), c_int(num_kv_heads), c_int(kdim), c_int(maps), _stream())
     _check(lib, rc, "fold_queries")
     return out
 
@@ -1946,17 +2160,19 @@ def fold_queries(q: torch.Tensor, mix: torch.Tensor, num_heads: int, num_kv_head
 def flash_mix(
     q: torch.Tensor, k_pages, v_pages, block_table, seq_start, seq_pos0, max_q_len: int, num_heads: int, num_kv_heads: int, kdim: int,
     vdim: int, scale: float, window: int = 0, sink: Optional[torch.Tensor] = None, folded: bool = False, gate: Optional[torch.Tensor] = None,
-    out_scale: float = 1.0, out: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0,
+    out_scale: float = 1.0, out: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0, maps: int = 1,
 ) -> torch.Tensor:
     """bfloat16 attention of a ragged batch over the paged cache on the tensor cores, keys of `kdim` and values of `vdim` numbers,
     with a window, chunks (a query sees the keys of its own chunk of positions only), capped scores (s <- c tanh(s / c)), a sink,
     a gate (out *= sigmoid(gate)) and a constant factor.  folded: q is what `fold_queries` made
-    ([T, H K kdim]: the heads' scores are mixed); else q holds [T, >= H kdim] rows."""
+    ([T, H K kdim]: the heads' scores are mixed); else q holds [T, >= H kdim] rows.  maps: as in `attn_ext` (not folded; kdim a
+    multiple of 16)."""
     _cuda(q, "flash_mix q", torch.bfloat16, contiguous=False)
     qs = _rows(q, "flash_mix q")
     T = q.shape[0]
     parts = num_kv_heads if folded else 1
-    _need(q.shape[1] >= num_heads * parts * kdim, "flash_mix: q rows too short")
+    _need(maps in (1, 2) and num_heads % maps == 0 and kdim % (8 * maps) == 0, f"flash_mix: {maps} maps in {num_heads} heads of {kdim}")
+    _need(q.shape[1] >= num_heads // maps * parts * kdim, "flash_mix: q rows too short")
     _need(flash_mix_takes(kdim, vdim, parts), f"flash_mix: sizes {kdim} / {vdim} with {parts} query parts are not built")
     _check_kv_pages(k_pages, v_pages, torch.bfloat16, num_kv_heads, kdim, vdim, "flash_mix")
     _cuda(block_table, "flash_mix block_table", torch.int32)
@@ -1979,7 +2195,7 @@ def flash_mix(
         _p(q), c_ll(qs), c_int(parts * kdim), c_int(parts), _p(k_pages), _p(v_pages), _p(block_table), c_int(block_table.shape[1]),
         _p(seq_start), _p(seq_pos0), _p(sink), _p(gate), c_int(gs), c_float(out_scale), _p(out), c_int(out.stride(0)), c_int(S),
         c_int(max_q_len), c_int(num_heads), c_int(num_kv_heads), c_int(kdim), c_int(vdim), c_int(PAGE_SIZE), c_int(window), c_float(scale),
-        c_int(chunk), c_float(softcap), _stream(),
+        c_int(chunk), c_float(softcap), c_int(maps), _stream(),
     )
     _check(lib, rc, "flash_mix")
     return out

@@ -31,7 +31,7 @@ class Model:
             # a layer may have no feed-forward at all
             ff = None if layer.feed_forward is None else FEED_FORWARDS.build(layer.feed_forward, runtime)
             norms = {name: NORMS.build(n, runtime) for name, n in layer.norms.items()}
-            self.blocks.append(BLOCKS.build(PartSpec(layer.block), runtime, mixer, ff, norms))
+            self.blocks.append(BLOCKS.build(PartSpec(layer.block, layer.block_params, layer.block_prefix), runtime, mixer, ff, norms))
         self.final_norm = NORMS.build(spec.final_norm, runtime)
         self.head = HEADS.build(spec.head, runtime)
         self.loaded = False
@@ -47,6 +47,7 @@ class Model:
 
         yield from walk(self.embedding)
         for b in self.blocks:
+            yield from walk(b)
             yield from walk(b.mixer)
             if b.feed_forward is not None:
                 yield from walk(b.feed_forward)

@@ -85,6 +85,7 @@ class Attention(Mixer):
     every size and both element types."""
 
     takes_out = True
+    maps = 1  # how many query heads of `_attend` share one row of `hd` query numbers (2: `DifferentialAttention`)
 
     def __init__(self, spec, runtime):
         super().__init__(spec, runtime)
@@ -130,7 +131,7 @@ class Attention(Mixer):
         # (the 32-bit attention kernel has none), and in bfloat16 a head size that moves in 16-byte pieces
         plain = self.vd == self.hd and not (self.has_mix or self.has_gate or self.has_bias) and self.out_scale == 1.0 and magnitude == 1.0
         plain = plain and not (self.zero_sink or self.qk_norm_eps is not None or self.softcap or self.chunk)
-        plain = plain and not (self.logistic or self.value_mix is not None)
+        plain = plain and not (self.logistic or self.value_mix is not None) and self.maps == 1
         if self.logistic and (self.has_sink or self.zero_sink):
             raise ConfigError("attention: logistic weights have no denominator for a sink to join")
         if self.value_mix is not None and self.has_bias:
@@ -257,7 +258,7 @@ class Attention(Mixer):
         if (bf and self.hd == self.vd and self.hd in ops.FLASH_TC_HEAD_DIMS and not self.has_mix and gate is None and self.out_scale == 1.0
                 and proj.stride(0) % 8 == 0 and proj.data_ptr() % 16 == 0):
             direct = out is not None and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0 and out.stride(1) == 1
-            if step.decode_only and self.hd in ops.ATTN_DECODE_TMA_HEAD_DIMS:
+            if step.decode_only and self.hd in ops.ATTN_DECODE_TMA_HEAD_DIMS and self.maps == 1:
                 keys = min(self.window, step.plan_kv_len) if self.window else step.plan_kv_len
                 keys = min(self.chunk, keys) if self.chunk else keys
                 n_splits = decode_splits(step.n_seqs, self.H, self.K, keys, self.hd)
@@ -271,21 +272,21 @@ class Attention(Mixer):
                 a = ops.flash_prefill_tc(
                     proj, cache.k_pages, cache.v_pages, cache.block_table, step.seq_start, step.seq_pos0, step.max_q_len, self.H, self.K,
                     self.hd, window=self.window, scale=self.scale, sink=self.sink, chunk=self.chunk, softcap=self.softcap,
-                    out=out if direct else None,
+                    out=out if direct else None, maps=self.maps,
                 )
             if out is not None and a is not out:
                 out.copy_(a)
                 a = out
             return a
         parts = self.K if self.has_mix else 1
-        if (bf and ops.flash_mix_takes(self.hd, self.vd, parts) and proj.stride(0) % 8 == 0
+        if (bf and ops.flash_mix_takes(self.hd, self.vd, parts) and self.hd % (8 * self.maps) == 0 and proj.stride(0) % 8 == 0 and proj.data_ptr() % 16 == 0
                 and (out is None or (out.stride(0) % 2 == 0 and out.data_ptr() % 4 == 0)) and (self.qd + self.kvd + self.vvd) % 2 == 0):
             if step.decode_only and ops.flash_mix_decode_takes(self.H, self.K, self.hd, self.vd):
                 # single tokens: all heads of a sequence are the rows of one block, which reads a key tile once for all of them;
                 # the key range is cut into parts of a page or more so that the blocks fill the GPU (a block is one or two warps: short chains matter more than few parts)
                 if self.fold_matrix is None:
                     self.fold_matrix = self.mix if self.has_mix else torch.eye(self.H, dtype=torch.float32, device=proj.device)
-                qf = ops.fold_queries(proj, self.fold_matrix, self.H, self.K, self.hd)
+                qf = ops.fold_queries(proj, self.fold_matrix, self.H, self.K, self.hd, maps=self.maps)
                 keys = min(self.window, step.plan_kv_len) if self.window else step.plan_kv_len
                 keys = min(self.chunk, keys) if self.chunk else keys
                 pages = (keys + ops.PAGE_SIZE - 1) // ops.PAGE_SIZE + 1
@@ -302,12 +303,12 @@ class Attention(Mixer):
             return ops.flash_mix(
                 q, cache.k_pages, cache.v_pages, cache.block_table, step.seq_start, step.seq_pos0, step.max_q_len, self.H, self.K,
                 self.hd, self.vd, self.scale, window=self.window, sink=self.sink, folded=self.has_mix, gate=gate, out_scale=self.out_scale,
-                out=out, chunk=self.chunk, softcap=self.softcap,
+                out=out, chunk=self.chunk, softcap=self.softcap, maps=self.maps,
             )
         return ops.attn_ext(
             proj, cache.k_pages, cache.v_pages, cache.block_table, step.tok_seq, step.tok_pos, self.H, self.K, self.hd, self.vd,
             self.scale, window=self.window, sink=self.sink, mix=self.mix, gate=gate, out_scale=self.out_scale, out=out, chunk=self.chunk,
-            softcap=self.softcap,
+            softcap=self.softcap, maps=self.maps,
         )
 
     def _attend_logistic(self, proj: torch.Tensor, gate, step, cache, out):
@@ -417,7 +418,7 @@ def chunked_attention_runner(proj, k_pages, v_pages, block_table, step, num_head
         step.plan_kv_len = int(step.seq_len.max())
     part = SimpleNamespace(
         rt=SimpleNamespace(dtype=proj.dtype, workspace=workspace or _Scratch()), H=num_heads, K=num_kv_heads, hd=kdim, vd=vdim, scale=scale,
-        window=window, chunk=chunk, softcap=softcap, sink=sink, mix=None, has_mix=False, out_scale=1.0, fold_matrix=None, logistic=False,
+        window=window, chunk=chunk, softcap=softcap, sink=sink, mix=None, has_mix=False, out_scale=1.0, fold_matrix=None, logistic=False, maps=1,
         qd=num_heads * kdim, kvd=num_kv_heads * kdim, vvd=num_kv_heads * vdim,
     )
     cache = SimpleNamespace(k_pages=k_pages, v_pages=v_pages, block_table=block_table)

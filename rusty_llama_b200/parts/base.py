@@ -187,33 +187,39 @@ class ResidualStream:
         # (weight, eps, bias) of an RMSNorm that what is pending goes through before it is added (a layer that
         # norms its sublayers' results); None: it is added as it is
         self.pending_norm = None
+        # (z [T, d], bias float32 [d]): what is pending is multiplied by the logistic function of z + bias before it is added
+        self.pending_gate = None
 
-    def add(self, delta: torch.Tensor, norm=None, bias: Optional[torch.Tensor] = None) -> None:
+    def add(self, delta: torch.Tensor, norm=None, bias: Optional[torch.Tensor] = None, gate=None) -> None:
         """norm: None, or (weight, eps): the stream receives rmsnorm(delta) * weight instead of delta.
+        gate: None, or (z, gate_bias): the stream receives delta * logistic(z + gate_bias), element by element.
         bias: None, or a float32 row [d] that belongs to every row of delta (the bias of the projection that made it); the
         kernel that norms delta adds it first, so it needs a norm."""
         if self.pending is not None:
             self.flush()
         if bias is not None and norm is None:
             raise ConfigError("a sublayer's result with a bias row can only be added through a norm of that result")
+        if gate is not None and norm is not None:
+            raise ConfigError("a sublayer's result goes through a norm of its own or through a gate, not both")
         self.pending = delta
         self.pending_norm = None if norm is None else (norm[0], norm[1], bias)
+        self.pending_gate = gate
 
-    def add_result(self, result, norm=None, bias: Optional[torch.Tensor] = None) -> None:
+    def add_result(self, result, norm=None, bias: Optional[torch.Tensor] = None, gate=None) -> None:
         """`add` for what a sublayer returned: a tensor, or `NormedTerms`, whose terms are added one after the other (each but the
         last by a pass of its own; the last stays pending for the next norm's kernel)."""
         if isinstance(result, NormedTerms):
-            if norm is not None or bias is not None:
-                raise ConfigError("a sublayer's result that is a sum of normed terms takes no further norm or bias row")
+            if norm is not None or bias is not None or gate is not None:
+                raise ConfigError("a sublayer's result that is a sum of normed terms takes no further norm, gate or bias row")
             for delta, term_norm in result:
                 self.add(delta, norm=term_norm)
         else:
-            self.add(result, norm=norm, bias=bias)
+            self.add(result, norm=norm, bias=bias, gate=gate)
 
     def take_pending(self):
-        """(delta, norm) of what is pending, which is the caller's to add from now on."""
-        out = (self.pending, self.pending_norm)
-        self.pending = self.pending_norm = None
+        """(delta, norm, gate) of what is pending, which is the caller's to add from now on."""
+        out = (self.pending, self.pending_norm, self.pending_gate)
+        self.pending = self.pending_norm = self.pending_gate = None
         return out
 
     def flush(self) -> None:
@@ -223,9 +229,11 @@ class ResidualStream:
             if self.pending_norm is not None:
                 ops.normed_add_rmsnorm(self.x, self.pending, self.pending_norm[0], self.pending_norm[1], None, 0.0, self.act_dtype,
                                        delta_bias=self.pending_norm[2])
+            elif self.pending_gate is not None:
+                ops.gated_add_rmsnorm(self.x, self.pending, self.pending_gate, None, 0.0, 1, self.act_dtype)
             else:
                 ops.add_rmsnorm(self.x, self.pending, None, 0.0, self.act_dtype)
-            self.pending = self.pending_norm = None
+            self.pending = self.pending_norm = self.pending_gate = None
 
 
 class Norm(Part):

@@ -7,9 +7,9 @@ import os
 import torch
 
 from ..kernels import ops
-from ..kernels.linear import STREAM_MAX_ROWS, linear_to_stream
+from ..kernels.linear import STREAM_MAX_ROWS, linear, linear_to_stream
 from ..errors import ConfigError
-from .base import BLOCKS, Block, ResidualStream
+from .base import BLOCKS, Block, ParamInfo, ResidualStream
 
 
 def _fold_enabled() -> bool:
@@ -118,3 +118,52 @@ class SharedNormBlock(Block):
         stream.add_result(self.mixer.forward(xn, step, cache, shared_cache), bias=self.mixer.output_bias())
         if self.feed_forward is not None:
             stream.add(self.feed_forward.forward(xn, step))
+
+
+@BLOCKS.register("gated_prenorm")
+class GatedPreNormBlock(Block):
+    """x += s(W_m h + b_m) * mixer(h), h = norm_m(x);  x += s(W_f h + b_f) * feed_forward(h), h = norm_f(x): every sublayer's result
+    is multiplied element by element by the logistic function s of a linear map of the sublayer's input.  norms: "mixer", and with a
+    feed-forward "feed_forward".
+
+    A result stays pending on the stream together with its gate's pre-activation; the kernel of the next norm applies bias and
+    logistic function, multiplies, adds and norms the sum, all in 32-bit and in one pass.
+
+    params: hidden_size, names (the gates' tensors after the block's prefix, keys mixer feed_forward; a bias is its name + ".b").
+    tensors: <prefix><name> [d, d], <prefix><name>.b [d]."""
+
+    def __init__(self, spec, runtime, mixer, feed_forward, norms):
+        super().__init__(spec, runtime, mixer, feed_forward, norms)
+        self.d = int(self._param("hidden_size"))
+        names = dict({"mixer": "gate_mixer", "feed_forward": "gate_feed_forward"}, **dict(spec.params.get("names", {})))
+        self.gate_names = {k: self.prefix + names[k] for k in (["mixer"] + (["feed_forward"] if feed_forward is not None else []))}
+        for k in self.gate_names:
+            if k not in self.norms:
+                raise ConfigError(f"gated_prenorm block: no norm '{k}'")
+        self.gates = {}
+
+    def param_infos(self):
+        infos = {}
+        for name in self.gate_names.values():
+            infos[name] = ParamInfo((self.d, self.d))
+            infos[name + ".b"] = ParamInfo((self.d,), "scalars", centre=0.0)
+        return infos
+
+    def load(self, tensors):
+        self.gates = {k: (tensors[name].contiguous(), tensors[name + ".b"].contiguous()) for k, name in self.gate_names.items()}
+
+    def _gate(self, which: str, h: torch.Tensor):
+        w, b = self.gates[which]
+        return linear(h, w), b
+
+    def forward(self, stream: ResidualStream, step, cache, shared_cache: bool = False) -> None:
+        h = self.norms["mixer"].forward(stream)
+        gate = self._gate("mixer", h)
+        if self.mixer.output_bias() is not None:
+            raise ConfigError("gated_prenorm block: a mixer with an output bias is not built")
+        stream.add_result(self.mixer.forward(h, step, cache, shared_cache), gate=gate)
+        if self.feed_forward is None:
+            return
+        h = self.norms["feed_forward"].forward(stream)
+        gate = self._gate("feed_forward", h)
+        stream.add(self.feed_forward.forward(h, step), gate=gate)

@@ -42,13 +42,16 @@ class LinearHead(Part):
     """logits = W xn in 32-bit (src/model.rs:1366); `tied_to` names the embedding
     tensor that serves as W when the model has no classifier of its own (src/model.rs:469-473).
 
-    params: vocab_size, hidden_size, tied_to (a tensor name or None), name (optional, as for the embedding)."""
+    params: vocab_size, hidden_size, tied_to (a tensor name or None), name (optional, as for the embedding), scale (optional,
+    default 1: a constant factor on the logits), softcap (optional, 0: the cap c of z <- c tanh(z / c) on the scaled logits)."""
 
     def __init__(self, spec, runtime):
         super().__init__(spec, runtime)
         self.vocab_size = int(self._param("vocab_size"))
         self.d = int(self._param("hidden_size"))
         self.tied_to = self._param("tied_to")
+        self.scale = float(spec.params.get("scale", 1.0))
+        self.softcap = float(spec.params.get("softcap", 0.0) or 0.0)
         self.weight: Optional[torch.Tensor] = None
 
     def weight_name(self) -> str:
@@ -61,4 +64,7 @@ class LinearHead(Part):
         self.weight = tensors[self.weight_name()]
 
     def forward(self, xn: torch.Tensor) -> torch.Tensor:
-        return linear(xn, self.weight, out_dtype=torch.float32)
+        logits = linear(xn, self.weight, out_dtype=torch.float32)
+        if self.scale != 1.0 or self.softcap:
+            ops.scale_softcap(logits, self.scale, self.softcap)
+        return logits

@@ -1,9 +1,11 @@
 """Mixers whose memory is a matrix per head that decays by gates computed from the current token: gated linear attention
 (a decay per key channel), the matrix memory of xLSTM (mLSTM: scalar input and forget gates per head, kept in range by a
-running maximum) and the gated delta rule (a decay per head, and a write that corrects what the state already holds for the key).
+running maximum), the state-space layer of Mamba-2 (a decay per head, keys and queries shared by groups of heads) and the gated
+delta rule (a decay per head, and a write that corrects what the state already holds for the key).
 
 All keep their state in 32-bit in the cache's state records, one record per sequence slot, zero when the sequence starts;
-the first two run on the same recurrence kernel (csrc/gated_recurrent.cu), the delta rule on its own (csrc/delta_rule.cu):
+the first three run on the same recurrence kernel (csrc/gated_recurrent.cu; for the state-space layer's prompts also
+csrc/state_space.cu), the delta rule on its own (csrc/delta_rule.cu):
 
     S_t = diag(a_t) S_(t-1) + b_t k_t v_t^T,   o_t = S_t^T q_t
 
@@ -307,9 +309,116 @@ class GatedDeltaRule(Mixer):
         memory, inputs = cache if self.taps > 1 else (cache, None)
         proj = linear(xn, self.w_in)
         C, vd, H = self.channels, self.vd, self.H
-        conv = ops.short_conv(proj[:, :C], self.w_conv, None if inputs is None else inputs.state, step.slot_ids, step.seq_start, step.tok_seq)
+        conv = ops.short_conv(proj[:, :C], self.w_conv, None if inputs is None else inputs.state, step.slot_ids, step.seq_start, step.tok_seq,
+                              single=step.decode_only)
         gate, ba = proj[:, C : C + vd], proj[:, C + vd : C + vd + 2 * H]
         qn, kn, kq, beta, decay = ops.delta_prep(conv[:, : 2 * self.qd], ba, self.a_log, self.dt_bias, self.G, H, self.dim, self.unit_eps, self.q_scale)
         o = ops.delta_rule(qn, kn, kq, conv[:, 2 * self.qd :], beta, decay, memory.state, step.slot_ids, step.seq_start, H, self.G, self.dim, self.vdim)
         a = ops.head_norm_gate(o, H, self.vdim, self.w_norm, self.eps, gate, ops.GATE_SILU, xn.dtype, out_scale=self.out_scale, out=out)
         return a, self.w_o
+
+
+@MIXERS.register("mamba2")
+class StateSpaceDuality(Mixer):
+    """The state-space layer of Mamba-2, per head with a state S [state, vdim]; head h reads the B and C of group h // (H / groups):
+
+        [z | x | B | C | dt] = W_in xn,   with [x | B | C] <- silu(conv([x | B | C]) + b_conv)         (inner = H vdim numbers of z and x)
+        dt <- softplus(dt + dt_bias),   a = exp(-exp(A_log) dt)                                         (one number per head each)
+        S_t = a_t S_(t-1) + dt_t B_t x_t^T,   y_t = S_t^T C_t + D x_t
+        result = W_o ( norm(y * silu(z)) * w_norm )                    (each of `norm_groups` equal parts of the row by its own rms)
+
+    conv is a causal convolution over time per channel with `taps` taps (zeros before a sequence's start); the last taps - 1
+    projected inputs of a sequence are a second record beside S.  Everything after the convolution's activation is 32-bit.
+
+    A prompt of a bfloat16 run goes chunk by chunk (`scalar_decay_chunked` on the tensor cores up to sizes of 128, else the FMA
+    kernels of `gated_attn_chunked`); single tokens, short portions and 32-bit runs go token by token (equal bits for every cut).
+
+    params: hidden_size, num_heads, vdim, state, groups, taps, norm_groups, eps (of the norm), out_scale (default 1),
+            names (optional: keys in conv conv_bias dt_bias a_log d norm o).
+    tensors: <prefix>in [2 inner + 2 groups state + H, d], conv [inner + 2 groups state, taps], conv.b, dt_bias [H], A_log [H], D [H],
+             norm [inner], o [d, inner]."""
+
+    takes_out = True
+    _NAMES = {"in": "in", "conv": "conv", "conv_bias": "conv.b", "dt_bias": "dt_bias", "a_log": "A_log", "d": "D", "norm": "norm", "o": "o"}
+
+    def __init__(self, spec, runtime):
+        super().__init__(spec, runtime)
+        self.d = int(self._param("hidden_size"))
+        self.H = int(self._param("num_heads"))
+        self.vdim = int(self._param("vdim"))
+        self.dim = int(self._param("state"))
+        self.G = int(self._param("groups"))
+        self.taps = int(self._param("taps"))
+        self.norm_groups = int(self._param("norm_groups"))
+        self.eps = float(self._param("eps"))
+        if min(self.H, self.G, self.dim, self.vdim) <= 0 or self.H % self.G or self.dim > 1024:
+            raise ConfigError(f"mamba2: sizes heads={self.H} on {self.G} groups, state={self.dim} vdim={self.vdim} (heads a multiple of the groups, state at most 1024)")
+        if not 1 <= self.taps <= ops.SHORT_CONV_MAX_TAPS:
+            raise ConfigError(f"mamba2: {self.taps} taps (1 to {ops.SHORT_CONV_MAX_TAPS})")
+        self.inner = self.H * self.vdim
+        if self.norm_groups <= 0 or self.inner % self.norm_groups:
+            raise ConfigError(f"mamba2: {self.norm_groups} norm groups do not divide {self.inner} numbers")
+        self.out_scale = float(spec.params.get("out_scale", 1.0))
+        self.names = dict(self._NAMES, **dict(spec.params.get("names", {})))
+        self.bc = self.G * self.dim
+        self.channels = self.inner + 2 * self.bc
+        self.w_in = self.w_conv = self.b_conv = self.dt_bias = self.a_log = self.skip = self.w_norm = self.w_o = None
+
+    def cache_need(self):
+        need = StateNeed((self.H, self.dim, self.vdim), torch.float32)
+        if self.taps > 1:  # the convolution's last inputs: exact in 32-bit whatever the run's type
+            return (need, StateNeed((self.taps - 1, self.channels), torch.float32))
+        return need
+
+    def param_infos(self) -> Dict[str, ParamInfo]:
+        p, n = self.prefix, self.names
+        return {
+            p + n["in"]: ParamInfo((self.inner + self.channels + self.H, self.d)),
+            p + n["conv"]: ParamInfo((self.channels, self.taps), "scalars"),
+            p + n["conv_bias"]: ParamInfo((self.channels,), "scalars", centre=0.0),
+            p + n["dt_bias"]: ParamInfo((self.H,), "scalars", centre=0.0),
+            p + n["a_log"]: ParamInfo((self.H,), "scalars", centre=0.0),
+            p + n["d"]: ParamInfo((self.H,), "scalars", centre=1.0),
+            p + n["norm"]: ParamInfo((self.inner,), "scalars", centre=1.0),
+            p + n["o"]: ParamInfo((self.d, self.inner)),
+        }
+
+    def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
+        p, n = self.prefix, self.names
+        self.w_in = tensors[p + n["in"]].contiguous()
+        self.w_conv = tensors[p + n["conv"]].t().contiguous()  # (stored [channels, taps]; the kernel reads [taps, channels])
+        self.b_conv, self.dt_bias, self.a_log, self.skip, self.w_norm = (
+            tensors[p + n[key]].contiguous() for key in ("conv_bias", "dt_bias", "a_log", "d", "norm"))
+        self.w_o = tensors[p + n["o"]].contiguous()
+
+    def forward(self, xn: torch.Tensor, step, cache, shared_cache: bool = False) -> torch.Tensor:
+        a, w_o = self.forward_unprojected(xn, step, cache, shared_cache)
+        return linear_to_stream(a, w_o)
+
+    def forward_unprojected(self, xn: torch.Tensor, step, cache, shared_cache: bool = False, out=None):
+        if shared_cache:
+            raise ConfigError("mamba2: a state cannot be another run's")
+        memory, inputs = cache if self.taps > 1 else (cache, None)
+        proj = linear(xn, self.w_in)
+        n = self.inner
+        z, raw_dt = proj[:, :n], proj[:, n + self.channels :]
+        conv = ops.short_conv(proj[:, n : n + self.channels], self.w_conv, None if inputs is None else inputs.state, step.slot_ids, step.seq_start,
+                              step.tok_seq, bias=self.b_conv, single=step.decode_only)
+        x, B, C = conv[:, :n], conv[:, n : n + self.bc], conv[:, n + self.bc :]
+        log_a, dt = ops.ssm_gates(raw_dt, self.a_log, self.dt_bias)
+        y = self._recurrence(C, B, x, log_a, dt, memory.state, step)
+        a = ops.ssm_gate_norm(y, x, self.skip, z, self.w_norm, self.eps, self.norm_groups, xn.dtype, out_scale=self.out_scale, out=out)
+        return a, self.w_o
+
+    def _recurrence(self, q, k, v, log_a, dt, state, step):
+        args = (q, k, v, log_a, dt, state, step.slot_ids, step.seq_start, self.H, self.dim, self.vdim)
+        if q.dtype == torch.bfloat16 and step.max_q_len >= _CHUNKED_MIN_TOKENS:
+            if ops.scalar_decay_chunked_takes(self.dim, self.vdim):
+                need = ops.scalar_decay_chunked_scratch_floats(step.n_seqs, step.max_q_len, self.H, self.dim, self.vdim)
+                scratch = self.rt.workspace.get("scalar_decay_chunks", need, torch.float32)
+                return ops.scalar_decay_chunked(*args, step.max_q_len, scratch, qk_heads=self.G)
+            if ops.gated_attn_chunked_takes(self.dim, self.vdim):
+                need = ops.gated_attn_chunked_scratch_floats(step.n_seqs, step.max_q_len, self.H, self.dim, self.vdim)
+                scratch = self.rt.workspace.get("gated_attn_chunks", need, torch.float32)
+                return ops.gated_attn_chunked(*args, step.max_q_len, scratch, qk_heads=self.G)
+        return ops.gated_attn(*args, qk_heads=self.G)

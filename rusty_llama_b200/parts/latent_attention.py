@@ -13,7 +13,7 @@ from ..kernels.linear import linear, linear_to_stream
 from ..spec import PartSpec
 from .base import MIXERS, POSITIONS, KVNeed, Mixer, ParamInfo
 
-_NAMES = {"q": "q", "kv": "dkv", "kv_norm": "dkv.norm", "k_up": "uk", "v_up": "uv", "sink": "sink", "gate": "g", "out": "o"}
+_NAMES = {"q": "q", "q_down": "dq", "q_norm": "dq.norm", "q_up": "uq", "kv": "dkv", "kv_norm": "dkv.norm", "k_up": "uk", "v_up": "uv", "sink": "sink", "gate": "g", "out": "o"}
 
 
 @MIXERS.register("latent_attention")
@@ -31,11 +31,15 @@ class LatentAttention(Mixer):
     (q_lat = W_uk[h]^T q_plain, so that the score is [q_lat | q_rot] . [c_j | kr_j]) and W_uv[h] to the
     probability-weighted sum of the latents, which is the same arithmetic in another order.
 
-    params: hidden_size, num_heads, dim, rot_dim, vdim, kv_rank, scale, eps (of the latent's norm),
+    With `q_rank` the queries come from a latent of their own, q[t] = W_uq (rmsnorm(W_dq xn[t]) * w_qnorm), in the place of W_q xn[t].
+
+    params: hidden_size, num_heads, dim, rot_dim, vdim, kv_rank, scale, eps (of the latents' norms),
             sink (bool), gate (bool), own_kv (bool: False for a layer that only reads another layer's cache),
-            window (0 = all keys), position (a PartSpec of kind "rotary" over the rotated part),
-            names (optional: tensor names after the prefix, keys q kv kv_norm k_up v_up sink gate out).
-    tensors: <prefix>q [H (dim + rot_dim), d], dkv [kv_rank + rot_dim, d], dkv.norm [kv_rank], uk [H dim, kv_rank],
+            window (0 = all keys), position (a PartSpec of kind "rotary" over the rotated part, pairs in either layout),
+            q_rank (0: no query latent),
+            names (optional: tensor names after the prefix, keys q q_down q_norm q_up kv kv_norm k_up v_up sink gate out).
+    tensors: <prefix>q [H (dim + rot_dim), d] (with q_rank: dq [q_rank, d], dq.norm [q_rank], uq [H (dim + rot_dim), q_rank]),
+             dkv [kv_rank + rot_dim, d], dkv.norm [kv_rank], uk [H dim, kv_rank],
              uv [H vdim, kv_rank], sink [H], g [H vdim, d], o [d, H vdim]."""
 
     def __init__(self, spec, runtime):
@@ -64,15 +68,16 @@ class LatentAttention(Mixer):
         fusion = self.position.decode_fusion()
         if fusion is None and getattr(self.position, "rotary_dim", 0):
             fusion = (self.position.inv_freq, self.position.rotary_dim, self.position.interleaved)
-        if fusion is None or (fusion[1] and not fusion[2]):
-            raise ConfigError("latent_attention: the position encoding must be a rotation of neighbouring pairs (or none)")
-        self.freq, rotary_dim = fusion[0], int(fusion[1])
+        if fusion is None:
+            raise ConfigError("latent_attention: the position encoding must be a rotation (or none)")
+        self.freq, rotary_dim, self.interleaved = fusion[0], int(fusion[1]), bool(fusion[2])
+        self.q_rank = int(spec.params.get("q_rank", 0) or 0)
         if rotary_dim > self.rot or rotary_dim % 2:
             raise ConfigError(f"latent_attention: {rotary_dim} rotated dimensions do not fit a rotated part of {self.rot}")
         self.n_pairs = rotary_dim // 2
         self.magnitude = float(getattr(self.position, "magnitude", 1.0))
         self.qd, self.vd, self.kvd = self.H * (self.dim + self.rot), self.H * self.vdim, self.rank + self.rot
-        self.w_in = self.w_o = self.w_ukT = self.w_uv = self.w_norm = self.sink = None
+        self.w_in = self.w_o = self.w_ukT = self.w_uv = self.w_norm = self.sink = self.w_uq = self.w_q_norm = None
 
     def cache_need(self):
         return KVNeed(1, self.kvd, self.window, values=False) if self.own_kv else None
@@ -82,12 +87,19 @@ class LatentAttention(Mixer):
 
     def param_infos(self) -> Dict[str, ParamInfo]:
         p, n = self.prefix, self.names
-        infos = {
-            p + n["q"]: ParamInfo((self.qd, self.d)),
+        if self.q_rank:
+            infos = {
+                p + n["q_down"]: ParamInfo((self.q_rank, self.d)),
+                p + n["q_norm"]: ParamInfo((self.q_rank,), "scalars", centre=1.0),
+                p + n["q_up"]: ParamInfo((self.qd, self.q_rank)),
+            }
+        else:
+            infos = {p + n["q"]: ParamInfo((self.qd, self.d))}
+        infos.update({
             p + n["k_up"]: ParamInfo((self.H * self.dim, self.rank)),
             p + n["v_up"]: ParamInfo((self.vd, self.rank)),
             p + n["out"]: ParamInfo((self.d, self.vd)),
-        }
+        })
         if self.own_kv:
             infos[p + n["kv"]] = ParamInfo((self.kvd, self.d))
             infos[p + n["kv_norm"]] = ParamInfo((self.rank,), "scalars")
@@ -99,8 +111,10 @@ class LatentAttention(Mixer):
 
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
         p, n = self.prefix, self.names
-        # one product serves the queries, the gate and (in a layer with a cache of its own) the latent row
-        parts = [tensors[p + n["q"]]]
+        # one product serves the queries (or their latent), the gate and (in a layer with a cache of its own) the latent row
+        parts = [tensors[p + n["q_down" if self.q_rank else "q"]]]
+        if self.q_rank:
+            self.w_q_norm, self.w_uq = tensors[p + n["q_norm"]].contiguous(), tensors[p + n["q_up"]].contiguous()
         if self.has_gate:
             parts.append(tensors[p + n["gate"]])
         if self.own_kv:
@@ -122,14 +136,18 @@ class LatentAttention(Mixer):
             raise ConfigError("latent_attention: a layer with a latent projection of its own fills its own cache, one without reads another's")
         T = xn.shape[0]
         proj = linear(xn, self.w_in)
-        q = proj[:, : self.qd]
-        g = proj[:, self.qd : self.qd + self.vd] if self.has_gate else None
+        first = self.q_rank or self.qd
+        q = proj[:, :first]
+        g = proj[:, first : first + self.vd] if self.has_gate else None
         kv = proj[:, proj.shape[1] - self.kvd :] if self.own_kv else None
         q_cat = torch.empty((T, self.H, self.kvd), dtype=xn.dtype, device=xn.device)
-        ops.latent_prep(
-            q, kv, self.w_norm, self.eps, self.freq, self.n_pairs, self.magnitude, step.tok_pos, step.tok_seq,
-            cache.block_table, cache.k_pages, q_cat, self.H, self.dim, self.rot, self.rank,
-        )
+        turn = (self.freq, self.n_pairs, self.magnitude, step.tok_pos, step.tok_seq, cache.block_table, cache.k_pages)
+        sizes = (self.H, self.dim, self.rot, self.rank, self.interleaved)
+        if self.q_rank:
+            # the queries' latent is normed beside the row that is cached; the queries exist after the product with it
+            c_q = ops.latent_prep(None, kv, self.w_norm, self.eps, *turn, None, *sizes, q_latent=q, q_norm=self.w_q_norm)
+            q, kv = linear(c_q, self.w_uq), None
+        ops.latent_prep(q, kv, self.w_norm, self.eps, *turn, q_cat, *sizes)
         if self.dim:
             ops.head_linear(q, self.dim + self.rot, self.w_ukT, q_cat.view(T, self.H * self.kvd), self.kvd)
         else:

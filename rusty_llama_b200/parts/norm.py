@@ -6,6 +6,7 @@ from typing import Dict, Mapping, Optional
 
 import torch
 
+from ..errors import ConfigError
 from ..kernels import ops
 from .base import NORMS, Norm, ParamInfo, ResidualStream
 
@@ -17,7 +18,8 @@ class RMSNorm(Norm):
     params: size, eps, name (optional: the tensor's name after the prefix, "weight" if absent), offset (optional, default 0:
     the stored tensor is the weight's distance from `offset`, y = ... * (offset + w); such a weight is kept in 32-bit whatever
     the run's type, since offset + w has more digits than w), float32 (optional bool: the weight is kept in 32-bit in every run,
-    for designs whose norms are 32-bit arithmetic throughout).  tensor: <prefix>weight [size]."""
+    for designs whose norms are 32-bit arithmetic throughout), groups (optional, default 1: the row is cut into that many equal
+    consecutive parts and each is divided by its own root mean square).  tensor: <prefix>weight [size]."""
 
     def __init__(self, spec, runtime):
         super().__init__(spec, runtime)
@@ -26,6 +28,9 @@ class RMSNorm(Norm):
         self.offset = float(spec.params.get("offset", 0.0))
         self.keep32 = bool(spec.params.get("float32", False))
         self.tensor_name = self.prefix + str(spec.params.get("name", "weight"))
+        self.groups = int(spec.params.get("groups", 1))
+        if self.groups < 1 or self.size % self.groups:
+            raise ConfigError(f"rmsnorm: {self.groups} groups do not divide a row of {self.size}")
         self.weight: Optional[torch.Tensor] = None
 
     def param_infos(self) -> Dict[str, ParamInfo]:
@@ -41,10 +46,14 @@ class RMSNorm(Norm):
             self.weight = (self.weight.to(torch.float32) + self.offset).contiguous()
 
     def rms_weight(self):
-        return self.weight, self.eps
+        return (self.weight, self.eps) if self.groups == 1 else None
 
     def forward(self, stream: ResidualStream, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
-        delta, delta_norm = stream.take_pending()
+        if self.groups > 1 and stream.pending_norm is not None:
+            stream.flush()  # (the kernel that norms a result before it adds it norms whole rows)
+        delta, delta_norm, gate = stream.take_pending()
+        if gate is not None or self.groups > 1:
+            return ops.gated_add_rmsnorm(stream.x, delta, gate, self.weight, self.eps, self.groups, stream.act_dtype, rows=rows, write_x=rows is None)
         if delta_norm is not None:
             return ops.normed_add_rmsnorm(
                 stream.x, delta, delta_norm[0], delta_norm[1], self.weight, self.eps, stream.act_dtype, rows=rows, write_x=rows is None,

@@ -33,12 +33,15 @@ class LayerSpec:
     """One layer: an arrangement (`block`) of a mixer, a feed-forward and norms.
 
     `norms` maps the names the arrangement uses ("mixer", "feed_forward" for a
-    pre-norm block) to norm parts.  `feed_forward` None: the layer has a mixer only."""
+    pre-norm block) to norm parts.  `feed_forward` None: the layer has a mixer only.
+    `block_params`, `block_prefix`: sizes, constants and tensor prefix of an arrangement that has tensors of its own."""
 
     block: str
     mixer: PartSpec
     feed_forward: Optional[PartSpec]
     norms: Mapping[str, PartSpec]
+    block_params: Mapping[str, Any] = field(default_factory=dict)
+    block_prefix: str = ""
 
 
 @dataclass(frozen=True)
