@@ -119,7 +119,7 @@ __global__ void short_conv_step_kernel(const T* __restrict__ x, int x_stride, co
   const int idx = blockIdx.x * blockDim.x + threadIdx.x;
   if (idx >= n_seqs * C) return;
   const int s = idx / C, c = idx - s * C;
-  float* rec = state + (size_t)slot_ids[s] * (taps - 1) * C + c;
+  float* rec = state + (size_t)__ldcg(slot_ids + s) * (taps - 1) * C + c;
   float v[CONV_MAX_TAPS];
 #pragma unroll
   for (int i = 0; i < CONV_MAX_TAPS; ++i)

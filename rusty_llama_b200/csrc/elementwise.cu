@@ -22,7 +22,7 @@ __global__ void embed_gather_kernel(const int* __restrict__ tokens, const TW* __
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x;
-  const TW* row = table + (size_t)tokens[t] * d;
+  const TW* row = table + (size_t)__ldcg(tokens + t) * d;
   float* o = out + (size_t)t * d;
   if (VEC) {  // d is a multiple of 4: every thread moves four values per round, all loads in flight at once
     for (int i = threadIdx.x * 4; i < d; i += blockDim.x * 4) {
@@ -317,8 +317,8 @@ __global__ void seq_begin_decode_kernel(int* __restrict__ state, const int* __re
   pdl_wait();
   const int i = blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= n_seqs) return;
-  int* rec = state + (size_t)slot_ids[i] * SEQ_FIELDS;
-  const int len = rec[0];
+  int* rec = state + (size_t)__ldcg(slot_ids + i) * SEQ_FIELDS;
+  const int len = __ldcg(rec);
   tok_pos[i] = len;
   seq_pos0[i] = len;
   seq_len[i] = len + 1;

@@ -24,6 +24,11 @@
 
 RL_DEFINE_ERROR_TEXT()
 
+// Every kernel here may start while its predecessors are still running (see pdl_wait), so whatever another kernel or a copy
+// writes is read through L2, never through the read-only path.
+template <typename T>
+__device__ __forceinline__ float gr_load(const T* p) { return to_f32(__ldcg(p)); }
+
 __device__ __forceinline__ float gr_logistic(float x) { return 1.0f / (1.0f + expf(-x)); }
 __device__ __forceinline__ float gr_log_logistic(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
 
@@ -36,7 +41,7 @@ __global__ void gla_log_decay_kernel(const T* __restrict__ z, int z_stride, cons
   for (long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (long long)gridDim.x * blockDim.x) {
     const long long t = idx / n;
     const int i = (int)(idx - t * n);
-    const float v = to_f32(z[t * z_stride + i]) + (bias ? bias[i] : 0.f);
+    const float v = gr_load(z + t * z_stride + i) + (bias ? bias[i] : 0.f);
     out[idx] = gr_log_logistic(v) * inv_tau;
   }
 }
@@ -68,17 +73,17 @@ __global__ void mlstm_gates_kernel(const T* __restrict__ gi, const T* __restrict
   pdl_wait();
   const int lane = threadIdx.x;
   const int s = blockIdx.x / H, h = blockIdx.x % H;
-  const int t0 = seq_start[s], t1 = seq_start[s + 1];
-  float* mp = m_state + (size_t)slot_ids[s] * H + h;
-  float m = *mp;
+  const int t0 = __ldcg(seq_start + s), t1 = __ldcg(seq_start + s + 1);
+  float* mp = m_state + (size_t)__ldcg(slot_ids + s) * H + h;
+  float m = __ldcg(mp);
   const float bi = bias_i ? bias_i[h] : 0.f, bf = bias_f ? bias_f[h] : 0.f;
   const float inv_cap = 1.0f / cap;
   for (int base = t0; base < t1; base += 32) {
     const int t = base + lane;
     float li = 0.f, lf = 0.f;
     if (t < t1) {
-      li = cap * tanhf((to_f32(gi[(size_t)t * in_stride + h]) + bi) * inv_cap);
-      lf = gr_log_logistic(cap * tanhf((to_f32(gf[(size_t)t * in_stride + h]) + bf) * inv_cap));
+      li = cap * tanhf((gr_load(gi + (size_t)t * in_stride + h) + bi) * inv_cap);
+      lf = gr_log_logistic(cap * tanhf((gr_load(gf + (size_t)t * in_stride + h) + bf) * inv_cap));
     }
     const int n = min(32, t1 - base);
     float la = 0.f, bb = 0.f, mo = 0.f;
@@ -119,17 +124,17 @@ mlstm_gates_scan_kernel(const T* __restrict__ gi, const T* __restrict__ gf, int 
   pdl_wait();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int s = blockIdx.x / H, h = blockIdx.x % H;
-  const int t0 = seq_start[s], t1 = seq_start[s + 1];
-  float* mp = m_state + (size_t)slot_ids[s] * H + h;
-  float m_in = *mp;
+  const int t0 = __ldcg(seq_start + s), t1 = __ldcg(seq_start + s + 1);
+  float* mp = m_state + (size_t)__ldcg(slot_ids + s) * H + h;
+  float m_in = __ldcg(mp);
   const float bi = bias_i ? bias_i[h] : 0.f, bf = bias_f ? bias_f[h] : 0.f;
   const float inv_cap = 1.0f / cap;
   for (int base = t0; base < t1; base += 32 * MG_WARPS) {
     const int t = base + threadIdx.x;
     float li = -INFINITY, lf = 0.f;  // past the end: the map that changes nothing
     if (t < t1) {
-      li = cap * tanhf((to_f32(gi[(size_t)t * in_stride + h]) + bi) * inv_cap);
-      lf = gr_log_logistic(cap * tanhf((to_f32(gf[(size_t)t * in_stride + h]) + bf) * inv_cap));
+      li = cap * tanhf((gr_load(gi + (size_t)t * in_stride + h) + bi) * inv_cap);
+      lf = gr_log_logistic(cap * tanhf((gr_load(gf + (size_t)t * in_stride + h) + bf) * inv_cap));
     }
     float F = lf, I = li;  // the tokens of this warp up to and with this lane's, as one map
 #pragma unroll
@@ -213,13 +218,13 @@ __global__ void gated_attn_kernel(const T* __restrict__ q, const T* __restrict__
   float* a_s = k_s + GR_TOK * dim;      // [GR_TOK][dim]
   float* v_s = a_s + GR_TOK * dim;      // [GR_TOK][32]
   float* part = v_s + GR_TOK * 32;      // [nw][GR_TOK][32]
-  const int t0 = seq_start[s], t1 = seq_start[s + 1];
-  float* st = state + (((size_t)slot_ids[s] * H + h) * dim) * vcols;
+  const int t0 = __ldcg(seq_start + s), t1 = __ldcg(seq_start + s + 1);
+  float* st = state + (((size_t)__ldcg(slot_ids + s) * H + h) * dim) * vcols;
   float S[32];
 #pragma unroll
   for (int r = 0; r < 32; ++r) {
     const int row = w * 32 + r;
-    S[r] = (row < dim && col_ok) ? st[(size_t)row * vcols + col] : 0.f;
+    S[r] = (row < dim && col_ok) ? __ldcg(st + (size_t)row * vcols + col) : 0.f;
   }
   for (int base = t0; base < t1; base += GR_TOK) {
     const int n = min(GR_TOK, t1 - base);
@@ -227,15 +232,15 @@ __global__ void gated_attn_kernel(const T* __restrict__ q, const T* __restrict__
       const int j = idx / dim, i = idx - j * dim;
       const int t = base + j;
       const size_t at = (size_t)t * in_stride + (size_t)qh * dim + i;
-      const float b = in_scale ? in_scale[(size_t)t * H + h] : 1.f;
-      q_s[idx] = to_f32(q[at]) * q_scale;
-      k_s[idx] = to_f32(k[at]) * b;
-      a_s[idx] = expf(per_channel ? log_decay[((size_t)t * H + h) * dim + i] : log_decay[(size_t)t * H + h]);
+      const float b = in_scale ? __ldcg(in_scale + (size_t)t * H + h) : 1.f;
+      q_s[idx] = gr_load(q + at) * q_scale;
+      k_s[idx] = gr_load(k + at) * b;
+      a_s[idx] = expf(per_channel ? __ldcg(log_decay + ((size_t)t * H + h) * dim + i) : __ldcg(log_decay + (size_t)t * H + h));
     }
     for (int idx = threadIdx.x; idx < n * 32; idx += blockDim.x) {
       const int j = idx >> 5, c = col0 + (idx & 31);
       float vv = 0.f;
-      if (c < vdim) vv = to_f32(v[(size_t)(base + j) * in_stride + (size_t)h * vdim + c]);
+      if (c < vdim) vv = gr_load(v + (size_t)(base + j) * in_stride + (size_t)h * vdim + c);
       else if (c < vcols) vv = 1.f;
       v_s[idx] = vv;
     }
@@ -344,8 +349,8 @@ gated_chunk_state_kernel(const T* __restrict__ k, const T* __restrict__ v, int i
   pdl_wait();
   const int s = blockIdx.x / H, h = blockIdx.x % H, c = blockIdx.y, col0 = blockIdx.z * GC_COLS, qh = h / (H / QH);
   const int vcols = vdim + ext;
-  const int t0 = seq_start[s] + c * GC;
-  const int n = min(GC, seq_start[s + 1] - t0);
+  const int t0 = __ldcg(seq_start + s) + c * GC;
+  const int n = min(GC, __ldcg(seq_start + s + 1) - t0);
   if (n <= 0) return;
   float* k_s = sm;             // [GC][dim]: first the decays' logarithms, then the weighted keys
   float* v_s = sm + GC * dim;  // [GC][GC_COLS]
@@ -355,16 +360,16 @@ gated_chunk_state_kernel(const T* __restrict__ k, const T* __restrict__ v, int i
   for (int idx = threadIdx.x; idx < n * dim; idx += 256) {
     const int i = idx / dim, r = idx - i * dim;
     const size_t th = (size_t)(t0 + i) * H + h;
-    k_s[idx] = GR_LOG2E * (per_channel ? log_decay[th * dim + r] : log_decay[th]);
+    k_s[idx] = GR_LOG2E * (per_channel ? __ldcg(log_decay + th * dim + r) : __ldcg(log_decay + th));
   }
   for (int idx = threadIdx.x; idx < n * narrow; idx += 256) {
     const int i = idx / narrow, e = idx - i * narrow, cc = col_x0 + e;
-    v_x[i * 4 + e] = cc < vdim ? to_f32(v[(size_t)(t0 + i) * in_stride + (size_t)h * vdim + cc]) : 1.f;
+    v_x[i * 4 + e] = cc < vdim ? gr_load(v + (size_t)(t0 + i) * in_stride + (size_t)h * vdim + cc) : 1.f;
   }
   for (int idx = threadIdx.x; idx < n * GC_COLS; idx += 256) {
     const int i = idx / GC_COLS, cc = col0 + (idx - i * GC_COLS);
     float vv = 0.f;
-    if (cc < vdim) vv = to_f32(v[(size_t)(t0 + i) * in_stride + (size_t)h * vdim + cc]);
+    if (cc < vdim) vv = gr_load(v + (size_t)(t0 + i) * in_stride + (size_t)h * vdim + cc);
     else if (cc < vcols) vv = 1.f;
     v_s[idx] = vv;
   }
@@ -382,8 +387,8 @@ gated_chunk_state_kernel(const T* __restrict__ k, const T* __restrict__ v, int i
   __syncthreads();
   for (int idx = threadIdx.x; idx < n * dim; idx += 256) {
     const int i = idx / dim, r = idx - i * dim;
-    const float b = in_scale ? in_scale[(size_t)(t0 + i) * H + h] : 1.f;
-    k_s[idx] = to_f32(k[(size_t)(t0 + i) * in_stride + (size_t)qh * dim + r]) * b * gr_exp2(k_s[idx]);
+    const float b = in_scale ? __ldcg(in_scale + (size_t)(t0 + i) * H + h) : 1.f;
+    k_s[idx] = gr_load(k + (size_t)(t0 + i) * in_stride + (size_t)qh * dim + r) * b * gr_exp2(k_s[idx]);
   }
   __syncthreads();
   const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
@@ -437,11 +442,11 @@ __global__ void gated_chunk_scan_kernel(float* __restrict__ state, const int* __
   const int e = blockIdx.y * blockDim.x + threadIdx.x;
   if (e >= elems) return;
   const int r = e / vcols;
-  const int len = seq_start[s + 1] - seq_start[s];
-  float* st = state + ((size_t)slot_ids[s] * H + h) * elems + e;
+  const int len = __ldcg(seq_start + s + 1) - __ldcg(seq_start + s);
+  float* st = state + ((size_t)__ldcg(slot_ids + s) * H + h) * elems + e;
   float* u = scratch + (size_t)blockIdx.x * max_chunks * elems + e;
   const float* g = chunk_decay + (size_t)blockIdx.x * max_chunks * dim + r;
-  float S = *st;
+  float S = __ldcg(st);
   const int n_chunks = (len + GC - 1) / GC;
   for (int c0 = 0; c0 < n_chunks; c0 += 8) {  // eight chunks' additions are asked for at once, then taken in order
     float add[8], dec[8];
@@ -476,8 +481,8 @@ gated_chunk_out_kernel(const T* __restrict__ q, const T* __restrict__ k, const T
   pdl_wait();
   const int s = blockIdx.x / H, h = blockIdx.x % H, c = blockIdx.y, qh = h / (H / QH);
   const int vcols = vdim + ext;
-  const int t0 = seq_start[s] + c * GC;
-  const int n = min(GC, seq_start[s + 1] - t0);
+  const int t0 = __ldcg(seq_start + s) + c * GC;
+  const int n = min(GC, __ldcg(seq_start + s + 1) - t0);
   if (n <= 0) return;
   const int DS = dim + 1;  // rows one apart in the banks
   float* q_s = sm;                    // [GC][DS]
@@ -490,7 +495,7 @@ gated_chunk_out_kernel(const T* __restrict__ q, const T* __restrict__ k, const T
   const int narrow = gc_narrow(vcols), wide_cols = vcols - narrow;
   for (int idx = threadIdx.x; idx < n * narrow; idx += 256) {
     const int i = idx / narrow, e = idx - i * narrow, cc = wide_cols + e;
-    v_x[i * 4 + e] = cc < vdim ? to_f32(v[(size_t)(t0 + i) * in_stride + (size_t)h * vdim + cc]) : 1.f;
+    v_x[i * 4 + e] = cc < vdim ? gr_load(v + (size_t)(t0 + i) * in_stride + (size_t)h * vdim + cc) : 1.f;
   }
   for (int idx = threadIdx.x; idx < GC * dim; idx += 256) {
     const int i = idx / dim, r = idx - i * dim;
@@ -498,9 +503,9 @@ gated_chunk_out_kernel(const T* __restrict__ q, const T* __restrict__ k, const T
     if (i < n) {
       const size_t at = (size_t)(t0 + i) * in_stride + (size_t)qh * dim + r;
       const size_t th = (size_t)(t0 + i) * H + h;
-      qv = to_f32(q[at]) * q_scale;
-      kv = to_f32(k[at]) * (in_scale ? in_scale[th] : 1.f);
-      la = GR_LOG2E * (per_channel ? log_decay[th * dim + r] : log_decay[th]);
+      qv = gr_load(q + at) * q_scale;
+      kv = gr_load(k + at) * (in_scale ? __ldcg(in_scale + th) : 1.f);
+      la = GR_LOG2E * (per_channel ? __ldcg(log_decay + th * dim + r) : __ldcg(log_decay + th));
     }
     q_s[i * DS + r] = qv;
     k_s[i * DS + r] = kv;
@@ -580,14 +585,14 @@ gated_chunk_out_kernel(const T* __restrict__ q, const T* __restrict__ k, const T
       const int i = idx / GC_COLS, cc = col0 + (idx - i * GC_COLS);
       float vv = 0.f;
       if (i < n) {
-        if (cc < vdim) vv = to_f32(v[(size_t)(t0 + i) * in_stride + (size_t)h * vdim + cc]);
+        if (cc < vdim) vv = gr_load(v + (size_t)(t0 + i) * in_stride + (size_t)h * vdim + cc);
         else if (cc < vcols) vv = 1.f;
       }
       v_s[idx] = vv;
     }
     for (int idx = threadIdx.x; idx < dim * GC_COLS; idx += 256) {
       const int r = idx / GC_COLS, cc = col0 + (idx - r * GC_COLS);
-      s_s[idx] = cc < vcols ? sp[(size_t)r * vcols + cc] : 0.f;
+      s_s[idx] = cc < vcols ? __ldcg(sp + (size_t)r * vcols + cc) : 0.f;
     }
     __syncthreads();
     float acc[4][4];
@@ -640,7 +645,7 @@ gated_chunk_out_kernel(const T* __restrict__ q, const T* __restrict__ k, const T
       const float qv = q_s[i * DS + r];
 #pragma unroll
       for (int e = 0; e < 4; ++e)
-        if (e < narrow) acc[e] += qv * sp[(size_t)r * vcols + wide_cols + e];
+        if (e < narrow) acc[e] += qv * __ldcg(sp + (size_t)r * vcols + wide_cols + e);
     }
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
@@ -722,13 +727,13 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ x, int x_stride,
   const int t = pair / H, h = pair - t * H;
   const float* xr = x + (size_t)t * x_stride + (size_t)h * xh;
   float inv_den = 1.f;
-  if (m != nullptr) inv_den = 1.0f / (fmaxf(fabsf(xr[n]), expf(-m[(size_t)t * H + h])) + den_eps);
+  if (m != nullptr) inv_den = 1.0f / (fmaxf(fabsf(__ldcg(xr + n)), expf(-__ldcg(m + (size_t)t * H + h))) + den_eps);
   float vals[HN_MAX_PER_LANE];
   float ss = 0.f;
 #pragma unroll
   for (int e = 0; e < HN_MAX_PER_LANE; ++e) {
     const int i = lane + 32 * e;
-    vals[e] = i < n ? xr[i] * inv_den : 0.f;
+    vals[e] = i < n ? __ldcg(xr + i) * inv_den : 0.f;
     ss += vals[e] * vals[e];
   }
   const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)n + eps);
@@ -742,7 +747,7 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ x, int x_stride,
       float y = vals[e] * inv;
       if (wv) y *= wv[i];
       if (g) {
-        const float gv = to_f32(g[i]);
+        const float gv = gr_load(g + i);
         y *= gate_act == 2 ? gv * gr_logistic(gv) : (gate_act == 1 ? gr_logistic(gv) : gv);
       }
       o[i] = from_f32<T>(y * out_scale);

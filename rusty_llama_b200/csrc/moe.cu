@@ -15,6 +15,8 @@
 // blocks without work leave, so a step with these kernels can be captured in a CUDA graph.  Each output is one
 // running 32-bit sum over ascending k, whatever the tile it lies in: a token's result does not depend on what
 // else is in the batch.
+#include <float.h>
+
 #include "common.cuh"
 
 RL_DEFINE_ERROR_TEXT()
@@ -113,7 +115,7 @@ __global__ void moe_router_choose_kernel(const float* __restrict__ logits, const
   for (int e = lane; e < E; e += 32) {
     const float s = logistic ? 1.0f / (1.0f + expf(-lg[e])) : expf(lg[e] - mx) / sum;
     z[e] = s;
-    choice[e] = s + (bias ? bias[e] : 0.f);
+    choice[e] = fmaxf(s + (bias ? bias[e] : 0.f), -FLT_MAX);  // (also what is not a number: every expert stays one that can be chosen once)
   }
   __syncwarp();
   float chosen_sum = 0.f;

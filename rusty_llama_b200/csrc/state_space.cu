@@ -238,8 +238,8 @@ scalar_chunk_state_kernel(const bf16* __restrict__ k, const bf16* __restrict__ v
   pdl_trigger();
   pdl_wait();
   const int s = blockIdx.x / H, h = blockIdx.x % H, c = blockIdx.y, qh = h / (H / QH);
-  const int t0 = seq_start[s] + c * SC;
-  const int n = min(SC, seq_start[s + 1] - t0);
+  const int t0 = __ldcg(seq_start + s) + c * SC;
+  const int n = min(SC, __ldcg(seq_start + s + 1) - t0);
   if (n <= 0) return;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int g = lane >> 2, t4 = lane & 3;
@@ -333,8 +333,8 @@ __global__ void scalar_chunk_scan_kernel(float* __restrict__ state, const int* _
   const int s = blockIdx.x / H, h = blockIdx.x % H;
   const int e = (blockIdx.y * blockDim.x + threadIdx.x) * V;
   if (e >= elems) return;
-  const int len = seq_start[s + 1] - seq_start[s];
-  float* st = state + ((size_t)slot_ids[s] * H + h) * elems + e;
+  const int len = __ldcg(seq_start + s + 1) - __ldcg(seq_start + s);
+  float* st = state + ((size_t)__ldcg(slot_ids + s) * H + h) * elems + e;
   float* u = scratch + (size_t)blockIdx.x * max_chunks * elems + e;
   const float* dec = chunk_decay + (size_t)blockIdx.x * max_chunks;
   const int n_chunks = (len + SC - 1) / SC;
@@ -381,8 +381,8 @@ scalar_chunk_out_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k, 
   pdl_trigger();
   pdl_wait();
   const int s = blockIdx.x / H, h = blockIdx.x % H, c = blockIdx.y, qh = h / (H / QH);
-  const int t0 = seq_start[s] + c * SC;
-  const int n = min(SC, seq_start[s + 1] - t0);
+  const int t0 = __ldcg(seq_start + s) + c * SC;
+  const int n = min(SC, __ldcg(seq_start + s + 1) - t0);
   if (n <= 0) return;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int g = lane >> 2, t4 = lane & 3;
