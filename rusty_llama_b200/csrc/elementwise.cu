@@ -551,85 +551,154 @@ RL_API int rl_normed_add_rmsnorm(float* x, const void* delta, int delta_dtype, i
 //   s = delta[0][t] + delta[1][t] + ...                                       (32-bit, in this order)
 //   v = x[t] + s * logistic(z[t] + bias)        (without a gate: x[t] + s)    x[t] = v
 //   if w: the row cut into `groups` equal consecutive parts, out[r] = v / sqrt(mean(v^2 over its part) + eps) * w
-// One block per row, the row in registers.  A unit is U neighbouring values (four where the sizes allow); every unit leaves its
-// sum of squares in shared memory, a warp per part adds them up in an order that depends on the sizes alone.  So a row's bits
-// depend neither on the number of rows nor on how many threads work it: the launcher takes few threads with several units each
-// for the many rows of a prompt step and a thread per unit for the few rows of a decode step.
+// One block per row, the row in registers.  A unit is U neighbouring values (four where the sizes allow).  Where a part is a
+// multiple of 32 units, a warp adds up the squares of 32 neighbouring units by its tree and every thread then adds the sums of its
+// part's runs of 32 in their order; else every unit leaves its sum in shared memory and a warp per part adds them up.  Either
+// way the order depends on the sizes alone, so a row's bits depend neither on the number of rows nor on how many threads work
+// it: the launcher takes few threads with several units each for the many rows of a prompt step and a thread per unit for the
+// few rows of a decode step.
 template <typename TA, typename TW, typename TD, int U, int UNITS>
-__global__ void __launch_bounds__(UNITS == 4 ? 256 : 1024)
+__global__ void __launch_bounds__(U == 4 && UNITS > 1 ? 512 : 1024)
 gated_add_rmsnorm_kernel(float* __restrict__ x, const TD* __restrict__ delta, int n_parts, long long part_stride,
                          const TA* __restrict__ z, int z_stride, const float* __restrict__ gate_bias, const TW* __restrict__ w,
                          TA* __restrict__ out, const int* __restrict__ rows, int d, int groups, float eps, int write_x) {
-  extern __shared__ __align__(16) float unit_ss[];  // [d / U], then 1 / rms of the parts [groups]
+  extern __shared__ __align__(16) float unit_ss[];  // sums of squares: [d / U] of the units, or of runs of 32; then 1 / rms of the parts
   pdl_trigger();
   pdl_wait();
   const int r = blockIdx.x;
   const int t = rows ? rows[r] : r;
   const int n_units = d / U, per_group = n_units / groups;
-  float* inv_rms = unit_ss + n_units;
+  const bool runs = per_group % 32 == 0;
   float* xr = x + (size_t)t * d;
-  float v[UNITS][U], wv[UNITS][U];
+  float v[UNITS][U], wv[UNITS][U], s[UNITS][U];
+  // everything a thread needs is asked for before anything is used
 #pragma unroll
   for (int c = 0; c < UNITS; ++c) {
     const int u = threadIdx.x + c * blockDim.x, i = u * U;
-    if (u >= n_units) continue;
-    float s[U], zv[U];
 #pragma unroll
-    for (int e = 0; e < U; ++e) s[e] = 0.f;
-    if (U == 4) {
-      load4_g<float>(xr + i, v[c]);
-      if (w != nullptr) load4_g<TW>(w + i, wv[c]);
-      if (z != nullptr) load4_g<TA>(z + (size_t)t * z_stride + i, zv);
-    } else {
-      v[c][0] = xr[i];
-      if (w != nullptr) wv[c][0] = to_f32(w[i]);
-      if (z != nullptr) zv[0] = to_f32(z[(size_t)t * z_stride + i]);
+    for (int e = 0; e < U; ++e) v[c][e] = wv[c][e] = s[c][e] = 0.f;
+    if (u < n_units) {
+      if (U == 4) {
+        load4_g<float>(xr + i, v[c]);
+        if (w != nullptr) load4_g<TW>(w + i, wv[c]);
+        if (n_parts > 0) load4_g<TD>(delta + (size_t)t * d + i, s[c]);
+      } else {
+        v[c][0] = xr[i];
+        if (w != nullptr) wv[c][0] = to_f32(w[i]);
+        if (n_parts > 0) s[c][0] = to_f32(delta[(size_t)t * d + i]);
+      }
     }
-    for (int p = 0; p < n_parts; ++p) {
-      float dv[U];
-      const TD* dp = delta + (size_t)p * part_stride + (size_t)t * d + i;
-      if (U == 4) load4_g<TD>(dp, dv);
-      else dv[0] = to_f32(dp[0]);
+  }
+  if (z != nullptr) {
+    float zv[UNITS][U], bv[UNITS][U];
 #pragma unroll
-      for (int e = 0; e < U; ++e) s[e] += dv[e];
+    for (int c = 0; c < UNITS; ++c) {
+      const int u = threadIdx.x + c * blockDim.x, i = u * U;
+      if (u < n_units) {
+        if (U == 4) {
+          load4_g<TA>(z + (size_t)t * z_stride + i, zv[c]);
+          load4_g<float>(gate_bias + i, bv[c]);
+        } else {
+          zv[c][0] = to_f32(z[(size_t)t * z_stride + i]);
+          bv[c][0] = gate_bias[i];
+        }
+      }
     }
-    if (z != nullptr) {
+    for (int p = 1; p < n_parts; ++p) {
 #pragma unroll
-      for (int e = 0; e < U; ++e) s[e] *= 1.0f / (1.0f + expf(-(zv[e] + gate_bias[i + e])));
+      for (int c = 0; c < UNITS; ++c) {
+        const int u = threadIdx.x + c * blockDim.x, i = u * U;
+        if (u < n_units) {
+          float dv[U];
+          const TD* dp = delta + (size_t)p * part_stride + (size_t)t * d + i;
+          if (U == 4) load4_g<TD>(dp, dv);
+          else dv[0] = to_f32(dp[0]);
+#pragma unroll
+          for (int e = 0; e < U; ++e) s[c][e] += dv[e];
+        }
+      }
     }
+#pragma unroll
+    for (int c = 0; c < UNITS; ++c)
+#pragma unroll
+      for (int e = 0; e < U; ++e) {
+        if (sizeof(TA) == 2) s[c][e] *= __fdividef(1.0f, 1.0f + __expf(-(zv[c][e] + bv[c][e])));  // (a few units in the last place of 32 bits)
+        else s[c][e] *= 1.0f / (1.0f + expf(-(zv[c][e] + bv[c][e])));
+      }
+  } else {
+    for (int p = 1; p < n_parts; ++p) {
+#pragma unroll
+      for (int c = 0; c < UNITS; ++c) {
+        const int u = threadIdx.x + c * blockDim.x, i = u * U;
+        if (u < n_units) {
+          float dv[U];
+          const TD* dp = delta + (size_t)p * part_stride + (size_t)t * d + i;
+          if (U == 4) load4_g<TD>(dp, dv);
+          else dv[0] = to_f32(dp[0]);
+#pragma unroll
+          for (int e = 0; e < U; ++e) s[c][e] += dv[e];
+        }
+      }
+    }
+  }
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
+#pragma unroll
+  for (int c = 0; c < UNITS; ++c) {
+    const int u = threadIdx.x + c * blockDim.x, i = u * U;
     float ss = 0.f;
+    if (u < n_units) {
 #pragma unroll
-    for (int e = 0; e < U; ++e) {
-      v[c][e] += s[e];
-      ss += v[c][e] * v[c][e];
+      for (int e = 0; e < U; ++e) {
+        v[c][e] += s[c][e];
+        ss += v[c][e] * v[c][e];
+      }
+      if (write_x) {
+        if (U == 4) store4<float>(xr + i, v[c]);
+        else xr[i] = v[c][0];
+      }
     }
-    if (write_x) {
-      if (U == 4) store4<float>(xr + i, v[c]);
-      else xr[i] = v[c][0];
+    if (w != nullptr && u - lane < n_units) {  // (uniform over the warp)
+      if (runs) {
+        ss = warp_sum(ss);
+        if (lane == 0) unit_ss[u >> 5] = ss;
+      } else if (u < n_units) {
+        unit_ss[u] = ss;
+      }
     }
-    unit_ss[u] = ss;
   }
   if (w == nullptr) return;
   __syncthreads();
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
-  for (int g = warp; g < groups; g += nwarps) {
-    float ss = 0.f;
-    for (int u = lane; u < per_group; u += 32) ss += unit_ss[g * per_group + u];
-    ss = warp_sum(ss);
-    if (lane == 0) inv_rms[g] = 1.0f / sqrtf(ss / (float)(per_group * U) + eps);
+  float* inv_rms = unit_ss + n_units;
+  if (!runs) {
+    for (int g = warp; g < groups; g += nwarps) {
+      float ss = 0.f;
+      for (int u = lane; u < per_group; u += 32) ss += unit_ss[g * per_group + u];
+      ss = warp_sum(ss);
+      if (lane == 0) inv_rms[g] = 1.0f / sqrtf(ss / (float)(per_group * U) + eps);
+    }
+    __syncthreads();
   }
-  __syncthreads();
+  const int run_len = per_group >> 5;
   TA* o = out + (size_t)r * d;
 #pragma unroll
   for (int c = 0; c < UNITS; ++c) {
     const int u = threadIdx.x + c * blockDim.x, i = u * U;
-    if (u >= n_units) continue;
-    const float inv = inv_rms[u / per_group];
-    float y[U];
+    if (u < n_units) {
+      float inv;
+      if (runs) {
+        const int first = (u >> 5) / run_len * run_len;
+        float ss = 0.f;
+        for (int k = 0; k < run_len; ++k) ss += unit_ss[first + k];
+        inv = 1.0f / sqrtf(ss / (float)(per_group * U) + eps);
+      } else {
+        inv = inv_rms[u / per_group];
+      }
+      float y[U];
 #pragma unroll
-    for (int e = 0; e < U; ++e) y[e] = v[c][e] * inv * wv[c][e];
-    if (U == 4) store4<TA>(o + i, y);
-    else o[i] = from_f32<TA>(y[0]);
+      for (int e = 0; e < U; ++e) y[e] = v[c][e] * inv * wv[c][e];
+      if (U == 4) store4<TA>(o + i, y);
+      else o[i] = from_f32<TA>(y[0]);
+    }
   }
 }
 
@@ -639,10 +708,10 @@ static int launch_gated_add_rmsnorm(float* x, const void* delta, int n_parts, lo
                                     float eps, int write_x, cudaStream_t stream) {
   // (which body runs depends on sizes and addresses only)
   const bool vec = (d / groups) % 4 == 0 && z_stride % 4 == 0 && part_stride % 4 == 0 &&
-                   (((uintptr_t)x | (uintptr_t)delta | (uintptr_t)z | (uintptr_t)w | (uintptr_t)out) % 16 == 0);
+                   (((uintptr_t)x | (uintptr_t)delta | (uintptr_t)z | (uintptr_t)w | (uintptr_t)out | (uintptr_t)gate_bias) % 16 == 0);
   const int n_units = vec ? d / 4 : d;
   const size_t smem = (size_t)(n_units + groups) * sizeof(float);
-  if (n_units > 8 * 1024 || smem > 48 * 1024) RL_REFUSE(3, "gated_add_rmsnorm: a row of %d values (%d parts) is too long", d, groups);
+  if (n_units > (vec ? 8 * 512 : 8 * 1024) || smem > 48 * 1024) RL_REFUSE(3, "gated_add_rmsnorm: a row of %d values (%d parts) is too long", d, groups);
   const int full = n_units >= 1024 ? 1024 : ((n_units + 31) / 32) * 32;
 #define RL_GAR(U, UNITS, TH, EARLY)                                                                                                    \
   do {                                                                                                                                 \
@@ -651,9 +720,11 @@ static int launch_gated_add_rmsnorm(float* x, const void* delta, int n_parts, lo
     return 0;                                                                                                                          \
   } while (0)
   if (vec) {
-    if (n_rows >= ROWS_KERNEL_MIN_ROWS && n_units > 256 && n_units <= 1024) RL_GAR(4, 4, 256, true);
+    if (n_rows >= ROWS_KERNEL_MIN_ROWS && n_units > 256 && n_units <= 512) RL_GAR(4, 2, 256, true);
+    if (n_rows >= ROWS_KERNEL_MIN_ROWS && n_units > 512 && n_units <= 1024) RL_GAR(4, 2, 512, true);
     if (n_units <= 1024) RL_GAR(4, 1, full, true);
-    RL_GAR(4, 8, 1024, true);
+    if (n_units <= 2048) RL_GAR(4, 4, 512, true);
+    RL_GAR(4, 8, 512, true);
   }
   if (n_units <= 1024) RL_GAR(1, 1, full, false);
   RL_GAR(1, 8, 1024, false);

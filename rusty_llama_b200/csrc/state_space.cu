@@ -50,7 +50,7 @@ RL_API int rl_ssm_gates(const void* raw, int dtype, int raw_stride, const float*
 // One block per row; a unit is U neighbouring numbers (four where the sizes allow), kept in registers; every unit leaves its sum of
 // squares in shared memory and a warp per part adds them up, so a row's bits depend on the sizes alone.
 template <typename T, int U, int UNITS>
-__global__ void __launch_bounds__(UNITS == 1 ? 1024 : 256)
+__global__ void __launch_bounds__(UNITS == 1 ? 1024 : 512)
 ssm_gate_norm_kernel(const float* __restrict__ y, int y_stride, const T* __restrict__ x, int x_stride, const float* __restrict__ D, int vdim,
                      const T* __restrict__ z, int z_stride, const float* __restrict__ w, float eps, int groups, T* __restrict__ out,
                      int out_stride, int n, float out_scale) {
@@ -125,11 +125,11 @@ static int launch_gate_norm(const float* y, int y_stride, const void* x, int x_s
   if (vec) {
     if (n_units <= 1024 && (n_rows < 64 || n_units <= 256)) RL_SGN(4, 1, full);
     if (n_units <= 1024) RL_SGN(4, 4, 256);
-    if (n_units <= 4096) RL_SGN(4, 16, 256);
-    RL_SGN(4, 32, 256);
+    if (n_units <= 2048) RL_SGN(4, 4, 512);
+    RL_SGN(4, 16, 512);
   }
   if (n_units <= 1024) RL_SGN(1, 1, full);
-  RL_SGN(1, 32, 256);
+  RL_SGN(1, 16, 512);
 #undef RL_SGN
 }
 

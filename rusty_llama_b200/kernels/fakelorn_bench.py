@@ -84,12 +84,13 @@ def kernel_table(z: dict, T: int, batch: int, ctx: int, peaks: dict) -> Dict[str
         seq_len = seq_pos0 + per
         slots = torch.arange(n_seqs, **i32)
         # ---- the gated result, the residual sum and the norm in parts
-        x = torch.randn(rows, d, device=dev)
-        delta, gate_z, w = torch.randn(rows, d, device=dev, dtype=bf), torch.randn(rows, d, device=dev, dtype=bf), torch.ones(d, device=dev)
-        bias = torch.zeros(d, device=dev)
         nbytes = rows * d * (4 + 4 + 2 + 2)
-        us_like = timed(lambda: ops.add_rmsnorm(x, delta, w, 1e-5, bf))
-        us = timed(lambda: ops.gated_add_rmsnorm(x, delta, (gate_z, bias), w, 1e-5, z["norm_groups"], bf))
+        nv = min(mb._copies(nbytes), 8) if prompt else 1  # (several sets of rows, together larger than the L2)
+        sets = [(torch.randn(rows, d, device=dev), torch.randn(rows, d, device=dev, dtype=bf), torch.randn(rows, d, device=dev, dtype=bf)) for _ in range(nv)]
+        w, bias = torch.ones(d, device=dev), torch.zeros(d, device=dev)
+        us_like = mb._time(lambda i: ops.add_rmsnorm(sets[i][0], sets[i][1], w, 1e-5, bf), nv, **it)
+        us = mb._time(lambda i: ops.gated_add_rmsnorm(sets[i][0], sets[i][1], (sets[i][2], bias), w, 1e-5, z["norm_groups"], bf), nv, **it)
+        del sets
         note(f"{tag}_gated_add_norm", us, nbytes + rows * d * 2, 0, ("add_rmsnorm", us_like, nbytes, 0))
         # ---- differential attention: store, the two maps' attention, their difference and its norm
         hd = 2 * MAP_DIM
