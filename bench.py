@@ -474,7 +474,7 @@ def main() -> int:
     ap.add_argument("--reps", type=int, default=5, help="repetitions of the timed steps (mean and standard deviation are reported)")
     ap.add_argument("--no-kernels", action="store_true", help="leave out the kernel-by-kernel table")
     ap.add_argument("--workload", action="store_true", help="with --sizes 1b or 13b: BASELINE.json's workload of unequal prompts through LLM.generate, instead of the contract line")
-    ap.add_argument("--design", default="", choices=["", "vezatar", "revirax", "tefavik", "namalix", "fakelorn"], help="instead of the contract line: this design beside Llama (Tefavik and Namalix: beside Revirax; Fakelorn: beside Vezatar) at equal sizes (prompt and decode steps through the engine, and its kernels alone)")
+    ap.add_argument("--design", default="", choices=["", "vezatar", "revirax", "tefavik", "namalix", "fakelorn"], help="instead of the default line: this design beside Llama (Tefavik and Namalix: beside Revirax; Fakelorn: beside Vezatar) at equal sizes (prompt and decode steps through the engine, and its kernels alone)")
     ap.add_argument("--design-sizes", default="small,lite", help="with --design: which of the sizes small, lite, wide")
     ap.add_argument("--design-tokens", type=int, default=2048, help="with --design: tokens of the prompt step, and the context of the decode steps")
     args = ap.parse_args()
