@@ -75,7 +75,7 @@ RL_DEFINE_ERROR_TEXT()
 
 struct SmallItems {
   uint64_t q_full, k_full[KV_STAGES], v_full[KV_STAGES];
-  uint64_t s_full[2], p_ready, pv_done[2];
+  uint64_t s_full[2], p_ready[2], pv_done[2];
   uint64_t drain_bar;              // an issuer that gives up waits here for the MMAs it has issued
   uint32_t tmem_slot;
   int abort_flag;
@@ -235,7 +235,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   uint64_t(&k_full)[KV_STAGES] = sm.k_full;
   uint64_t(&v_full)[KV_STAGES] = sm.v_full;
   uint64_t(&s_full)[2] = sm.s_full;
-  uint64_t& p_ready = sm.p_ready;
+  uint64_t(&p_ready)[2] = sm.p_ready;
   uint64_t(&pv_done)[2] = sm.pv_done;
   uint64_t& drain_bar = sm.drain_bar;
   uint32_t& tmem_slot = sm.tmem_slot;
@@ -272,7 +272,8 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     }
     mbar_init(&s_full[0], 1);
     mbar_init(&s_full[1], 1);
-    mbar_init(&p_ready, SOFTMAX_WARPS);  // one arrival per softmax warp
+    mbar_init(&p_ready[0], SOFTMAX_WARPS);  // one arrival per softmax warp
+    mbar_init(&p_ready[1], SOFTMAX_WARPS);
     mbar_init(&pv_done[0], 1);
     mbar_init(&pv_done[1], 1);
     mbar_init(&drain_bar, 1);
@@ -342,7 +343,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       // go out as two blocks of instructions (qk_block, pv_block), each with ONE commit.  Each block also asks about
       // data that is needed later (mbarrier.test_wait, before its MMAs, read after them); the answers are NOT used
       // to skip the waits below: the tensor-core GEMM's issuer, built the same way, gave up on a stage about once in
-      // 10^5 launches when it skipped its wait after a yes, and until that is understood every tile is waited for.
+      // 10^5 launches when it skipped its wait after a yes (before p_ready had two barriers), so every tile is waited for.
       // (a map's half starts at the second sub-tile of 64 dims, or 64 bytes into the only one)
       constexpr uint64_t HALF_Q = HD == 128 ? SUBQ_BYTES / 16 : 4, HALF_K = HD == 128 ? SUBK_BYTES / 16 : 4;
       const uint64_t q_desc = make_smem_desc(q_addr) + (MAPS > 1 ? (h % MAPS) * HALF_Q : 0);
@@ -370,7 +371,9 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       for (int j = 0; j < n_tiles && ok; ++j) {
         // S of tile j + 1 was issued before this tile's softmax began (above, or at the end of the trip before).  Its
         // buffer was last read by the P V of tile j - 1, which stands before it in this thread's order.
-        if (!(ok = wait_for(&p_ready, j & 1, 15))) break;
+        // (P has a barrier per S buffer: the softmax warps may finish tile j + 1 before this thread looks for tile j, and a wait
+        // on the parity of ONE barrier that had completed both phases by then would never return)
+        if (!(ok = wait_for(&p_ready[j & 1], (j >> 1) & 1, 15))) break;
         const int st = j % KV_STAGES;
         if (!(ok = wait_for(&v_full[st], (j / KV_STAGES) & 1, 16))) break;
         tc_fence_after();
@@ -500,7 +503,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       // P is complete (and the accumulator rescaled if it had to be): hand both to the tensor core
       tc_fence_before();
       __syncwarp();
-      if (lane == 0) mbar_arrive(&p_ready);
+      if (lane == 0) mbar_arrive(&p_ready[j & 1]);
     }
     if (ok && !mbar_wait_role(&pv_done[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1, ctl, 20)) give_up(20);
     ok = __all_sync(0xffffffffu, ok);  // (the way out below works as a warp)

@@ -313,7 +313,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
           // (Issuing the slice as one block of instructions, with the next stage's wait asked ahead by a
           // mbarrier.test_wait and skipped when the answer was yes, took a single tile from 0.785 to 0.975 of the tensor
           // core's nominal rate; in long runs of decode steps at batch 64 about one launch in 10^5 then gave up on a stage
-          // that never arrived, and the cause was not found: the loop waits, issues and commits in turn.)
+          // that never arrived: the loop waits, issues and commits in turn.  A fault in the prompt attention that made its
+          // successor give up in that way has been found and fixed since; the other form has not been tried again.)
           umma_bf16_x4(tmem_d, a_desc0 + stage_off, b_desc0 + stage_off, idesc, kb > kb0 ? 1u : 0u);
           umma_commit(&empty_bar[s]);
           stage_off += (uint64_t)(STG_BYTES >> 4);

@@ -94,3 +94,69 @@ def test_the_model_sees_a_wrong_parity():
                 seen.add(n)
                 queue.append(n)
     assert problem is not None
+
+
+def _explore_attention(T: int, p_barriers: int):
+    """csrc/attention_prefill_tc.cu over T key tiles, with `p_barriers` barriers for "the probabilities are ready".  Actors: the
+    producer (K and V tiles into two stages each; a K stage is free when the S it fed is complete, a V stage when its P V is), the
+    copy engine, the issuer (S 0, S 1, then for every tile j: wait for P j and V j, issue P V j, wait for K j + 2, issue S j + 2),
+    the tensor pipe (in order), and the softmax warps as one actor (wait for S j, announce P j).  Returns the first problem
+    found or None."""
+    loads = [(kind, j) for j in range(T) for kind in "KV"]
+    order = [("S", j) for j in range(min(2, T))]
+    for j in range(T):
+        order.append(("O", j))
+        if j + 2 < T:
+            order.append(("S", j + 2))
+    zero = (0, 0)
+    bump = lambda b, i: tuple(n + (k == i) for k, n in enumerate(b))  # noqa: E731
+    # producer's place, copies in flight, completed phases of k_full, v_full, s_full, pv_done, p_ready, issuer's place, half a wait, issued, softmax's place
+    start = (0, (), zero, zero, zero, zero, (0,) * p_barriers, 0, 0, (), 0)
+    seen, queue = {start}, deque([start])
+    while queue:
+        lo, fly, kf, vf, sf, pv, pr, io, half, iss, sm = queue.popleft()
+        nxt = []
+        if lo < len(loads):
+            kind, j = loads[lo]
+            if j < 2 or _ok((sf if kind == "K" else pv)[j & 1], ((j >> 1) - 1) & 1):
+                nxt.append((lo + 1, fly + (loads[lo],), kf, vf, sf, pv, pr, io, half, iss, sm))
+        for n, (kind, j) in enumerate(fly):
+            k2, v2 = (bump(kf, j & 1), vf) if kind == "K" else (kf, bump(vf, j & 1))
+            nxt.append((lo, fly[:n] + fly[n + 1:], k2, v2, sf, pv, pr, io, half, iss, sm))
+        if io < len(order):
+            kind, j = order[io]
+            if kind == "S":
+                if _ok(kf[j & 1], (j >> 1) & 1):
+                    nxt.append((lo, fly, kf, vf, sf, pv, pr, io + 1, 0, iss + (order[io],), sm))
+            elif half == 0:
+                if _ok(pr[j % p_barriers], (j // p_barriers) & 1):
+                    if sm <= j:
+                        return f"P V {j} goes on before its probabilities are there"
+                    nxt.append((lo, fly, kf, vf, sf, pv, pr, io, 1, iss, sm))
+            elif _ok(vf[j & 1], (j >> 1) & 1):
+                nxt.append((lo, fly, kf, vf, sf, pv, pr, io + 1, 0, iss + (order[io],), sm))
+        if iss:
+            kind, j = iss[0]
+            s2, o2 = (bump(sf, j & 1), pv) if kind == "S" else (sf, bump(pv, j & 1))
+            nxt.append((lo, fly, kf, vf, s2, o2, pr, io, half, iss[1:], sm))
+        if sm < T and _ok(sf[sm & 1], (sm >> 1) & 1):
+            nxt.append((lo, fly, kf, vf, sf, pv, bump(pr, sm % p_barriers), io, half, iss, sm + 1))
+        if not nxt and (lo < len(loads) or io < len(order) or sm < T):
+            return f"nothing can move: producer at {loads[lo:lo + 1]}, issuer at {order[io:io + 1]}, softmax at {sm}"
+        for n in nxt:
+            if n not in seen:
+                seen.add(n)
+                queue.append(n)
+    return None
+
+
+@pytest.mark.parametrize("T", [1, 2, 3, 4, 5, 8])
+def test_prompt_attention_never_stalls_with_a_barrier_per_score_buffer(T):
+    assert _explore_attention(T, p_barriers=2) is None
+
+
+def test_prompt_attention_with_one_barrier_for_the_probabilities_can_stall():
+    """Tile j + 1's scores are under way before the issuer looks for tile j's probabilities, so the softmax warps can announce both
+    first; the parity of a single barrier is then back where it was, and the producer ends waiting for a value stage."""
+    problem = _explore_attention(4, p_barriers=1)
+    assert problem is not None and "nothing can move" in problem and "('V'" in problem
