@@ -25,6 +25,9 @@
 // eight product warps.  At head size 64 a page's keys and values are half as many bytes, so the ring
 // has six stages instead of three and the same bytes are in flight.
 //
+// A learned bias by head and distance (`rl_distance_bias`): a thread's four scores of a page need four numbers, asked for before
+// the page is waited for; beyond the last distance with a number of its own they are two registers.
+//
 // Every mbarrier wait is bounded; on expiry a code goes to status[0] and the block drains.
 #include "tc_common.cuh"
 #include "attention_merge.cuh"
@@ -100,7 +103,8 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
                        const float* __restrict__ inv_freq, int rot, int interleaved,
                        unsigned int* __restrict__ counters, bf16* __restrict__ out, int out_stride,
                        const float* __restrict__ q_parts, int n_parts, long long part_stride, int test_role,
-                       uint32_t test_ns, const float* __restrict__ sink, int chunk, float softcap, int maps) {
+                       uint32_t test_ns, const float* __restrict__ sink, int chunk, float softcap, int maps,
+                       const float* __restrict__ bias, int bias_len) {
   // all shared memory is dynamic, so that the ring starts at the block's first byte (1024-byte
   // aligned, as the 128-byte swizzle needs)
   constexpr int STAGES = Shape<HD>::STAGES, STAGE_BYTES = Shape<HD>::STAGE_BYTES, BOXES = Shape<HD>::BOXES;
@@ -317,10 +321,25 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
       }
     }
   }
+  const float* bias_rows[2] = {bias, bias};
+  float far_bias[2] = {0.f, 0.f};
+  if (bias != nullptr) {  // (a column past the group's last head reads that head's numbers and is not stored)
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      bias_rows[j] += (size_t)(h0 + min(2 * t4 + j, n_heads - 1)) * bias_len;
+      far_bias[j] = bias_rows[j][bias_len - 1] * 1.4426950408889634f;
+    }
+  }
   bool ok = true;
   int done = 0;
   for (int tile = my_lo; tile <= my_hi && ok; ++tile, ++done) {
     const int st = done % STAGES;
+    float score_bias[4] = {far_bias[0], far_bias[1], far_bias[0], far_bias[1]};  // (key g [+8], head 2*t4 [+1]), base-2 exponents
+    if (bias != nullptr && pos - (tile * PAGE + warp * 16 + 15) < bias_len - 1) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        score_bias[e] = rl_distance_bias(bias_rows[e & 1], bias_len, pos - (tile * PAGE + warp * 16 + g + 8 * (e >> 1))) * 1.4426950408889634f;
+    }
     if (!mbar_wait_role(&bars.full[st], (done / STAGES) & 1, ctl, 52)) {
       if (lane == 0) {
         give_up_code(status, 52);
@@ -399,7 +418,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     float tmax[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      float v = rl_score_log2(s_acc[e], scale_log2, softcap);
+      float v = rl_score_log2(s_acc[e], scale_log2, softcap) + score_bias[e];
       if (need_mask) {
         const int key = key0 + g + 8 * (e >> 1);
         if (key < first || key > pos) v = -INFINITY;
@@ -588,7 +607,7 @@ static int launch_decode_tma(const void* q, int q_stride, const void* k_pages, c
                              int* status, int fuse, const float* inv_freq, int rot, int interleaved, unsigned int* counters,
                              const float* q_parts, int n_parts, long long part_stride, int wait_test_role,
                              unsigned int wait_test_ns, const float* sink, int chunk, float softcap, int maps, float pair_lambda, float pair_eps,
-                             float pair_factor, cudaStream_t stream) {
+                             float pair_factor, const float* bias, int bias_len, cudaStream_t stream) {
   CUtensorMap map_k, map_v;
   if (make_page_map(&map_k, k_pages, n_pages, K, PAGE, HD, PAGE) || make_page_map(&map_v, v_pages, n_pages, K, PAGE, HD, PAGE))
     RL_REFUSE(10, "attn_decode_tma: cannot describe the cache pages to TMA");
@@ -602,7 +621,7 @@ static int launch_decode_tma(const void* q, int q_stride, const void* k_pages, c
                             table_width, seq_len, part_o, part_ml, H, K, window, scale * 1.4426950408889634f, n_splits, status,
                             fuse, (bf16*)const_cast<void*>(k_pages), (bf16*)const_cast<void*>(v_pages), inv_freq, fuse ? rot : 0,
                             interleaved, counters, (bf16*)out, out_stride, q_parts, n_parts, part_stride, wait_test_role,
-                            (uint32_t)wait_test_ns, sink, chunk, softcap, maps));
+                            (uint32_t)wait_test_ns, sink, chunk, softcap, maps, bias, bias_len));
   if (maps == 2) {
     dim3 grid1(H / 2, n_seqs);
     RL_LAUNCH_CHECK(rl_launch(attn_decode_merge_pair_kernel, grid1, HD, 0, stream, (const float*)part_o, (const float*)part_ml, (bf16*)out,
@@ -622,7 +641,9 @@ RL_API int rl_attn_decode_tma(const void* q, int q_stride, const void* k_pages, 
                               float scale, int n_splits, int* status, int fuse, const float* inv_freq, int rot,
                               int interleaved, unsigned int* counters, const float* q_parts, int n_parts,
                               long long part_stride, int wait_test_role, unsigned int wait_test_ns, const float* sink,
-                              int chunk, float softcap, int maps, float pair_lambda, float pair_eps, float pair_factor, cudaStream_t stream) {
+                              int chunk, float softcap, int maps, float pair_lambda, float pair_eps, float pair_factor,
+                              const float* bias, int bias_len, cudaStream_t stream) {
+  if (bias != nullptr && bias_len <= 0) RL_REFUSE(16, "attn_decode_tma: a bias by distance of %d numbers a head", bias_len);
   if (maps < 1 || maps > 2 || H % maps || (maps == 2 && (counters != nullptr || rot != 0)))
     RL_REFUSE(15, "attn_decode_tma: %d maps in %d heads (two maps: no rotation, no counters)", maps, H);
   if (n_seqs <= 0 || H <= 0 || K <= 0 || n_pages <= 0) RL_REFUSE(1, "attn_decode_tma: S=%d H=%d K=%d pages=%d", n_seqs, H, K, n_pages);
@@ -643,7 +664,7 @@ RL_API int rl_attn_decode_tma(const void* q, int q_stride, const void* k_pages, 
   return launch_decode_tma<HDV>(q, q_stride, k_pages, v_pages, n_pages, block_table, table_width, seq_len, part_o, part_ml, out, \
                                 out_stride, n_seqs, H, K, window, scale, n_splits, status, fuse, inv_freq, rot, interleaved,      \
                                 counters, q_parts, n_parts, part_stride, wait_test_role, wait_test_ns, sink, chunk, softcap, maps, pair_lambda,    \
-                                pair_eps, pair_factor, stream)
+                                pair_eps, pair_factor, bias, bias_len, stream)
   if (hd == 64) RL_DECODE_TMA(64);
   RL_DECODE_TMA(128);
 #undef RL_DECODE_TMA

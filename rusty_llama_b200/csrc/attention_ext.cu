@@ -3,7 +3,12 @@
 //   - keys of `kdim` and values of `vdim` numbers per head (the two may differ),
 //   - biases on the projected q, k and v,
 //   - an RMS norm of every q head and every k head over the head's numbers (one weight row for all q heads, one for all k
-//     heads), after the biases and before the rotation,
+//     heads), after the biases and before the rotation; or one norm over all q heads together and one over all k heads together
+//     (`norm_whole`), with a weight for every column,
+//   - a temperature of the queries that grows with the position: q at position p is multiplied by
+//     1 + temp_coef ln(floor((p + 1) / temp_every) + 1), after the norm,
+//   - values that are the keys as projected, before their norm (`v_from_k`; the rows then hold no values),
+//   - a learned bias on every score by head and distance (`rl_distance_bias`), added after scale, mixing and cap,
 //   - a rotation of the first `rot` dimensions of q and k in either pair layout, cosines and sines
 //     multiplied by a constant `magnitude`,
 //   - a score scale given by the caller,
@@ -32,7 +37,11 @@
 
 RL_DEFINE_ERROR_TEXT()
 
-// ---------------------------------------------------------------- biases, rotation, cache write
+// ---------------------------------------------------------------- biases, norms, rotation, cache write
+__device__ __forceinline__ float qp_temperature(int pos, float coef, int every) {
+  return 1.0f + coef * logf((float)((pos + 1) / every) + 1.0f);
+}
+
 // One block per token.  row = qkv[t]: H query heads of kdim, then K key heads of kdim, then K value heads of vdim.
 template <typename T>
 __global__ void qkv_prep_kernel(T* __restrict__ qkv, int row_stride, const float* __restrict__ bias,
@@ -41,7 +50,8 @@ __global__ void qkv_prep_kernel(T* __restrict__ qkv, int row_stride, const float
                                 T* __restrict__ v_pages, const float* __restrict__ inv_freq, float magnitude,
                                 const float* __restrict__ q_norm, const float* __restrict__ k_norm, float norm_eps, int H, int K,
                                 int kdim, int vdim, int rot, int interleaved, int page_size, const T* __restrict__ v_src,
-                                int v_src_stride, const float* __restrict__ v_lambda) {
+                                int v_src_stride, const float* __restrict__ v_lambda, int norm_whole, int v_from_k, float temp_coef,
+                                int temp_every) {
   extern __shared__ float trig[];  // cos[rot/2], sin[rot/2], both times the magnitude; then 1 / rms of every q and k head
   const int t = blockIdx.x;
   const int pos = tok_pos[t];
@@ -68,11 +78,22 @@ __global__ void qkv_prep_kernel(T* __restrict__ qkv, int row_stride, const float
         ss += x * x;
       }
       ss = warp_sum(ss);
-      if (lane == 0) inv_rms[h] = ((h < H ? q_norm : k_norm) != nullptr) ? 1.0f / sqrtf(ss / (float)kdim + norm_eps) : 1.f;
+      if (lane == 0) inv_rms[h] = norm_whole ? ss : ((h < H ? q_norm : k_norm) != nullptr) ? 1.0f / sqrtf(ss / (float)kdim + norm_eps) : 1.f;
+    }
+    if (norm_whole) {  // one thread adds the q heads' sums in their order, another the k heads'
+      __syncthreads();
+      if (threadIdx.x < 2) {
+        const int lo = threadIdx.x == 0 ? 0 : H, hi = threadIdx.x == 0 ? H : H + K;
+        float ss = 0.f;
+        for (int h = lo; h < hi; ++h) ss += inv_rms[h];
+        const float inv = ((threadIdx.x == 0 ? q_norm : k_norm) != nullptr) ? 1.0f / sqrtf(ss / (float)((hi - lo) * kdim) + norm_eps) : 1.f;
+        for (int h = lo; h < hi; ++h) inv_rms[h] = inv;
+      }
     }
   }
   __syncthreads();
-  const int page = block_table[(size_t)tok_seq[t] * table_width + pos / page_size];
+  const float temp = temp_every > 0 ? qp_temperature(pos, temp_coef, temp_every) : 1.f;
+  const int page = K > 0 ? block_table[(size_t)tok_seq[t] * table_width + pos / page_size] : 0;
   const int in_page = pos % page_size;
   // q and k heads: one thread per rotated pair or per unrotated value
   const int per_head = half + (kdim - rot);
@@ -81,7 +102,9 @@ __global__ void qkv_prep_kernel(T* __restrict__ qkv, int row_stride, const float
     T* head = row + (size_t)h * kdim;
     const float* b = bias ? bias + (size_t)h * kdim : nullptr;
     const float* nw = h < H ? q_norm : k_norm;
+    if (nw && norm_whole) nw += (size_t)(h < H ? h : h - H) * kdim;
     const float inv = nw ? inv_rms[h] : 1.f;
+    const float by = h < H ? temp : 1.f;
     T* dst = h < H ? head : k_pages + (((size_t)page * K + (h - H)) * page_size + in_page) * kdim;
     if (e < half) {
       const int i0 = interleaved ? 2 * e : e;
@@ -92,16 +115,18 @@ __global__ void qkv_prep_kernel(T* __restrict__ qkv, int row_stride, const float
         x0 = x0 * inv * nw[i0];
         x1 = x1 * inv * nw[i1];
       }
+      x0 *= by;
+      x1 *= by;
       dst[i0] = from_f32<T>(x0 * cs[e] - x1 * sn[e]);
       dst[i1] = from_f32<T>(x1 * cs[e] + x0 * sn[e]);
     } else {
       const int i = rot + (e - half);
       float x = to_f32(head[i]) + (b ? b[i] : 0.f);
       if (nw) x = x * inv * nw[i];
-      dst[i] = from_f32<T>(x);
+      dst[i] = from_f32<T>(x * by);
     }
   }
-  const T* vrow = row + (size_t)(H + K) * kdim;
+  const T* vrow = row + (size_t)(v_from_k ? H : H + K) * kdim;
   const float* vb = bias ? bias + (size_t)(H + K) * kdim : nullptr;
   const float lam = v_src ? v_lambda[0] : 0.f;
   const T* vs = v_src ? v_src + (size_t)t * v_src_stride : nullptr;
@@ -114,8 +139,8 @@ __global__ void qkv_prep_kernel(T* __restrict__ qkv, int row_stride, const float
 }
 
 // The same for bfloat16 rows whose sizes are multiples of 8 and whose pairs are neighbours (or that are not rotated at all): a
-// thread takes 8 numbers of a head with one 16-byte load, the kdim / 8 threads of a head add their squares up by shuffles, and
-// the four pairs a thread holds are rotated in its registers; q goes back and k, v go to their pages with 16-byte stores.
+// thread takes 8 numbers of a head with one 16-byte load, the kdim / 8 threads of a head (in a run of a power of two of lanes, the
+// rest of which idle) add their squares up by shuffles, a norm over all heads by a pass over the row before that, and the four pairs a thread holds are rotated in its registers; q goes back and k, v go to their pages with 16-byte stores.
 __device__ __forceinline__ void qp_unpack8(const uint4& raw, float* x) {
   const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw);
 #pragma unroll
@@ -146,7 +171,8 @@ qkv_prep_rows8_kernel(bf16* __restrict__ qkv, int row_stride, const float* __res
                       bf16* __restrict__ k_pages, bf16* __restrict__ v_pages, const float* __restrict__ inv_freq, float magnitude,
                       const float* __restrict__ q_norm, const float* __restrict__ k_norm, float norm_eps, int H, int K, int kdim,
                       int vdim, int rot, int page_size, const bf16* __restrict__ v_src, int v_src_stride,
-                      const float* __restrict__ v_lambda) {
+                      const float* __restrict__ v_lambda, int g, int norm_whole, int v_from_k, float temp_coef, int temp_every) {
+  __shared__ float red[32];
   extern __shared__ float trig[];  // cos[rot/2], sin[rot/2], both times the magnitude
   const int t = blockIdx.x;
   const int pos = tok_pos[t];
@@ -162,15 +188,32 @@ qkv_prep_rows8_kernel(bf16* __restrict__ qkv, int row_stride, const float* __res
   }
   __syncthreads();
   bf16* row = qkv + (size_t)t * row_stride;
-  const int page = block_table[(size_t)tok_seq[t] * table_width + pos / page_size];
+  const int page = K > 0 ? block_table[(size_t)tok_seq[t] * table_width + pos / page_size] : 0;
   const int in_page = pos % page_size;
-  const int g = kdim >> 3;  // threads to a head: a power of two up to 32
-  const int total = (H + K) * g;
-  const bool normed = q_norm != nullptr || k_norm != nullptr;
+  const int total = (H + K) * g;  // g: lanes to a head, the power of two from kdim / 8 on, up to 32
+  const bool normed = (q_norm != nullptr || k_norm != nullptr) && !norm_whole;
+  const float temp = temp_every > 0 ? qp_temperature(pos, temp_coef, temp_every) : 1.f;
+  float whole_q = 1.f, whole_k = 1.f;  // 1 / rms of all q heads, of all k heads
+  if (norm_whole) {
+    float own_q = 0.f, own_k = 0.f;
+    const int nq = (H * kdim) >> 3, n8 = ((H + K) * kdim) >> 3;
+    for (int c = threadIdx.x; c < n8; c += blockDim.x) {
+      float x[8], sum = 0.f;
+      qp_unpack8(*reinterpret_cast<const uint4*>(row + (size_t)c * 8), x);
+      if (bias) qp_add8(x, bias + (size_t)c * 8);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) sum += x[j] * x[j];
+      if (c < nq) own_q += sum;
+      else own_k += sum;
+    }
+    const float sq = block_sum(own_q, red), sk = block_sum(own_k, red);
+    if (q_norm) whole_q = 1.0f / sqrtf(sq / (float)(H * kdim) + norm_eps);
+    if (k_norm && K > 0) whole_k = 1.0f / sqrtf(sk / (float)(K * kdim) + norm_eps);
+  }
   for (int base = 0; base < total; base += blockDim.x) {
     const int idx = base + threadIdx.x;
-    const bool valid = idx < total;  // (a head's threads are all valid or all not; every lane takes part in the shuffles)
-    const int h = valid ? idx / g : 0, i0 = valid ? (idx - h * g) * 8 : 0;
+    const bool valid = idx < total && (idx & (g - 1)) * 8 < kdim;  // (every lane takes part in the shuffles)
+    const int h = valid ? idx / g : 0, i0 = valid ? (idx & (g - 1)) * 8 : 0;
     float x[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
     if (valid) {
       qp_unpack8(*reinterpret_cast<const uint4*>(row + (size_t)h * kdim + i0), x);
@@ -189,6 +232,19 @@ qkv_prep_rows8_kernel(bf16* __restrict__ qkv, int row_stride, const float* __res
         x[4] = x[4] * inv * w1.x; x[5] = x[5] * inv * w1.y; x[6] = x[6] * inv * w1.z; x[7] = x[7] * inv * w1.w;
       }
     }
+    if (norm_whole && valid) {
+      const float* nw = h < H ? (q_norm ? q_norm + (size_t)h * kdim + i0 : nullptr) : (k_norm ? k_norm + (size_t)(h - H) * kdim + i0 : nullptr);
+      if (nw) {
+        const float inv = h < H ? whole_q : whole_k;
+        const float4 w0 = *reinterpret_cast<const float4*>(nw), w1 = *reinterpret_cast<const float4*>(nw + 4);
+        x[0] = x[0] * inv * w0.x; x[1] = x[1] * inv * w0.y; x[2] = x[2] * inv * w0.z; x[3] = x[3] * inv * w0.w;
+        x[4] = x[4] * inv * w1.x; x[5] = x[5] * inv * w1.y; x[6] = x[6] * inv * w1.z; x[7] = x[7] * inv * w1.w;
+      }
+    }
+    if (temp_every > 0 && h < H) {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) x[j] *= temp;
+    }
     if (valid) {
       if (i0 < rot) {
 #pragma unroll
@@ -203,7 +259,7 @@ qkv_prep_rows8_kernel(bf16* __restrict__ qkv, int row_stride, const float* __res
       *reinterpret_cast<uint4*>(dst) = qp_pack8(x);
     }
   }
-  const bf16* vrow = row + (size_t)(H + K) * kdim;
+  const bf16* vrow = row + (size_t)(v_from_k ? H : H + K) * kdim;
   const float* vb = bias ? bias + (size_t)(H + K) * kdim : nullptr;
   const int gv = vdim >> 3;
   for (int idx = threadIdx.x; idx < K * gv; idx += blockDim.x) {
@@ -230,33 +286,39 @@ RL_API int rl_qkv_prep(void* qkv, int dtype, int row_stride, const float* bias, 
                        const int* block_table, int table_width, void* k_pages, void* v_pages, const float* inv_freq,
                        float magnitude, const float* q_norm, const float* k_norm, float norm_eps, int n_tokens, int H, int K, int kdim,
                        int vdim, int rot, int interleaved, int page_size, const void* v_src, int v_src_stride, const float* v_lambda,
-                       cudaStream_t stream) {
+                       int norm_whole, int v_from_k, float temp_coef, int temp_every, cudaStream_t stream) {
+  if (v_from_k && (vdim != kdim || v_src != nullptr || bias != nullptr)) RL_REFUSE(9, "qkv_prep: values that are the keys are as long (%d, %d), with no bias and no mixing", kdim, vdim);
+  if (temp_every < 0) RL_REFUSE(10, "qkv_prep: temperature steps of %d positions", temp_every);
   if (v_src != nullptr && (v_lambda == nullptr || v_src_stride < K * vdim)) RL_REFUSE(8, "qkv_prep: values to mix in need a factor and rows of %d numbers", K * vdim);
-  if (n_tokens <= 0 || H < 0 || K <= 0 || kdim <= 0 || vdim <= 0 || page_size <= 0 || table_width <= 0)  // (H 0: rows that hold keys and values only)
+  if (n_tokens <= 0 || H < 0 || K < 0 || H + K <= 0 || kdim <= 0 || vdim <= 0 || page_size <= 0 || table_width <= 0)  // (H 0: rows of keys and values only; K 0: of queries)
     RL_REFUSE(1, "qkv_prep: T=%d H=%d K=%d kdim=%d vdim=%d page=%d", n_tokens, H, K, kdim, vdim, page_size);
   if (rot < 0 || rot > kdim || (rot & 1)) RL_REFUSE(2, "qkv_prep: %d rotated dimensions do not fit a head of %d", rot, kdim);
-  if (row_stride < (H + K) * kdim + K * vdim) RL_REFUSE(3, "qkv_prep: row stride %d too small", row_stride);
+  if (row_stride < (H + K) * kdim + (v_from_k ? 0 : K * vdim)) RL_REFUSE(3, "qkv_prep: row stride %d too small", row_stride);
   if (rot > 0 && inv_freq == nullptr) RL_REFUSE(4, "qkv_prep: no frequency table");
-  if (!block_table || !k_pages || !v_pages || !tok_pos || !tok_seq) RL_REFUSE(5, "qkv_prep: pages, page table and positions are needed");
+  if (!tok_pos || !tok_seq || (K > 0 && (!block_table || !k_pages || !v_pages))) RL_REFUSE(5, "qkv_prep: pages, page table and positions are needed");
   const size_t smem = ((size_t)rot + H + K) * sizeof(float);
   if (smem > 48 * 1024) RL_REFUSE(6, "qkv_prep: rotary size %d or %d heads too large", rot, H + K);
   const int threads = 256;
-  const int g = kdim >> 3;
+  int g = 1;
+  while (g * 8 < kdim) g *= 2;
   const uintptr_t bits = (uintptr_t)qkv | (uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)bias | (uintptr_t)q_norm | (uintptr_t)k_norm |
                          (uintptr_t)v_src;
   if (dtype == RL_BF16 && (interleaved || rot == 0) && kdim % 8 == 0 && vdim % 8 == 0 && rot % 8 == 0 && row_stride % 8 == 0 &&
-      v_src_stride % 8 == 0 && g <= 32 && (g & (g - 1)) == 0 && (bits & 15) == 0)
+      v_src_stride % 8 == 0 && g <= 32 && (bits & 15) == 0)
     qkv_prep_rows8_kernel<<<n_tokens, threads, (size_t)rot * sizeof(float), stream>>>(
         (bf16*)qkv, row_stride, bias, tok_pos, tok_seq, block_table, table_width, (bf16*)k_pages, (bf16*)v_pages, inv_freq, magnitude,
-        q_norm, k_norm, norm_eps, H, K, kdim, vdim, rot, page_size, (const bf16*)v_src, v_src_stride, v_lambda);
+        q_norm, k_norm, norm_eps, H, K, kdim, vdim, rot, page_size, (const bf16*)v_src, v_src_stride, v_lambda,
+        g, norm_whole, v_from_k, temp_coef, temp_every);
   else if (dtype == RL_BF16)
     qkv_prep_kernel<bf16><<<n_tokens, threads, smem, stream>>>((bf16*)qkv, row_stride, bias, tok_pos, tok_seq, block_table, table_width,
                                                                (bf16*)k_pages, (bf16*)v_pages, inv_freq, magnitude, q_norm, k_norm, norm_eps, H, K,
-                                                               kdim, vdim, rot, interleaved, page_size, (const bf16*)v_src, v_src_stride, v_lambda);
+                                                               kdim, vdim, rot, interleaved, page_size, (const bf16*)v_src, v_src_stride, v_lambda,
+                                                               norm_whole, v_from_k, temp_coef, temp_every);
   else if (dtype == RL_F32)
     qkv_prep_kernel<float><<<n_tokens, threads, smem, stream>>>((float*)qkv, row_stride, bias, tok_pos, tok_seq, block_table, table_width,
                                                                 (float*)k_pages, (float*)v_pages, inv_freq, magnitude, q_norm, k_norm, norm_eps, H, K,
-                                                                kdim, vdim, rot, interleaved, page_size, (const float*)v_src, v_src_stride, v_lambda);
+                                                                kdim, vdim, rot, interleaved, page_size, (const float*)v_src, v_src_stride, v_lambda,
+                                                                norm_whole, v_from_k, temp_coef, temp_every);
   else
     RL_REFUSE(7, "qkv_prep: unknown dtype %d", dtype);
   RL_LAUNCH_RESULT();
@@ -271,7 +333,8 @@ __global__ void attn_ext_kernel(const T* __restrict__ q, int q_stride, const T* 
                                 const int* __restrict__ block_table, int table_width, const int* __restrict__ tok_seq,
                                 const int* __restrict__ tok_pos, const float* __restrict__ sink, const float* __restrict__ mix,
                                 const T* __restrict__ gate, int gate_stride, float out_scale, T* __restrict__ out, int out_stride,
-                                int H, int K, int kdim, int vdim, int page_size, int window, float scale, int chunk, float softcap, int maps) {
+                                int H, int K, int kdim, int vdim, int page_size, int window, float scale, int chunk, float softcap, int maps,
+                                const float* __restrict__ bias, int bias_len) {
   extern __shared__ float smem[];  // q of the block's heads [HB][kdim], then (with mix) scores [HB][32]
   const int lane = threadIdx.x;
   const int hb = threadIdx.y, HB = blockDim.y;
@@ -317,6 +380,7 @@ __global__ void attn_ext_kernel(const T* __restrict__ q, int q_stride, const T* 
       s = mixed;
     }
     if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+    if (bias != nullptr) s += rl_distance_bias(bias + (size_t)h * bias_len, bias_len, pos - key);
     if (!valid) s = -INFINITY;
     const float m_new = fmaxf(m, warp_max(s));  // finite: the group holds at least key `base`
     const float alpha = expf(m - m_new);        // 0 for the first group without a sink, where m is -inf
@@ -355,7 +419,9 @@ __global__ void attn_ext_kernel(const T* __restrict__ q, int q_stride, const T* 
 RL_API int rl_attn_ext(const void* q, int dtype, int q_stride, const void* k_pages, const void* v_pages, const int* block_table,
                        int table_width, const int* tok_seq, const int* tok_pos, const float* sink, const float* mix,
                        const void* gate, int gate_stride, float out_scale, void* out, int out_stride, int n_tokens, int H, int K,
-                       int kdim, int vdim, int page_size, int window, float scale, int chunk, float softcap, int maps, cudaStream_t stream) {
+                       int kdim, int vdim, int page_size, int window, float scale, int chunk, float softcap, int maps,
+                       const float* bias, int bias_len, cudaStream_t stream) {
+  if (bias != nullptr && bias_len <= 0) RL_REFUSE(10, "attn_ext: a bias by distance of %d numbers a head", bias_len);
   if (maps < 1 || maps > 2 || H % maps || kdim % maps || (maps > 1 && mix != nullptr)) RL_REFUSE(9, "attn_ext: %d maps in %d heads of %d numbers%s", maps, H, kdim, mix ? " whose scores are mixed" : "");
   if (n_tokens <= 0 || H <= 0 || K <= 0 || kdim <= 0 || vdim <= 0 || page_size <= 0)
     RL_REFUSE(1, "attn_ext: T=%d H=%d K=%d kdim=%d vdim=%d page=%d", n_tokens, H, K, kdim, vdim, page_size);
@@ -372,12 +438,12 @@ RL_API int rl_attn_ext(const void* q, int dtype, int q_stride, const void* k_pag
     attn_ext_kernel<bf16><<<grid, block, smem, stream>>>((const bf16*)q, q_stride, (const bf16*)k_pages, (const bf16*)v_pages,
                                                          block_table, table_width, tok_seq, tok_pos, sink, mix, (const bf16*)gate,
                                                          gate_stride, out_scale, (bf16*)out, out_stride, H, K, kdim, vdim, page_size,
-                                                         window, scale, chunk, softcap, maps);
+                                                         window, scale, chunk, softcap, maps, bias, bias_len);
   else if (dtype == RL_F32)
     attn_ext_kernel<float><<<grid, block, smem, stream>>>((const float*)q, q_stride, (const float*)k_pages, (const float*)v_pages,
                                                           block_table, table_width, tok_seq, tok_pos, sink, mix, (const float*)gate,
                                                           gate_stride, out_scale, (float*)out, out_stride, H, K, kdim, vdim, page_size,
-                                                          window, scale, chunk, softcap, maps);
+                                                          window, scale, chunk, softcap, maps, bias, bias_len);
   else
     RL_REFUSE(8, "attn_ext: unknown dtype %d", dtype);
   RL_LAUNCH_RESULT();

@@ -11,7 +11,9 @@
 // A block of four warps owns 64 query rows of one head of one sequence (eight warps and 128 rows for folded queries of a
 // prompt, whose many parts in shared memory leave room for one block per SM only).  A key tile is one cache page.  The loads of a tile
 // are, in order, the keys of each part and then the values; they go through a ring of three buffers with cp.async, two loads
-// ahead of the one in use.  The online softmax (max, sum, rescale) is 32-bit, in base-2 exponents.  Sizes are padded with
+// ahead of the one in use.  The online softmax (max, sum, rescale) is 32-bit, in base-2 exponents.  A learned bias by head and
+// distance (`rl_distance_bias`) is added to the scores; a tile that lies wholly beyond the last distance with a number of its own
+// adds one number.  Sizes are padded with
 // zeros to HD in shared memory, so key and value sizes in multiples of 8 up to 256 are served.  Prompts and single tokens
 // alike: a decode step is a batch of sequences with one query row each.
 #include "common.cuh"
@@ -128,7 +130,8 @@ flash_mix_kernel(const bf16* __restrict__ q, long long q_row_stride, int q_head_
                  const bf16* __restrict__ v_pages, const int* __restrict__ block_table, int table_width,
                  const int* __restrict__ seq_start, const int* __restrict__ seq_pos0, const float* __restrict__ sink,
                  const bf16* __restrict__ gate, int gate_stride, float out_scale, bf16* __restrict__ out, int out_stride, int H, int K,
-                 int kdim, int vdim, int window, float scale_log2, int chunk, float softcap, int maps) {
+                 int kdim, int vdim, int window, float scale_log2, int chunk, float softcap, int maps, const float* __restrict__ bias,
+                 int bias_len) {
   constexpr int STRIDE = HD + 8;  // 16 bytes of padding per row keep ldmatrix free of bank conflicts
   constexpr int KSTEPS = HD / 16;
   constexpr int NTHREADS = BM * 2;  // a warp per 16 query rows
@@ -198,6 +201,7 @@ flash_mix_kernel(const bf16* __restrict__ q, long long q_row_stride, int q_head_
   const int qpos[2] = {first_pos + warp * 16 + g, first_pos + warp * 16 + g + 8};
   const int qlow[2] = {rl_first_key(qpos[0], window, chunk), rl_first_key(qpos[1], window, chunk)};
   float s_acc[BN / 8][4];
+  const float* bias_row = bias != nullptr ? bias + (size_t)h * bias_len : nullptr;
 
   for (int n = 0; n < n_loads; ++n) {
     if (n + 2 < n_loads) issue(n + 2);
@@ -229,6 +233,8 @@ flash_mix_kernel(const bf16* __restrict__ q, long long q_row_stride, int q_head_
       // ---- mask, scale (to base-2 exponents) and the online softmax
       const int key0 = tile * BN;
       float tile_max[2] = {-INFINITY, -INFINITY};
+      const bool near = bias_row != nullptr && first_pos - (key0 + BN - 1) < bias_len - 1;
+      const float far_bias = bias_row != nullptr ? bias_row[bias_len - 1] * 1.4426950408889634f : 0.f;
 #pragma unroll
       for (int nn = 0; nn < BN / 8; ++nn) {
 #pragma unroll
@@ -236,6 +242,7 @@ flash_mix_kernel(const bf16* __restrict__ q, long long q_row_stride, int q_head_
           const int r = e >> 1;
           float v = rl_score_log2(s_acc[nn][e], scale_log2, softcap);
           const int key = key0 + nn * 8 + 2 * t4 + (e & 1);
+          v += near ? rl_distance_bias(bias_row, bias_len, qpos[r] - key) * 1.4426950408889634f : far_bias;
           const bool seen = key <= qpos[r] && key >= qlow[r];
           if (!seen) v = -INFINITY;
           s_acc[nn][e] = v;
@@ -323,7 +330,7 @@ template <int HD, int BM>
 static int launch_mix_rows(const bf16* q, long long q_row_stride, int q_head_stride, int parts, const bf16* k_pages, const bf16* v_pages,
                       const int* block_table, int table_width, const int* seq_start, const int* seq_pos0, const float* sink,
                       const bf16* gate, int gate_stride, float out_scale, bf16* out, int out_stride, int n_seqs, int max_q_len, int H, int K,
-                      int kdim, int vdim, int window, float scale, int chunk, float softcap, int maps, cudaStream_t stream) {
+                      int kdim, int vdim, int window, float scale, int chunk, float softcap, int maps, const float* bias, int bias_len, cudaStream_t stream) {
   const size_t smem = (size_t)(NBUF * BN + parts * BM) * (HD + 8) * sizeof(bf16);
   auto kern = flash_mix_kernel<HD, BM>;
   if (smem > 227 * 1024) RL_REFUSE(8, "flash_mix: %zu bytes of shared memory for %d query parts exceed the SM's", smem, parts);
@@ -334,7 +341,7 @@ static int launch_mix_rows(const bf16* q, long long q_row_stride, int q_head_str
   dim3 grid(H * n_seqs, (max_q_len + BM - 1) / BM);
   kern<<<grid, BM * 2, smem, stream>>>(q, q_row_stride, q_head_stride, parts, k_pages, v_pages, block_table, table_width, seq_start,
                                          seq_pos0, sink, gate, gate_stride, out_scale, out, out_stride, H, K, kdim, vdim, window,
-                                         scale * 1.4426950408889634f, chunk, softcap, maps);
+                                         scale * 1.4426950408889634f, chunk, softcap, maps, bias, bias_len);
   RL_LAUNCH_RESULT();
 }
 
@@ -342,7 +349,7 @@ template <int HD>
 static int launch_mix(const bf16* q, long long q_row_stride, int q_head_stride, int parts, const bf16* k_pages, const bf16* v_pages,
                       const int* block_table, int table_width, const int* seq_start, const int* seq_pos0, const float* sink,
                       const bf16* gate, int gate_stride, float out_scale, bf16* out, int out_stride, int n_seqs, int max_q_len, int H, int K,
-                      int kdim, int vdim, int window, float scale, int chunk, float softcap, int maps, cudaStream_t stream) {
+                      int kdim, int vdim, int window, float scale, int chunk, float softcap, int maps, const float* bias, int bias_len, cudaStream_t stream) {
   // 128 rows to a block where several query parts would leave one block of 64 rows alone on its SM anyway and the step has
   // the rows to fill it
   const size_t smem128 = (size_t)(NBUF * BN + parts * 128) * (HD + 8) * sizeof(bf16);
@@ -350,9 +357,9 @@ static int launch_mix(const bf16* q, long long q_row_stride, int q_head_stride, 
   if (HD <= 128 && parts > 1 && max_q_len > 64 && smem128 <= 227 * 1024 && 2 * smem64 > 227 * 1024)
     return launch_mix_rows<HD, 128>(q, q_row_stride, q_head_stride, parts, k_pages, v_pages, block_table, table_width, seq_start, seq_pos0,
                                     sink, gate, gate_stride, out_scale, out, out_stride, n_seqs, max_q_len, H, K, kdim, vdim, window, scale,
-                                    chunk, softcap, maps, stream);
+                                    chunk, softcap, maps, bias, bias_len, stream);
   return launch_mix_rows<HD, 64>(q, q_row_stride, q_head_stride, parts, k_pages, v_pages, block_table, table_width, seq_start, seq_pos0, sink,
-                                 gate, gate_stride, out_scale, out, out_stride, n_seqs, max_q_len, H, K, kdim, vdim, window, scale, chunk, softcap, maps, stream);
+                                 gate, gate_stride, out_scale, out, out_stride, n_seqs, max_q_len, H, K, kdim, vdim, window, scale, chunk, softcap, maps, bias, bias_len, stream);
 }
 
 // q: the queries [T][..], row stride q_row_stride, head h at h * q_head_stride, part p of a head at + p * kdim.
@@ -361,7 +368,9 @@ static int launch_mix(const bf16* q, long long q_row_stride, int q_head_stride, 
 RL_API int rl_flash_mix(const void* q, long long q_row_stride, int q_head_stride, int parts, const void* k_pages, const void* v_pages,
                         const int* block_table, int table_width, const int* seq_start, const int* seq_pos0, const float* sink,
                         const void* gate, int gate_stride, float out_scale, void* out, int out_stride, int n_seqs, int max_q_len, int H,
-                        int K, int kdim, int vdim, int page_size, int window, float scale, int chunk, float softcap, int maps, cudaStream_t stream) {
+                        int K, int kdim, int vdim, int page_size, int window, float scale, int chunk, float softcap, int maps, const float* bias,
+                        int bias_len, cudaStream_t stream) {
+  if (bias != nullptr && bias_len <= 0) RL_REFUSE(11, "flash_mix: a bias by distance of %d numbers a head", bias_len);
   if (maps < 1 || maps > 2 || H % maps || kdim % (8 * maps) || (maps > 1 && parts > 1)) RL_REFUSE(10, "flash_mix: %d maps in %d heads of %d numbers", maps, H, kdim);
   if (n_seqs <= 0 || max_q_len <= 0 || H <= 0 || K <= 0 || kdim <= 0 || vdim <= 0)
     RL_REFUSE(1, "flash_mix: S=%d max_q=%d H=%d K=%d kdim=%d vdim=%d", n_seqs, max_q_len, H, K, kdim, vdim);
@@ -378,7 +387,7 @@ RL_API int rl_flash_mix(const void* q, long long q_row_stride, int q_head_stride
 #define RL_MIX(HDV)                                                                                                                   \
   return launch_mix<HDV>((const bf16*)q, q_row_stride, q_head_stride, parts, (const bf16*)k_pages, (const bf16*)v_pages, block_table,  \
                          table_width, seq_start, seq_pos0, sink, (const bf16*)gate, gate_stride, out_scale, (bf16*)out, out_stride,      \
-                         n_seqs, max_q_len, H, K, kdim, vdim, window, scale, chunk, softcap, maps, stream)
+                         n_seqs, max_q_len, H, K, kdim, vdim, window, scale, chunk, softcap, maps, bias, bias_len, stream)
   if (hd <= 32) RL_MIX(32);
   if (hd <= 64) RL_MIX(64);
   if (hd <= 128) RL_MIX(128);
@@ -398,7 +407,8 @@ template <int HD>
 __global__ void flash_mix_decode_kernel(const bf16* __restrict__ qf, const bf16* __restrict__ k_pages, const bf16* __restrict__ v_pages,
                                         const int* __restrict__ block_table, int table_width, const int* __restrict__ seq_pos0,
                                         const float* __restrict__ sink, float* __restrict__ part_o, float* __restrict__ part_ml, int H,
-                                        int K, int kdim, int vdim, int window, float scale_log2, int n_splits, int chunk, float softcap) {
+                                        int K, int kdim, int vdim, int window, float scale_log2, int n_splits, int chunk, float softcap,
+                                        const float* __restrict__ bias, int bias_len) {
   constexpr int STRIDE = HD + 8;
   constexpr int KSTEPS = HD / 16;
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -469,6 +479,15 @@ __global__ void flash_mix_decode_kernel(const bf16* __restrict__ qf, const bf16*
     // kv heads that this warp's sixteen rows read
     const int c_first = (warp * 16) / rep, c_last = min(H - 1, warp * 16 + 15) / rep;
     const int kv_lo = r_lo / rep, kv_hi = r_hi / rep;
+    // the bias rows of this thread's two heads (a row past the last head reads the last one's and is not stored)
+    const float* bias_rows[2] = {bias, bias};
+    float far_bias[2] = {0.f, 0.f};
+    if (bias != nullptr) {
+      bias_rows[0] += (size_t)min(r_lo, H - 1) * bias_len;
+      bias_rows[1] += (size_t)min(r_hi, H - 1) * bias_len;
+      far_bias[0] = bias_rows[0][bias_len - 1] * 1.4426950408889634f;
+      far_bias[1] = bias_rows[1][bias_len - 1] * 1.4426950408889634f;
+    }
     for (int n = 0; n < n_loads; ++n) {
       if (n + 2 < n_loads) issue(n + 2);
       cp_async_commit();
@@ -500,12 +519,14 @@ __global__ void flash_mix_decode_kernel(const bf16* __restrict__ qf, const bf16*
           // ---- the tile's scores are complete: mask, scale and the online softmax, once per tile
           const int key0 = tile * BN;
           float tile_max[2] = {-INFINITY, -INFINITY};
+          const bool near = bias != nullptr && pos - (key0 + BN - 1) < bias_len - 1;
 #pragma unroll
           for (int nn = 0; nn < BN / 8; ++nn) {
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
               const int key = key0 + nn * 8 + 2 * t4 + (e & 1);
               float v = rl_score_log2(s_acc[nn][e], scale_log2, softcap);
+              v += near ? rl_distance_bias(bias_rows[e >> 1], bias_len, pos - key) * 1.4426950408889634f : far_bias[e >> 1];
               if (key > pos || key < first) v = -INFINITY;
               s_acc[nn][e] = v;
               tile_max[e >> 1] = fmaxf(tile_max[e >> 1], v);
@@ -619,7 +640,7 @@ template <int HD>
 static int launch_mix_decode(const bf16* qf, const bf16* k_pages, const bf16* v_pages, const int* block_table, int table_width,
                              const int* seq_pos0, const float* sink, const bf16* gate, int gate_stride, float out_scale, float* part_o,
                              float* part_ml, bf16* out, int out_stride, int n_seqs, int H, int K, int kdim, int vdim, int window, float scale,
-                             int n_splits, int chunk, float softcap, cudaStream_t stream) {
+                             int n_splits, int chunk, float softcap, const float* bias, int bias_len, cudaStream_t stream) {
   const int warps = (H + 15) / 16;
   const size_t smem = (size_t)(NBUF * BN + K * warps * 16) * (HD + 8) * sizeof(bf16);
   auto kern = flash_mix_decode_kernel<HD>;
@@ -628,7 +649,7 @@ static int launch_mix_decode(const bf16* qf, const bf16* k_pages, const bf16* v_
     RL_REFUSE(8, "flash_mix_decode: cannot get %zu bytes of shared memory", smem);
   dim3 grid(n_splits, n_seqs);
   kern<<<grid, warps * 32, smem, stream>>>(qf, k_pages, v_pages, block_table, table_width, seq_pos0, sink, part_o, part_ml, H, K, kdim, vdim,
-                                           window, scale * 1.4426950408889634f, n_splits, chunk, softcap);
+                                           window, scale * 1.4426950408889634f, n_splits, chunk, softcap, bias, bias_len);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) {
     snprintf(rl_error_buf, sizeof(rl_error_buf), "%s", cudaGetErrorString(e));
@@ -649,7 +670,8 @@ RL_API int rl_flash_mix_decode_smem(int H, int K, int hd_max) {
 RL_API int rl_flash_mix_decode(const void* qf, const void* k_pages, const void* v_pages, const int* block_table, int table_width,
                                const int* seq_pos0, const float* sink, const void* gate, int gate_stride, float out_scale, float* part_o,
                                float* part_ml, void* out, int out_stride, int n_seqs, int H, int K, int kdim, int vdim, int page_size,
-                               int window, float scale, int n_splits, int chunk, float softcap, cudaStream_t stream) {
+                               int window, float scale, int n_splits, int chunk, float softcap, const float* bias, int bias_len, cudaStream_t stream) {
+  if (bias != nullptr && bias_len <= 0) RL_REFUSE(10, "flash_mix_decode: a bias by distance of %d numbers a head", bias_len);
   if (n_seqs <= 0 || H <= 0 || K <= 0 || kdim <= 0 || vdim <= 0 || n_splits <= 0 || !part_o || !part_ml)
     RL_REFUSE(1, "flash_mix_decode: S=%d H=%d K=%d kdim=%d vdim=%d splits=%d", n_seqs, H, K, kdim, vdim, n_splits);
   if (H % K || H > 256) RL_REFUSE(2, "flash_mix_decode: %d heads on %d kv heads (at most 256 heads)", H, K);
@@ -662,7 +684,7 @@ RL_API int rl_flash_mix_decode(const void* qf, const void* k_pages, const void* 
 #define RL_MIXD(HDV)                                                                                                                    \
   return launch_mix_decode<HDV>((const bf16*)qf, (const bf16*)k_pages, (const bf16*)v_pages, block_table, table_width, seq_pos0, sink,    \
                                 (const bf16*)gate, gate_stride, out_scale, part_o, part_ml, (bf16*)out, out_stride, n_seqs, H, K, kdim,    \
-                                vdim, window, scale, n_splits, chunk, softcap, stream)
+                                vdim, window, scale, n_splits, chunk, softcap, bias, bias_len, stream)
   if (hd <= 32) RL_MIXD(32);
   if (hd <= 64) RL_MIXD(64);
   if (hd <= 128) RL_MIXD(128);

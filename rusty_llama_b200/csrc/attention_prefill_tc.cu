@@ -51,6 +51,10 @@
 // tokens has too few blocks for two per SM and pays for the short tiles: 12.3 us against 10.5.
 // Softmax statistics, the accumulator and the final division are 32-bit.
 //
+// A learned bias by head and distance (`rl_distance_bias`): the head's numbers lie in shared memory (times log2 e; in global
+// memory where they do not fit beside the tiles), neighbouring rows of a tile read neighbouring ones.  A tile that lies wholly
+// beyond the last distance with a number of its own adds one number to every score, which goes into the exponent's constant.
+//
 // Every mbarrier wait is bounded; on expiry a code goes to status[0] and the block drains.
 #include "tc_common.cuh"
 
@@ -68,6 +72,7 @@ RL_DEFINE_ERROR_TEXT()
 #define O_COL 128
 #define RESCALE_THRESHOLD 8.0f          // in base-2 exponents
 #define SMALL_BYTES 512
+#define BIAS_SMEM_FLOATS(HD) ((113 * 1024 - SMEM_NEEDED(HD)) / 4)  // what is left of half an SM's shared memory
 // Q is HD / 64 sub-tiles of 16 KB; a K or V tile HD / 64 sub-tiles of 8 KB.  Two blocks must fit an SM and
 // no more (a third would wait for tensor memory): at head size 64 the request is padded to that end.
 #define SMEM_NEEDED(HD) ((HD) / 64 * SUBQ_BYTES + 2 * KV_STAGES * ((HD) / 64) * SUBK_BYTES + SMALL_BYTES)
@@ -216,13 +221,14 @@ __device__ __forceinline__ uint32_t pv_block(uint32_t tmem_o, uint32_t tmem_p, u
 
 // MAPS 2: query heads 2h and 2h + 1 are the two halves of the HD numbers of row h (the values are the same for both); the row's
 // tile is loaded whole and a block's scores use its half of it and of the keys.
-template <int HD, int MAPS>
+template <int HD, int MAPS, bool BIAS>
 __global__ void __launch_bounds__(NUM_THREADS, 2)
 flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                         const __grid_constant__ CUtensorMap map_v, const int* __restrict__ block_table, int table_width,
                         const int* __restrict__ seq_start, const int* __restrict__ seq_pos0, bf16* __restrict__ out,
                         int out_stride, int H, int K, int window, float scale_log2, int* __restrict__ status,
-                        int test_role, uint32_t test_ns, const float* __restrict__ sink, int chunk, float softcap) {
+                        int test_role, uint32_t test_ns, const float* __restrict__ sink, int chunk, float softcap,
+                        const float* __restrict__ bias, int bias_len, int bias_in_smem) {
   // All shared memory is dynamic, so that the tiles start at the block's first byte (1024-byte
   // aligned, as the 128-byte swizzle needs) and the small items fit behind them.
   constexpr int SUBS = HD / 64, Q_BYTES = SUBS * SUBQ_BYTES, KV_BYTES = SUBS * SUBK_BYTES;
@@ -263,6 +269,12 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   const int lowest_key = rl_first_key(first_pos, window, chunk);
   const int tile_lo = lowest_key / BNK, tile_hi = last_pos / BNK;
   const int n_tiles = tile_hi - tile_lo + 1;
+  const float* bias_row = BIAS ? bias + (size_t)h * bias_len : nullptr;
+  if (BIAS && bias_in_smem) {
+    float* b = reinterpret_cast<float*>(smem_dyn + SMEM_NEEDED(HD));
+    for (int i = threadIdx.x; i < bias_len; i += NUM_THREADS) b[i] = bias_row[i];
+    bias_row = b;
+  }
 
   if (threadIdx.x == 0) {
     mbar_init(&q_full, 1);
@@ -405,6 +417,8 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     const int last_low = rl_first_key(last_pos, window, chunk);
     // with a cap c the scores become tanh(raw * scale / c) first, and c log2(e) takes the scale's place from there on
     const float exp_scale = softcap != 0.f ? softcap * 1.4426950408889634f : scale_log2;
+    const float far_bias = BIAS ? bias_row[bias_len - 1] * 1.4426950408889634f : 0.f;
+    const float bias_unit = BIAS ? 1.4426950408889634f / exp_scale : 0.f;  // the bias in units of the scores before exp_scale
     const float cap_in = softcap != 0.f ? scale_log2 / exp_scale : 0.f;
     const uint32_t lane_addr = tmem_base + ((uint32_t)(warp * 32) << 16);
     const uint32_t o_addr = lane_addr + O_COL;
@@ -446,6 +460,17 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
 #pragma unroll
         for (int i = 0; i < BNK; ++i) v[i] = __float_as_uint(rl_tanh_sfu(__uint_as_float(v[i]) * cap_in));
       }
+      float add = 0.f;  // what every score of the tile is raised by, in base-2 exponents
+      if (BIAS) {
+        if (first_pos - (key0 + BNK - 1) >= bias_len - 1) {
+          add = far_bias;
+        } else {
+          const int gap = qpos - key0;
+#pragma unroll
+          for (int i = 0; i < BNK; ++i)
+            v[i] = __float_as_uint(fmaf(rl_distance_bias(bias_row, bias_len, gap - i), bias_unit, __uint_as_float(v[i])));
+        }
+      }
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
       if (need_mask) {
 #pragma unroll
@@ -459,14 +484,14 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         for (int i = 0; i < BNK; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(v[i]));
       }
       float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
-      mx *= exp_scale;   // the scale is positive: the maximum commutes with it
+      mx = fmaf(mx, exp_scale, add);   // the scale is positive: the maximum commutes with it
       // raise the running maximum only when it pays (see the header); the first tile sets it
       const bool raise = mx > m_run + RESCALE_THRESHOLD || (m_run == -INFINITY && mx != -INFINITY);
       const float m_next = raise ? mx : m_run;
       const float a = (raise && m_run != -INFINITY) ? exp2f(m_run - m_next) : 1.0f;
       const bool rescale = j > 0 && __any_sync(0xffffffffu, raise && m_run != -INFINITY);
       m_run = m_next;
-      const float neg_m = (m_run == -INFINITY) ? 0.f : -m_run;  // a row past the sequence's end may see nothing
+      const float neg_m = (m_run == -INFINITY) ? 0.f : add - m_run;  // a row past the sequence's end may see nothing
       if (rescale) {
         // the accumulator holds sums scaled by 2^-m_run(old): bring this warp's rows to 2^-m_next, once the product
         // of the tile before is done
@@ -548,24 +573,26 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
 // Head sizes this kernel is built for: 64 and 128 (1 if `hd` is one of them).
 RL_API int rl_flash_prefill_tc_takes(int hd) { return hd == 64 || hd == 128; }
 
-template <int HD, int MAPS>
+template <int HD, int MAPS, bool BIAS>
 static int launch_flash_tc(const void* q, int q_stride, int n_tokens, const void* k_pages, const void* v_pages, int n_pages,
                            const int* block_table, int table_width, const int* seq_start, const int* seq_pos0, void* out,
                            int out_stride, int n_seqs, int max_q_len, int H, int K, int window, float scale, int* status,
-                           int wait_test_role, unsigned int wait_test_ns, const float* sink, int chunk, float softcap, cudaStream_t stream) {
+                           int wait_test_role, unsigned int wait_test_ns, const float* sink, int chunk, float softcap, const float* bias, int bias_len, cudaStream_t stream) {
   CUtensorMap map_q, map_k, map_v;
   if (make_matrix_map(&map_q, q, n_tokens, q_stride, q_stride, BMQ))
     RL_REFUSE(10, "flash_prefill_tc: cannot describe the query tensor to TMA");
   if (make_page_map(&map_k, k_pages, n_pages, K, PAGE, HD, PAGE) || make_page_map(&map_v, v_pages, n_pages, K, PAGE, HD, PAGE))
     RL_REFUSE(11, "flash_prefill_tc: cannot describe the cache pages to TMA");
-  const size_t smem = SMEM_BYTES_OF(HD);
-  auto kern = flash_prefill_tc_kernel<HD, MAPS>;
+  const int bias_in_smem = BIAS && bias_len <= BIAS_SMEM_FLOATS(HD);
+  size_t smem = SMEM_BYTES_OF(HD);
+  if (bias_in_smem && SMEM_NEEDED(HD) + (size_t)bias_len * 4 > smem) smem = SMEM_NEEDED(HD) + (size_t)bias_len * 4;
+  auto kern = flash_prefill_tc_kernel<HD, MAPS, BIAS>;
   if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
     RL_REFUSE(12, "flash_prefill_tc: cannot get %zu bytes of shared memory", smem);
   dim3 grid(H * n_seqs, (max_q_len + BMQ - 1) / BMQ);
   RL_LAUNCH_CHECK(rl_launch(kern, grid, NUM_THREADS, smem, stream, map_q, map_k, map_v, block_table, table_width, seq_start, seq_pos0,
                             (bf16*)out, out_stride, H, K, window, scale * 1.4426950408889634f, status, wait_test_role,
-                            (uint32_t)wait_test_ns, sink, chunk, softcap));
+                            (uint32_t)wait_test_ns, sink, chunk, softcap, bias, bias_len, bias_in_smem));
   return 0;
 }
 
@@ -579,7 +606,9 @@ RL_API int rl_flash_prefill_tc(const void* q, int q_stride, int n_tokens, const 
                                int n_pages, const int* block_table, int table_width, const int* seq_start,
                                const int* seq_pos0, void* out, int out_stride, int n_seqs, int max_q_len, int H, int K,
                                int hd, int page_size, int window, float scale, int* status, int wait_test_role,
-                               unsigned int wait_test_ns, const float* sink, int chunk, float softcap, int maps, cudaStream_t stream) {
+                               unsigned int wait_test_ns, const float* sink, int chunk, float softcap, int maps, const float* bias,
+                               int bias_len, cudaStream_t stream) {
+  if (bias != nullptr && (bias_len <= 0 || maps != 1)) RL_REFUSE(13, "flash_prefill_tc: a bias by distance of %d numbers a head, %d maps (one is built)", bias_len, maps);
   if (maps < 1 || maps > 2 || H % maps) RL_REFUSE(9, "flash_prefill_tc: %d maps in %d heads", maps, H);
   if (n_seqs <= 0 || max_q_len <= 0 || H <= 0 || K <= 0 || n_tokens <= 0 || n_pages <= 0)
     RL_REFUSE(1, "flash_prefill_tc: S=%d max_q=%d H=%d K=%d T=%d pages=%d", n_seqs, max_q_len, H, K, n_tokens, n_pages);
@@ -592,13 +621,15 @@ RL_API int rl_flash_prefill_tc(const void* q, int q_stride, int n_tokens, const 
     RL_REFUSE(7, "flash_prefill_tc: H=%d x S=%d blocks or %d query rows exceed the grid", H, n_seqs, max_q_len);
   if (window < 0 || chunk < 0 || softcap < 0.f || status == nullptr || !(scale > 0.f))
     RL_REFUSE(8, "flash_prefill_tc: bad window, chunk, cap or scale, or no status word");
-#define RL_FTC(HDV, MAPSV)                                                                                                                  \
-  return launch_flash_tc<HDV, MAPSV>(q, q_stride, n_tokens, k_pages, v_pages, n_pages, block_table, table_width, seq_start, seq_pos0, out,  \
+#define RL_FTC(HDV, MAPSV, BIASV)                                                                                                                  \
+  return launch_flash_tc<HDV, MAPSV, BIASV>(q, q_stride, n_tokens, k_pages, v_pages, n_pages, block_table, table_width, seq_start, seq_pos0, out,  \
                                      out_stride, n_seqs, max_q_len, H, K, window, scale, status, wait_test_role, wait_test_ns, sink, chunk, \
-                                     softcap, stream)
-  if (hd == 64 && maps == 2) RL_FTC(64, 2);
-  if (hd == 64) RL_FTC(64, 1);
-  if (maps == 2) RL_FTC(128, 2);
-  RL_FTC(128, 1);
+                                     softcap, bias, bias_len, stream)
+  if (bias != nullptr && hd == 64) RL_FTC(64, 1, true);
+  if (bias != nullptr) RL_FTC(128, 1, true);
+  if (hd == 64 && maps == 2) RL_FTC(64, 2, false);
+  if (hd == 64) RL_FTC(64, 1, false);
+  if (maps == 2) RL_FTC(128, 2, false);
+  RL_FTC(128, 1, false);
 #undef RL_FTC
 }

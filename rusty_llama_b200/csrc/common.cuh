@@ -144,6 +144,12 @@ __device__ __forceinline__ int rl_first_key(int pos, int window, int chunk) {
   return first;
 }
 
+// The learned bias of a score by how far the key lies behind the query.  row: one head's numbers by distance, `len` of them; the last
+// one also serves every larger distance.  (A weight: no kernel writes it, so it may be asked for before pdl_wait.)
+__device__ __forceinline__ float rl_distance_bias(const float* row, int len, int distance) {
+  return row[min(max(distance, 0), len - 1)];
+}
+
 // tanh for the capped scores of the bfloat16 attention kernels: 1 - 2 / (exp(2x) + 1) on the special-function unit (two of its
 // operations and three others, where tanhf takes a branch and a polynomial).  The absolute error stays near 2e-7 for every x
 // (which is what a score's exponential sees); the relative error of small results does not.

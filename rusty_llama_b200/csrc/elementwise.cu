@@ -63,7 +63,7 @@ RL_API int rl_embed_gather(const int* tokens, const void* table, int table_dtype
 // For output row r (stream row t = rows ? rows[r] : r):
 //   v = x[t] + delta[0][t] + delta[1][t] + ...        (32-bit, in this order)
 //   if write_x: x[t] = v
-//   if w: out[r] = v * (1 / sqrt(sum(v^2)/d + eps)) * w   (src/backend/cpu.rs:96-105)
+//   if w: out[r] = v * (1 / sqrt(sum(v^2)/d + eps)) * w   (src/backend/cpu.rs:96-105); an output without a weight is v itself
 // The row is held in shared memory between the two passes.
 // With VEC (d a multiple of 4) a thread handles four neighbouring values per round and the block
 // is sized so that a row of up to 4096 values takes one round: all loads are in flight together,
@@ -113,7 +113,10 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ x, const TD* __restrict__
 #pragma unroll
       for (int e = 0; e < 4; ++e) ss += v[e] * v[e];
     }
-    if (w == nullptr) return;
+    if (w == nullptr) {
+      if (out != nullptr && mine) store4<TA>(out + (size_t)r * d + i, v);
+      return;
+    }
     const float total = block_sum(ss, red);
     const float inv = 1.0f / sqrtf(total / (float)d + eps);
     if (mine) {
@@ -147,10 +150,18 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ x, const TD* __restrict__
       ss += v * v;
     }
   }
-  if (w == nullptr) return;
+  TA* o = out + (size_t)r * d;
+  if (w == nullptr) {
+    if (out == nullptr) return;  // (each thread reads back what it put into the row itself)
+    if (VEC) {
+      for (int i = threadIdx.x * 4; i < d; i += blockDim.x * 4) store4<TA>(o + i, row + i);
+    } else {
+      for (int i = threadIdx.x; i < d; i += blockDim.x) o[i] = from_f32<TA>(row[i]);
+    }
+    return;
+  }
   const float total = block_sum(ss, red);
   const float inv = 1.0f / sqrtf(total / (float)d + eps);
-  TA* o = out + (size_t)r * d;
   if (VEC) {
     for (int i = threadIdx.x * 4; i < d; i += blockDim.x * 4) {
       float v[4], wv[4];
@@ -236,10 +247,18 @@ add_rmsnorm_rows_kernel(float* __restrict__ x, const TD* __restrict__ delta, int
 #pragma unroll
     for (int e = 0; e < 4; ++e) ss += v[c][e] * v[c][e];
   }
-  if (w == nullptr) return;
+  TA* o = out + (size_t)r * d;
+  if (w == nullptr) {
+    if (out == nullptr) return;
+#pragma unroll
+    for (int c = 0; c < CHUNKS; ++c) {
+      const int i = (threadIdx.x + c * 256) * 4;
+      if (i < d) store4<TA>(o + i, v[c]);
+    }
+    return;
+  }
   const float total = block_sum(ss, red);
   const float inv = 1.0f / sqrtf(total / (float)d + eps);
-  TA* o = out + (size_t)r * d;
 #pragma unroll
   for (int c = 0; c < CHUNKS; ++c) {
     const int i = (threadIdx.x + c * 256) * 4;
@@ -433,7 +452,7 @@ RL_API int rl_clamped_glu(const void* gate_up, void* h, int act_dtype, int n_tok
 // For a layer that norms what its sublayer returns before adding it (and norms the stream again for the next sublayer):
 //   s = delta[0][t] + delta[1][t] + ... (+ bias)                 (32-bit, in this order; bias: a row of d numbers or none)
 //   v = x[t] + s / sqrt(mean(s^2) + eps_d) * wd                 x[t] = v
-//   if w: out[t] = v / sqrt(mean(v^2) + eps) * w
+//   if w: out[t] = v / sqrt(mean(v^2) + eps) * w; an output without a weight is v itself (a next sublayer that reads the stream as it is)
 // One block per row, the row in shared memory between the passes; every sum in the block's fixed order.
 template <typename TA, typename TW, typename TD, bool VEC>
 __global__ void normed_add_rmsnorm_kernel(float* __restrict__ x, const TD* __restrict__ delta, int n_parts, long long part_stride,
@@ -489,12 +508,14 @@ __global__ void normed_add_rmsnorm_kernel(float* __restrict__ x, const TD* __res
       }
       store4<float>(row + i, v);
       if (write_x) store4<float>(xr + i, v);
+      if (w == nullptr && out != nullptr) store4<TA>(o + i, v);
     }
   } else {
     for (int i = threadIdx.x; i < d; i += blockDim.x) {
       const float v = xr[i] + row[i] * inv_d * to_f32(wd[i]);
       row[i] = v;
       if (write_x) xr[i] = v;
+      if (w == nullptr && out != nullptr) o[i] = from_f32<TA>(v);
       ss += v * v;
     }
   }

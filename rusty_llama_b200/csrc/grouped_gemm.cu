@@ -2,7 +2,8 @@
 //
 //   moe_gemm_mma     the products of a routed feed-forward: a block takes one row tile of the plan that `moe_plan`
 //                    left on the device (rows of ONE expert, gathered through `order`) and 64 columns of that expert's
-//                    matrix; with ACT it computes the gate and the up product together and writes gated_act(gate, up) (silu(gate) * up, or the clamped form)
+//                    matrix; with ACT it computes the gate and the up product together and writes gated_act(gate, up) (silu(gate) * up, or the clamped form),
+//                    without it the sums may go through relu(x)^2 (`unary_post`)
 //   head_linear_mma  out[t, h, :] = W[h] x[t, h, :] for every head h, optionally times sigmoid(gate[t, h, :])
 //
 // Both are the same tile loop: BM rows x BN columns per block, k in slices of 64 through two stages of shared memory
@@ -159,6 +160,7 @@ moe_gemm_mma_kernel(const bf16* __restrict__ x, int ldx, const int* __restrict__
           if (n >= N) continue;
           float v = acc[i][j][2 * hh + c];
           if (ACT) v = gated_act(v, acc2[ACT ? i : 0][ACT ? j : 0][2 * hh + c], act_alpha, act_limit);
+          else v = unary_post(v, act_limit);
           out[(size_t)(r0 + r) * ldo + n] = from_f32<TO>(v);
         }
     }

@@ -8,8 +8,11 @@
 //                with the inverse `place`), and cuts each expert's range into row tiles (`tiles`) of a given height
 //   moe_gemm     one kernel for all experts: a block takes one row tile (rows of ONE expert) and one column
 //                tile; rows are gathered through `order`; with ACT the block computes the gate and the up
-//                product together and writes act(gate) * up
+//                product together and writes act(gate) * up; without it the sums may go through relu(x)^2
 //   moe_combine  out[t] = sum_j weight[t,j] * y[place[t,j]]  (+ gate[t] * shared[t]), in the order j = 0, 1, ...
+//
+// The router may score more choices than there are experts: those behind the experts hand the token's input on.  They have
+// no rows in the plan (their place is -1), and moe_combine takes x[t] in the place of y for them.
 //
 // Nothing here depends on the host knowing how many tokens an expert got: grids are sized by upper bounds and
 // blocks without work leave, so a step with these kernels can be captured in a CUDA graph.  Each output is one
@@ -205,7 +208,8 @@ moe_plan_kernel(const int* __restrict__ ids, int n, int E, int* __restrict__ ord
   int mine = 0;
   for (int i = lo; i < hi; ++i) {
     const int id = ids[i];
-    atomicAdd(&cnt[id], 1);
+    if (id < E) atomicAdd(&cnt[id], 1);
+    else if (e == 0) place[i] = -1;  // (no expert of the plan: it has no row)
     mine += id == e;
   }
   scan[tid] = mine;
@@ -351,6 +355,7 @@ moe_gemm_kernel(const TA* __restrict__ x, int ldx, const int* __restrict__ order
       if (n >= N) continue;
       float v = acc[i][j];
       if (ACT) v = gated_act(v, acc2[i][j], act_alpha, act_limit);
+      else v = unary_post(v, act_limit);
       out[(size_t)(r0 + r) * ldo + n] = from_f32<TO>(v);
     }
   }
@@ -377,27 +382,35 @@ RL_API int rl_moe_gemm(const void* x, int ldx, int dtype, const int* order, int 
 }
 
 // ---------------------------------------------------------------- weighted sum of a token's experts
-// out[t, :] = sum_j weights[t, j] * y[place[t * top + j], :]  (+ gate[t] * shared[t, :]); y is float32.
+// out[t, :] = sum_j weights[t, j] * y[place[t * top + j], :]  (+ gate[t] * shared[t, :]); y is float32.  A negative place takes
+// x[t, :], the experts' input (of type TS, like `shared`), in the place of y.
 template <typename TS, typename TO>
 __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ place, const float* __restrict__ weights,
-                                   int top, const TS* __restrict__ shared, const float* __restrict__ gate, TO* __restrict__ out, int d) {
+                                   int top, const TS* __restrict__ shared, const float* __restrict__ gate, TO* __restrict__ out, int d,
+                                   const TS* __restrict__ x, int ldx) {
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x;
   for (int i = threadIdx.x; i < d; i += blockDim.x) {
     float v = 0.f;
-    for (int j = 0; j < top; ++j) v += weights[(size_t)t * top + j] * y[(size_t)place[(size_t)t * top + j] * d + i];
+    for (int j = 0; j < top; ++j) {
+      const int p = place[(size_t)t * top + j];
+      v += weights[(size_t)t * top + j] * (p >= 0 ? y[(size_t)p * d + i] : x != nullptr ? to_f32(x[(size_t)t * ldx + i]) : 0.f);
+    }
     if (shared) v += (gate ? gate[t] : 1.f) * to_f32(shared[(size_t)t * d + i]);
     out[(size_t)t * d + i] = from_f32<TO>(v);
   }
 }
 
 RL_API int rl_moe_combine(const float* y, const int* place, const float* weights, int top, const void* shared, int shared_dtype,
-                          const float* gate, void* out, int out_dtype, int n_tokens, int d, cudaStream_t stream) {
+                          const float* gate, void* out, int out_dtype, int n_tokens, int d, const void* x, int x_dtype, int ldx,
+                          cudaStream_t stream) {
   if (n_tokens <= 0 || d <= 0 || top <= 0) RL_REFUSE(1, "moe_combine: T=%d d=%d top=%d", n_tokens, d, top);
+  if (shared == nullptr && x != nullptr) shared_dtype = x_dtype;
+  if (x != nullptr && shared_dtype != x_dtype) RL_REFUSE(3, "moe_combine: shared result of type %d beside an input of type %d", shared_dtype, x_dtype);
 #define RL_MC(TS, TO)                                                                                                          \
   RL_LAUNCH_CHECK(rl_launch<false>(moe_combine_kernel<TS, TO>, n_tokens, 256, 0, stream, y, place, weights, top, (const TS*)shared, \
-                                   gate, (TO*)out, d))
+                                   gate, (TO*)out, d, (const TS*)x, ldx))
   if (shared_dtype == RL_BF16 && out_dtype == RL_F32) RL_MC(bf16, float);
   else if (shared_dtype == RL_F32 && out_dtype == RL_F32) RL_MC(float, float);
   else if (shared_dtype == RL_BF16 && out_dtype == RL_BF16) RL_MC(bf16, bf16);

@@ -111,11 +111,12 @@ def add_rmsnorm(
     rows: Optional[torch.Tensor] = None,
     write_x: bool = True,
     out: Optional[torch.Tensor] = None,
+    plain_out: bool = False,
 ) -> Optional[torch.Tensor]:
     """x (float32 [T, d]) += sum of delta parts; returns rmsnorm(x) * weight in `act_dtype`.
 
     delta: None, [T, d] or [parts, T, d], in `act_dtype` or in float32 (partial sums of a product
-    split over k).  weight None: only the sum.
+    split over k).  weight None: only the sum; with plain_out the sum itself is returned in `act_dtype`.
     rows: int32 indices of the rows to produce (all rows if None).
     """
     _cuda(x, "add_rmsnorm x", torch.float32)
@@ -146,6 +147,8 @@ def add_rmsnorm(
             out = torch.empty((n_rows, d), dtype=act_dtype, device=x.device)
         _cuda(out, "add_rmsnorm out", act_dtype)
         _need(tuple(out.shape) == (n_rows, d), "add_rmsnorm: out has the wrong shape")
+    elif plain_out:
+        out = torch.empty((n_rows, d), dtype=act_dtype, device=x.device)
     else:
         _need(delta is not None, "add_rmsnorm: neither a delta nor a weight, nothing to do")
         out = None
@@ -310,6 +313,16 @@ def _check_sink(sink, num_heads: int, what: str) -> None:
         _need(sink.numel() == num_heads, f"{what}: one sink per head")
 
 
+def _bias_args(bias, num_heads: int, what: str):
+    """A learned bias by head and distance: None, or float32 [H, L]; a score of head h and a key n positions behind its query is
+    raised by bias[h, min(n, L - 1)], after everything else that makes the score."""
+    if bias is None:
+        return c_void_p(0), c_int(0)
+    _cuda(bias, f"{what} bias", torch.float32)
+    _need(bias.dim() == 2 and bias.shape[0] == num_heads and bias.shape[1] > 0, f"{what}: bias {tuple(bias.shape)} for {num_heads} heads")
+    return _p(bias), c_int(bias.shape[1])
+
+
 def attn_decode_scratch_floats(n_seqs: int, num_heads: int, head_dim: int, n_splits: int) -> int:
     return n_seqs * num_heads * n_splits * (head_dim + 2)
 
@@ -320,8 +333,11 @@ def attn_decode(
     out: Optional[torch.Tensor] = None, impl: str = "auto", fuse: int = 0,
     inv_freq: Optional[torch.Tensor] = None, rotary_dim: int = 0, interleaved: bool = False,
     counters: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0, pair=None,
+    bias: Optional[torch.Tensor] = None,
 ) -> torch.Tensor:
     """One query token per sequence over keys 0..seq_len-1, the key range cut into `n_splits`.
+
+    bias (the "tma" kernel only): None, or float32 [H, L], a learned bias of the scores by head and distance (`_bias_args`).
 
     pair (the "tma" kernel only): None, or (lambda, eps, factor): query heads 2h and 2h + 1 are two maps, the two halves of row h's
     head_dim numbers (q's rows hold H / 2 such rows, k and v follow them with fuse = 2) against the same halves of the keys, and the
@@ -406,11 +422,11 @@ def attn_decode(
             c_int(1 if interleaved else 0), _p(counters) if counters is not None else c_void_p(0),
             _p(q_parts) if q_parts is not None else c_void_p(0), c_int(0 if q_parts is None else q_parts.shape[0]),
             c_ll(0 if q_parts is None else q_parts.stride(0)), *_wt(), _p(sink), c_int(chunk), c_float(softcap), c_int(maps),
-            *(c_float(x) for x in (pair or (0.0, 0.0, 0.0))), _stream(),
+            *(c_float(x) for x in (pair or (0.0, 0.0, 0.0))), *_bias_args(bias, num_heads, "attn_decode"), _stream(),
         )
         _check(lib, rc, "attn_decode_tma", kernels=1 if counters is not None else 2)
         return out
-    _need(chunk == 0 and softcap == 0.0 and pair is None, "attn_decode: only the TMA kernel takes chunks, capped scores and two maps per head")
+    _need(chunk == 0 and softcap == 0.0 and pair is None and bias is None, "attn_decode: only the TMA kernel takes chunks, capped scores, a bias and two maps per head")
     lib = build.load("attention_decode")
     rc = lib.rl_attn_decode_sink(
         _p(q), c_int(_dt(q, "attn_decode")), c_int(qs), _p(k_pages), _p(v_pages), _p(block_table),
@@ -462,11 +478,13 @@ def flash_prefill_tc(
     q: torch.Tensor, k_pages, v_pages, block_table, seq_start, seq_pos0, max_q_len: int, num_heads: int,
     num_kv_heads: int, head_dim: int, window: int = 0, scale: Optional[float] = None,
     out: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0, maps: int = 1,
+    bias: Optional[torch.Tensor] = None,
 ) -> torch.Tensor:
     """`flash_prefill` on the tcgen05 tensor cores (TMA-fed, S and P V in tensor memory); head sizes 64 and 128.
     chunk: 0, or the size of the chunks of positions (counted from 0) outside of which a query sees nothing; softcap: 0, or the
     cap c of s <- c tanh(s / c) on the scaled scores.
-    maps: 1, or 2: query heads 2h and 2h + 1 are the two halves of row h's head_dim numbers, against the same halves of the keys."""
+    maps: 1, or 2: query heads 2h and 2h + 1 are the two halves of row h's head_dim numbers, against the same halves of the keys.
+    bias: None, or float32 [H, L], a learned bias of the scores by head and distance (`_bias_args`; one map only)."""
     _need(maps in (1, 2) and num_heads % maps == 0, f"flash_prefill_tc: {maps} maps in {num_heads} heads")
     _need(head_dim in FLASH_TC_HEAD_DIMS, f"flash_prefill_tc: head size {head_dim}, this kernel is built for {FLASH_TC_HEAD_DIMS}")
     _cuda(q, "flash_prefill_tc q", torch.bfloat16, contiguous=False)
@@ -493,7 +511,7 @@ def flash_prefill_tc(
         _p(q), c_int(qs), c_int(T), _p(k_pages), _p(v_pages), c_int(k_pages.shape[0]), _p(block_table),
         c_int(block_table.shape[1]), _p(seq_start), _p(seq_pos0), _p(out), c_int(out.stride(0)), c_int(S), c_int(max_q_len),
         c_int(num_heads), c_int(num_kv_heads), c_int(head_dim), c_int(PAGE_SIZE), c_int(window), c_float(scale), _p(status), *_wt(), _p(sink),
-        c_int(chunk), c_float(softcap), c_int(maps), _stream(),
+        c_int(chunk), c_float(softcap), c_int(maps), *_bias_args(bias, num_heads, "flash_prefill_tc"), _stream(),
     )
     _check(lib, rc, "flash_prefill_tc")
     return out
@@ -925,9 +943,10 @@ def sample_chain(
 def normed_add_rmsnorm(
     x: torch.Tensor, delta: torch.Tensor, delta_weight: torch.Tensor, delta_eps: float, weight: Optional[torch.Tensor], eps: float,
     act_dtype: torch.dtype, rows: Optional[torch.Tensor] = None, write_x: bool = True, delta_bias: Optional[torch.Tensor] = None,
+    plain_out: bool = False,
 ) -> Optional[torch.Tensor]:
     """x (float32 [T, d]) += rmsnorm(sum of delta parts + delta_bias) * delta_weight; returns rmsnorm(x) * weight in `act_dtype`
-    (None without a weight).  delta: [T, d] or [parts, T, d], in `act_dtype` or float32.  Both norm weights have one type.
+    (without a weight: None, or with plain_out the new x itself in `act_dtype`).  delta: [T, d] or [parts, T, d], in `act_dtype` or float32.  Both norm weights have one type.
     delta_bias: None or float32 [d], a row that belongs to every row of the summed delta (a projection's bias)."""
     _cuda(x, "normed_add_rmsnorm x", torch.float32)
     T, d = x.shape
@@ -946,6 +965,7 @@ def normed_add_rmsnorm(
     if weight is not None:
         _cuda(weight, "normed_add_rmsnorm weight", delta_weight.dtype)
         _need(tuple(weight.shape) == (d,), "normed_add_rmsnorm: weight does not match d")
+    if weight is not None or plain_out:
         out = torch.empty((n_rows, d), dtype=act_dtype, device=x.device)
     if rows is not None:
         _cuda(rows, "normed_add_rmsnorm rows", torch.int32)
@@ -1235,6 +1255,7 @@ def moe_max_tiles(n_pairs: int, n_experts: int, tile_rows: int = 0) -> int:
 
 def moe_plan(ids: torch.Tensor, n_experts: int, tile_rows: int = 0):
     """ids int32 [T, top] -> (order [T top], place [T top], tiles [1 + 3 max_tiles], max_tiles), all on the device.
+    A pair whose id is n_experts or more names no expert of the plan: it has no row, and its place is -1.
     tile_rows: the height of a row tile (0: the plain product's)."""
     _cuda(ids, "moe_plan ids", torch.int32)
     n = ids.numel()
@@ -1256,7 +1277,7 @@ def moe_gemm(
     """out[r] = w[expert of r] . x[row of r] for the n_rows rows of a plan's layout; w: [E, N, K].
 
     order given: row r reads x[order[r] // gather_div], else x[r].  w2 given: out = silu(w x) * (w2 x), or with act = (alpha, limit)
-    g s(alpha g) (u + 1), g = min(w x, limit), u = clamp(w2 x, -limit, limit).
+    g s(alpha g) (u + 1), g = min(w x, limit), u = clamp(w2 x, -limit, limit).  Without w2, act "relu2": out = relu(w x)^2.
     tile_rows: the height of the plan's tiles; bfloat16 operands whose rows can be moved in 16-byte pieces go to the
     tensor cores if it is one of MOE_MMA_TILE_ROWS, everything else to the plain kernel (which wants its own height)."""
     _cuda(x, "moe_gemm x", contiguous=False)
@@ -1269,6 +1290,7 @@ def moe_gemm(
     out_dtype = out_dtype or x.dtype
     out = torch.empty((n_rows, N), dtype=out_dtype, device=x.device)
     tile_rows = tile_rows or moe_tile_rows()
+    _need(act is None or (act == "relu2") == (w2 is None), "moe_gemm: an activation of one argument goes with one matrix, a gate's with two")
     alpha, limit = _act(act)
     if x.dtype == torch.bfloat16 and tile_rows in MOE_MMA_TILE_ROWS and grouped_gemm_takes(K, x.stride(0), 0) and x.data_ptr() % 16 == 0:
         lib = build.load("grouped_gemm")
@@ -1290,9 +1312,10 @@ def moe_gemm(
 
 def moe_combine(
     y: torch.Tensor, place: torch.Tensor, weights: torch.Tensor, shared: Optional[torch.Tensor], gate: Optional[torch.Tensor],
-    out_dtype: torch.dtype = torch.float32,
+    out_dtype: torch.dtype = torch.float32, x: Optional[torch.Tensor] = None,
 ) -> torch.Tensor:
-    """out[t] = sum_j weights[t, j] * y[place[t, j]] (+ gate[t] * shared[t]); y float32 [T top, d]."""
+    """out[t] = sum_j weights[t, j] * y[place[t, j]] (+ gate[t] * shared[t]); y float32 [T top, d].  Where place is negative the
+    term is weights[t, j] * x[t] (x [T, d], the experts' input: a choice that hands the input on)."""
     _cuda(y, "moe_combine y", torch.float32)
     _cuda(weights, "moe_combine weights", torch.float32)
     _cuda(place, "moe_combine place", torch.int32)
@@ -1306,11 +1329,16 @@ def moe_combine(
         shared_dt = _dt(shared, "moe_combine shared")
     if gate is not None:
         _cuda(gate, "moe_combine gate", torch.float32)
+    x_dt, xs = _F32, 0
+    if x is not None:
+        _cuda(x, "moe_combine x", contiguous=False)
+        _need(tuple(x.shape) == (T, d), "moe_combine: x has the wrong shape")
+        x_dt, xs = _dt(x, "moe_combine x"), _rows(x, "moe_combine x")
     out = torch.empty((T, d), dtype=out_dtype, device=y.device)
     lib = build.load("moe")
     rc = lib.rl_moe_combine(
         _p(y), _p(place), _p(weights), c_int(top), _p(shared), c_int(shared_dt), _p(gate), _p(out), c_int(_dt(out, "moe_combine out")),
-        c_int(T), c_int(d), _stream(),
+        c_int(T), c_int(d), _p(x), c_int(x_dt), c_int(xs), _stream(),
     )
     _check(lib, rc, "moe_combine")
     return out
@@ -1380,35 +1408,46 @@ def qkv_prep(
     qkv: torch.Tensor, bias: Optional[torch.Tensor], tok_pos: torch.Tensor, tok_seq: torch.Tensor, block_table: torch.Tensor,
     k_pages: torch.Tensor, v_pages: torch.Tensor, inv_freq: Optional[torch.Tensor], magnitude: float, num_heads: int, num_kv_heads: int,
     kdim: int, vdim: int, rotary_dim: int, interleaved: bool, q_norm: Optional[torch.Tensor] = None, k_norm: Optional[torch.Tensor] = None,
-    norm_eps: float = 0.0, v_src: Optional[torch.Tensor] = None, v_lambda: Optional[torch.Tensor] = None,
+    norm_eps: float = 0.0, v_src: Optional[torch.Tensor] = None, v_lambda: Optional[torch.Tensor] = None, norm_whole: bool = False,
+    v_from_k: bool = False, temperature=None,
 ) -> None:
     """qkv[T, >= (H + K) kdim + K vdim]: add `bias` (float32, one number per column, or None), divide every q head (k head) by its
     root mean square and multiply it by `q_norm` (`k_norm`; float32 [kdim], None: no norm), rotate the first `rotary_dim`
     dimensions of every q head (in place) and k head by position * inv_freq, cosines and sines times `magnitude`, and store
     k and v at each token's place in the paged cache (k_pages [pages, K, PAGE_SIZE, kdim], v_pages [..., vdim]).
     v_src ([T, K vdim] rows of qkv's type) with v_lambda (float32, one number on the device): what is stored as the value is
-    (1 - lambda) v + lambda v_src[t]."""
+    (1 - lambda) v + lambda v_src[t].
+    norm_whole: the norm is taken over all q heads at once and over all k heads at once (q_norm [H kdim], k_norm [K kdim]).
+    v_from_k: the rows hold no values; what is stored as the value is the key as projected, before its norm (vdim = kdim).
+    temperature: None, or (coef, every): q at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1) after its norm.
+    num_kv_heads 0: rows of queries only; nothing is stored, and the pages may be None."""
     _cuda(qkv, "qkv_prep qkv", contiguous=False)
     stride = _rows(qkv, "qkv_prep qkv")
     T = qkv.shape[0]
-    cols = (num_heads + num_kv_heads) * kdim + num_kv_heads * vdim
+    cols = (num_heads + num_kv_heads) * kdim + (0 if v_from_k else num_kv_heads * vdim)
     _need(qkv.shape[1] >= cols, "qkv_prep: qkv rows too short")
     _cuda(tok_pos, "qkv_prep tok_pos", torch.int32)
     _cuda(tok_seq, "qkv_prep tok_seq", torch.int32)
     _need(tok_pos.numel() == T and tok_seq.numel() == T, "qkv_prep: one position and one sequence index per token")
-    _cuda(block_table, "qkv_prep block_table", torch.int32)
-    _need(block_table.dim() == 2, "qkv_prep: block_table must be [S, width]")
-    _check_kv_pages(k_pages, v_pages, qkv.dtype, num_kv_heads, kdim, vdim, "qkv_prep")
+    if num_kv_heads:
+        _cuda(block_table, "qkv_prep block_table", torch.int32)
+        _need(block_table.dim() == 2, "qkv_prep: block_table must be [S, width]")
+        _check_kv_pages(k_pages, v_pages, qkv.dtype, num_kv_heads, kdim, vdim, "qkv_prep")
+    else:
+        block_table = k_pages = v_pages = None
+    coef, every = temperature or (0.0, 0)
+    _need(temperature is None or int(every) > 0, f"qkv_prep: a temperature that grows every {every} positions")
     if bias is not None:
         _cuda(bias, "qkv_prep bias", torch.float32)
         _need(bias.numel() == cols, f"qkv_prep: bias has {bias.numel()} numbers for {cols} columns")
     if rotary_dim:
         _cuda(inv_freq, "qkv_prep inv_freq", torch.float32)
         _need(inv_freq.numel() == rotary_dim // 2, "qkv_prep: inv_freq must hold rotary_dim/2 values")
-    for name, w in (("q_norm", q_norm), ("k_norm", k_norm)):
+    for name, w, heads in (("q_norm", q_norm, num_heads), ("k_norm", k_norm, num_kv_heads)):
         if w is not None:
             _cuda(w, f"qkv_prep {name}", torch.float32)
-            _need(w.numel() == kdim, f"qkv_prep: {name} must hold one weight per number of a head ({kdim})")
+            want = heads * kdim if norm_whole else kdim
+            _need(w.numel() == want, f"qkv_prep: {name} must hold one weight per number of {'all heads' if norm_whole else 'a head'} ({want})")
     vs_stride = 0
     if v_src is not None:
         _cuda(v_src, "qkv_prep v_src", qkv.dtype, contiguous=False)
@@ -1418,10 +1457,10 @@ def qkv_prep(
         _need(v_lambda.numel() == 1, "qkv_prep: v_lambda is one number")
     lib = build.load("attention_ext")
     rc = lib.rl_qkv_prep(
-        _p(qkv), c_int(_dt(qkv, "qkv_prep")), c_int(stride), _p(bias), _p(tok_pos), _p(tok_seq), _p(block_table), c_int(block_table.shape[1]),
+        _p(qkv), c_int(_dt(qkv, "qkv_prep")), c_int(stride), _p(bias), _p(tok_pos), _p(tok_seq), _p(block_table), c_int(1 if block_table is None else block_table.shape[1]),
         _p(k_pages), _p(v_pages), _p(inv_freq if rotary_dim else None), c_float(magnitude), _p(q_norm), _p(k_norm), c_float(norm_eps), c_int(T), c_int(num_heads),
         c_int(num_kv_heads), c_int(kdim), c_int(vdim), c_int(rotary_dim), c_int(1 if interleaved else 0), c_int(PAGE_SIZE),
-        _p(v_src), c_int(vs_stride), _p(v_lambda), _stream(),
+        _p(v_src), c_int(vs_stride), _p(v_lambda), c_int(1 if norm_whole else 0), c_int(1 if v_from_k else 0), c_float(coef), c_int(int(every)), _stream(),
     )
     _check(lib, rc, "qkv_prep")
 
@@ -1430,9 +1469,11 @@ def attn_ext(
     q: torch.Tensor, k_pages, v_pages, block_table, tok_seq, tok_pos, num_heads: int, num_kv_heads: int, kdim: int, vdim: int,
     scale: float, window: int = 0, sink: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None,
     gate: Optional[torch.Tensor] = None, out_scale: float = 1.0, out: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0,
-    maps: int = 1,
+    maps: int = 1, bias: Optional[torch.Tensor] = None,
 ) -> torch.Tensor:
     """Attention of each token over its sequence's cached keys, both element types, prompts and decoding.
+
+    bias: None, or float32 [H, L], a learned bias of the scores by head and distance (`_bias_args`).
 
     maps: 1, or 2: query heads 2h and 2h + 1 are the two halves of row h's kdim numbers, against the same halves of the keys (the
     values are whole; `map_combine` makes one head of the two results).
@@ -1472,7 +1513,8 @@ def attn_ext(
     rc = lib.rl_attn_ext(
         _p(q), c_int(_dt(q, "attn_ext")), c_int(qs), _p(k_pages), _p(v_pages), _p(block_table), c_int(block_table.shape[1]), _p(tok_seq),
         _p(tok_pos), _p(sink), _p(mix), _p(gate), c_int(gs), c_float(out_scale), _p(out), c_int(out.stride(0)), c_int(T), c_int(num_heads),
-        c_int(num_kv_heads), c_int(kdim), c_int(vdim), c_int(PAGE_SIZE), c_int(window), c_float(scale), c_int(chunk), c_float(softcap), c_int(maps), _stream(),
+        c_int(num_kv_heads), c_int(kdim), c_int(vdim), c_int(PAGE_SIZE), c_int(window), c_float(scale), c_int(chunk), c_float(softcap), c_int(maps),
+        *_bias_args(bias, num_heads, "attn_ext"), _stream(),
     )
     _check(lib, rc, "attn_ext")
     return out
@@ -2161,12 +2203,13 @@ def flash_mix(
     q: torch.Tensor, k_pages, v_pages, block_table, seq_start, seq_pos0, max_q_len: int, num_heads: int, num_kv_heads: int, kdim: int,
     vdim: int, scale: float, window: int = 0, sink: Optional[torch.Tensor] = None, folded: bool = False, gate: Optional[torch.Tensor] = None,
     out_scale: float = 1.0, out: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0, maps: int = 1,
+    bias: Optional[torch.Tensor] = None,
 ) -> torch.Tensor:
     """bfloat16 attention of a ragged batch over the paged cache on the tensor cores, keys of `kdim` and values of `vdim` numbers,
     with a window, chunks (a query sees the keys of its own chunk of positions only), capped scores (s <- c tanh(s / c)), a sink,
     a gate (out *= sigmoid(gate)) and a constant factor.  folded: q is what `fold_queries` made
     ([T, H K kdim]: the heads' scores are mixed); else q holds [T, >= H kdim] rows.  maps: as in `attn_ext` (not folded; kdim a
-    multiple of 16)."""
+    multiple of 16).  bias: as in `attn_ext`."""
     _cuda(q, "flash_mix q", torch.bfloat16, contiguous=False)
     qs = _rows(q, "flash_mix q")
     T = q.shape[0]
@@ -2195,7 +2238,7 @@ def flash_mix(
         _p(q), c_ll(qs), c_int(parts * kdim), c_int(parts), _p(k_pages), _p(v_pages), _p(block_table), c_int(block_table.shape[1]),
         _p(seq_start), _p(seq_pos0), _p(sink), _p(gate), c_int(gs), c_float(out_scale), _p(out), c_int(out.stride(0)), c_int(S),
         c_int(max_q_len), c_int(num_heads), c_int(num_kv_heads), c_int(kdim), c_int(vdim), c_int(PAGE_SIZE), c_int(window), c_float(scale),
-        c_int(chunk), c_float(softcap), c_int(maps), _stream(),
+        c_int(chunk), c_float(softcap), c_int(maps), *_bias_args(bias, num_heads, "flash_mix"), _stream(),
     )
     _check(lib, rc, "flash_mix")
     return out
@@ -2219,11 +2262,11 @@ def flash_mix_decode_scratch_floats(n_seqs: int, num_heads: int, vdim: int, n_sp
 def flash_mix_decode(
     qf: torch.Tensor, k_pages, v_pages, block_table, seq_pos0, num_heads: int, num_kv_heads: int, kdim: int, vdim: int, scale: float,
     n_splits: int, scratch: torch.Tensor, window: int = 0, sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-    out_scale: float = 1.0, out: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0,
+    out_scale: float = 1.0, out: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0, bias: Optional[torch.Tensor] = None,
 ) -> torch.Tensor:
     """One query token per sequence, at position seq_pos0[s], over its sequence's cached keys (its own among them), the key range
     cut into `n_splits` parts; a block's rows are the heads.  qf: folded queries [S, H K kdim] (`fold_queries`, with the identity
-    matrix for an attention without mixing).  scratch: float32, `flash_mix_decode_scratch_floats(...)`."""
+    matrix for an attention without mixing).  scratch: float32, `flash_mix_decode_scratch_floats(...)`.  bias: as in `attn_ext`."""
     _cuda(qf, "flash_mix_decode qf", torch.bfloat16)
     S = qf.shape[0]
     _need(qf.dim() == 2 and qf.shape[1] == num_heads * num_kv_heads * kdim, "flash_mix_decode: qf must be [S, H K kdim]")
@@ -2251,7 +2294,7 @@ def flash_mix_decode(
         _p(qf), _p(k_pages), _p(v_pages), _p(block_table), c_int(block_table.shape[1]), _p(seq_pos0), _p(sink), _p(gate), c_int(gs),
         c_float(out_scale), c_void_p(scratch.data_ptr()), c_void_p(scratch.data_ptr() + 4 * n_o), _p(out), c_int(out.stride(0)), c_int(S),
         c_int(num_heads), c_int(num_kv_heads), c_int(kdim), c_int(vdim), c_int(PAGE_SIZE), c_int(window), c_float(scale), c_int(n_splits),
-        c_int(chunk), c_float(softcap), _stream(),
+        c_int(chunk), c_float(softcap), *_bias_args(bias, num_heads, "flash_mix_decode"), _stream(),
     )
     _check(lib, rc, "flash_mix_decode", kernels=2)
     return out

@@ -1,3 +1,3 @@
 """Architectures.  Importing this package registers them."""
 
-from . import fakelorn, llama, namalix, revirax, tefavik, vezatar  # noqa: F401
+from . import damadra, fakelorn, llama, namalix, revirax, tefavik, vezatar  # noqa: F401

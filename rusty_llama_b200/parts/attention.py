@@ -12,7 +12,7 @@ from ..kernels import ops
 from ..kernels.device import sm_count
 from ..kernels.linear import linear, linear_to_stream
 from ..spec import PartSpec
-from .base import MIXERS, POSITIONS, KVNeed, Mixer, ParamInfo
+from .base import MIXERS, POSITIONS, KVNeed, Mixer, ParamInfo, PositionEncoding
 
 # one-warp blocks of the decode kernel that an SM holds at once (four at head size 128, its shared
 # memory's limit): measured best when the splits fill the GPU once and no more
@@ -70,12 +70,18 @@ class Attention(Mixer):
     head_bias (bool: one learned number per head, added to the score; with logistic weights only), gate "head" (one gate number
     per head instead of one per value: Wg is [H, d]), value_mix (None, or {"key": a name, "role": "source" or "mix"}: the
     "source" layer leaves the values it projected for the step's tokens under that name, a "mix" layer stores and attends to
-    (1 - lambda) v + lambda v_source, lambda a learned number; both kinds of layer have the tensor), names (tensor names after the
+    (1 - lambda) v + lambda v_source, lambda a learned number; both kinds of layer have the tensor), qk_norm_span ("head", or "all":
+    the norm is taken over all q heads at once and over all k heads at once, with a weight for every number of the projection),
+    values ("own", or "keys": the values are the keys as projected, before their norm; no tensor of their own), q_temperature (None, or
+    (coef, every): the queries at position p are multiplied by 1 + coef ln(floor((p + 1) / every) + 1) after their norm), own_kv (bool,
+    default true; false: the layer has queries only and reads the keys and values of the run that the schedule names), names (tensor names after the
     prefix, keys q k v o gate sink head_mix q_bias k_bias v_bias o_bias q_norm k_norm head_bias value_mix).
     tensors: <prefix>q_proj.weight [H hd, d], k_proj.weight [K hd, d], v_proj.weight [K vd, d],
              o_proj.weight [d, H vd]; with the options also g [H vd, d], sink [H], talk [H, H] and the biases.
              q, k, v (and the gate) are kept as one matrix so that one product
              serves them all (src/backend/cuda.rs:423-442).
+
+    A position encoding with a `score_bias` (a learned bias by head and distance) is one of the options.
 
     A plain attention, with or without a sink, runs on the kernels built for it (tensor-core prompt attention, TMA-fed
     decode attention, the rotation fused with the cache write or with the decode kernel).  With any other option (and with a
@@ -101,6 +107,14 @@ class Attention(Mixer):
         self.qk_norm_eps = None if qk_norm is None else float(qk_norm)
         self.softcap = float(spec.params.get("softcap", 0.0) or 0.0)
         self.chunk = int(spec.params.get("chunk", 0) or 0)
+        span, values = spec.params.get("qk_norm_span", "head"), spec.params.get("values", "own")
+        if span not in ("head", "all") or values not in ("own", "keys"):
+            raise ConfigError(f"attention: a norm over '{span}' or values '{values}' are not built (known: head, all; own, keys)")
+        self.norm_whole, self.v_from_k = span == "all" and self.qk_norm_eps is not None, values == "keys"
+        self.q_temperature = spec.params.get("q_temperature")
+        self.own_kv = bool(spec.params.get("own_kv", True))
+        if self.v_from_k and self.vd != self.hd:
+            raise ConfigError(f"attention: values that are the keys have their size, not {self.vd} beside {self.hd}")
         if self.softcap < 0 or self.chunk < 0:
             raise ConfigError(f"attention: softcap {self.softcap} and chunk {self.chunk} must not be negative")
         self.has_mix = bool(spec.params.get("head_mix", False))
@@ -132,6 +146,12 @@ class Attention(Mixer):
         plain = self.vd == self.hd and not (self.has_mix or self.has_gate or self.has_bias) and self.out_scale == 1.0 and magnitude == 1.0
         plain = plain and not (self.zero_sink or self.qk_norm_eps is not None or self.softcap or self.chunk)
         plain = plain and not (self.logistic or self.value_mix is not None) and self.maps == 1
+        self.has_score_bias = type(self.position).score_bias is not PositionEncoding.score_bias
+        plain = plain and not (self.has_score_bias or self.v_from_k or self.q_temperature is not None) and self.own_kv
+        if self.logistic and self.has_score_bias:
+            raise ConfigError("attention: a score bias beside logistic weights is not built")
+        if (self.v_from_k or not self.own_kv) and (self.has_bias or self.value_mix is not None):
+            raise ConfigError("attention: biases or value mixing in a layer without values of its own are not built")
         if self.logistic and (self.has_sink or self.zero_sink):
             raise ConfigError("attention: logistic weights have no denominator for a sink to join")
         if self.value_mix is not None and self.has_bias:
@@ -154,6 +174,10 @@ class Attention(Mixer):
                 f"(a float32 run takes any head size up to 256)")
         self.scale = float(spec.params.get("scale") or 1.0 / math.sqrt(self.hd))
         self.qd, self.kvd, self.vvd, self.od = self.H * self.hd, self.K * self.hd, self.K * self.vd, self.H * self.vd
+        if self.v_from_k:
+            self.vvd = 0  # columns of the projection's rows, as the two below
+        if not self.own_kv:
+            self.kvd = self.vvd = 0
         self.gd = self.H if self.head_gate else self.od  # rows of the gate's matrix
         self.head_bias = self.v_lambda = None
         self.w_qkv = None
@@ -162,6 +186,8 @@ class Attention(Mixer):
         self.fold_matrix = None  # what `fold_queries` mixes by in a decode step: the mixing matrix, or the identity
 
     def cache_need(self):
+        if not self.own_kv:
+            return None
         return KVNeed(self.K, self.hd, self.window, value_dim=self.vd if self.vd != self.hd else None, chunk=self.chunk)
 
     def children(self):
@@ -171,10 +197,12 @@ class Attention(Mixer):
         p, n = self.prefix, self.names
         infos = {
             p + n["q"]: ParamInfo((self.qd, self.d)),
-            p + n["k"]: ParamInfo((self.kvd, self.d)),
-            p + n["v"]: ParamInfo((self.vvd, self.d)),
             p + n["o"]: ParamInfo((self.d, self.od)),
         }
+        if self.own_kv:
+            infos[p + n["k"]] = ParamInfo((self.kvd, self.d))
+            if not self.v_from_k:
+                infos[p + n["v"]] = ParamInfo((self.vvd, self.d))
         if self.has_gate:
             infos[p + n["gate"]] = ParamInfo((self.gd, self.d))
         if self.has_head_bias:
@@ -184,8 +212,9 @@ class Attention(Mixer):
         if self.has_sink and not self.zero_sink:
             infos[p + n["sink"]] = ParamInfo((self.H,), "scalars")
         if self.qk_norm_eps is not None:
-            infos[p + n["q_norm"]] = ParamInfo((self.hd,), "scalars", centre=1.0)
-            infos[p + n["k_norm"]] = ParamInfo((self.hd,), "scalars", centre=1.0)
+            infos[p + n["q_norm"]] = ParamInfo((self.qd if self.norm_whole else self.hd,), "scalars", centre=1.0)
+            if self.own_kv:
+                infos[p + n["k_norm"]] = ParamInfo((self.kvd if self.norm_whole else self.hd,), "scalars", centre=1.0)
         if self.has_mix:
             infos[p + n["head_mix"]] = ParamInfo((self.H, self.H), "scalars")
         if self.has_bias:
@@ -196,7 +225,11 @@ class Attention(Mixer):
 
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
         p, n = self.prefix, self.names
-        parts = [tensors[p + n["q"]], tensors[p + n["k"]], tensors[p + n["v"]]]
+        parts = [tensors[p + n["q"]]]
+        if self.own_kv:
+            parts.append(tensors[p + n["k"]])
+            if not self.v_from_k:
+                parts.append(tensors[p + n["v"]])
         if self.has_gate:
             parts.append(tensors[p + n["gate"]])
         self.w_qkv = torch.cat(parts, dim=0).contiguous()
@@ -206,7 +239,8 @@ class Attention(Mixer):
         elif self.has_sink:
             self.sink = tensors[p + n["sink"]].contiguous()
         if self.qk_norm_eps is not None:
-            self.w_q_norm, self.w_k_norm = tensors[p + n["q_norm"]].contiguous(), tensors[p + n["k_norm"]].contiguous()
+            self.w_q_norm = tensors[p + n["q_norm"]].contiguous()
+            self.w_k_norm = tensors[p + n["k_norm"]].contiguous() if self.own_kv else None
         if self.has_mix:
             self.mix = tensors[p + n["head_mix"]].contiguous()
         if self.has_head_bias:
@@ -226,8 +260,8 @@ class Attention(Mixer):
         return linear_to_stream(a, w_o)
 
     def _forward_extended(self, xn: torch.Tensor, step, cache, shared_cache: bool, out):
-        if shared_cache:
-            raise ConfigError("attention: a layer that reads another layer's cache cannot have this mixer's options")
+        if shared_cache == self.own_kv:
+            raise ConfigError("attention: with this mixer's options a layer reads another layer's cache if, and only if, it has no keys and values of its own")
         proj = linear(xn, self.w_qkv)
         inv_freq, rotary_dim, interleaved, magnitude = self.rotation
         v_src = None
@@ -241,8 +275,9 @@ class Attention(Mixer):
                     raise ConfigError(f"attention: no values '{key}' of {self.vvd} numbers a token were left by an earlier layer of this step")
         ops.qkv_prep(
             proj, self.b_in, step.tok_pos, step.tok_seq, cache.block_table, cache.k_pages, cache.v_pages, inv_freq, magnitude,
-            self.H, self.K, self.hd, self.vd, rotary_dim, interleaved, q_norm=self.w_q_norm, k_norm=self.w_k_norm,
-            norm_eps=self.qk_norm_eps or 0.0, v_src=v_src, v_lambda=self.v_lambda if v_src is not None else None,
+            self.H, self.K if self.own_kv else 0, self.hd, self.vd, rotary_dim, interleaved, q_norm=self.w_q_norm, k_norm=self.w_k_norm,
+            norm_eps=self.qk_norm_eps or 0.0, v_src=v_src, v_lambda=self.v_lambda if v_src is not None else None, norm_whole=self.norm_whole,
+            v_from_k=self.v_from_k and self.own_kv, temperature=self.q_temperature,
         )
         gate = proj[:, self.qd + self.kvd + self.vvd :] if self.has_gate else None
         return self._attend(proj, gate, step, cache, out), self.w_o
@@ -253,6 +288,7 @@ class Attention(Mixer):
         128, no mixed scores, no gate), else the tensor-core kernel for unequal sizes, mixed scores and gates; 32-bit runs and
         the remaining sizes take the general kernel."""
         bf = self.rt.dtype == torch.bfloat16
+        bias = self.position.score_bias()
         if self.logistic:
             return self._attend_logistic(proj, gate, step, cache, out)
         if (bf and self.hd == self.vd and self.hd in ops.FLASH_TC_HEAD_DIMS and not self.has_mix and gate is None and self.out_scale == 1.0
@@ -266,13 +302,13 @@ class Attention(Mixer):
                 a = ops.attn_decode(
                     proj, cache.k_pages, cache.v_pages, cache.block_table, step.seq_len, self.H, self.K, self.hd, n_splits, scratch,
                     window=self.window, scale=self.scale, sink=self.sink, chunk=self.chunk, softcap=self.softcap, impl="tma",
-                    out=out if direct else None,
+                    out=out if direct else None, bias=bias,
                 )
             else:
                 a = ops.flash_prefill_tc(
                     proj, cache.k_pages, cache.v_pages, cache.block_table, step.seq_start, step.seq_pos0, step.max_q_len, self.H, self.K,
                     self.hd, window=self.window, scale=self.scale, sink=self.sink, chunk=self.chunk, softcap=self.softcap,
-                    out=out if direct else None, maps=self.maps,
+                    out=out if direct else None, maps=self.maps, bias=bias,
                 )
             if out is not None and a is not out:
                 out.copy_(a)
@@ -295,7 +331,7 @@ class Attention(Mixer):
                 return ops.flash_mix_decode(
                     qf, cache.k_pages, cache.v_pages, cache.block_table, step.seq_pos0, self.H, self.K, self.hd, self.vd, self.scale,
                     n_splits, scratch, window=self.window, sink=self.sink, gate=gate, out_scale=self.out_scale, out=out, chunk=self.chunk,
-                    softcap=self.softcap,
+                    softcap=self.softcap, bias=bias,
                 )
             # the tensor-core kernel for prompts (and single tokens of sizes the decode kernel does not take); mixed scores come
             # from folded queries
@@ -303,12 +339,12 @@ class Attention(Mixer):
             return ops.flash_mix(
                 q, cache.k_pages, cache.v_pages, cache.block_table, step.seq_start, step.seq_pos0, step.max_q_len, self.H, self.K,
                 self.hd, self.vd, self.scale, window=self.window, sink=self.sink, folded=self.has_mix, gate=gate, out_scale=self.out_scale,
-                out=out, chunk=self.chunk, softcap=self.softcap, maps=self.maps,
+                out=out, chunk=self.chunk, softcap=self.softcap, maps=self.maps, bias=bias,
             )
         return ops.attn_ext(
             proj, cache.k_pages, cache.v_pages, cache.block_table, step.tok_seq, step.tok_pos, self.H, self.K, self.hd, self.vd,
             self.scale, window=self.window, sink=self.sink, mix=self.mix, gate=gate, out_scale=self.out_scale, out=out, chunk=self.chunk,
-            softcap=self.softcap, maps=self.maps,
+            softcap=self.softcap, maps=self.maps, bias=bias,
         )
 
     def _attend_logistic(self, proj: torch.Tensor, gate, step, cache, out):
@@ -397,7 +433,7 @@ class Attention(Mixer):
 
 
 def chunked_attention_runner(proj, k_pages, v_pages, block_table, step, num_heads: int, num_kv_heads: int, kdim: int, vdim: int, scale: float,
-                             chunk: int, softcap: float, sink, window: int = 0, workspace=None):
+                             chunk: int, softcap: float, sink, window: int = 0, workspace=None, bias=None):
     """A callable that runs the attention of `Attention` (the kernel choice included) over ready rows, for timing it alone.
     step: tok_seq, tok_pos, seq_start, seq_pos0, seq_len (or none: positions after the step), max_q_len, n_seqs, decode_only."""
     from types import SimpleNamespace
@@ -419,7 +455,7 @@ def chunked_attention_runner(proj, k_pages, v_pages, block_table, step, num_head
     part = SimpleNamespace(
         rt=SimpleNamespace(dtype=proj.dtype, workspace=workspace or _Scratch()), H=num_heads, K=num_kv_heads, hd=kdim, vd=vdim, scale=scale,
         window=window, chunk=chunk, softcap=softcap, sink=sink, mix=None, has_mix=False, out_scale=1.0, fold_matrix=None, logistic=False, maps=1,
-        qd=num_heads * kdim, kvd=num_kv_heads * kdim, vvd=num_kv_heads * vdim,
+        qd=num_heads * kdim, kvd=num_kv_heads * kdim, vvd=num_kv_heads * vdim, position=SimpleNamespace(score_bias=lambda: bias),
     )
     cache = SimpleNamespace(k_pages=k_pages, v_pages=v_pages, block_table=block_table)
     return lambda: Attention._attend(part, proj, None, step, cache, None)

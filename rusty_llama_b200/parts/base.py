@@ -265,6 +265,11 @@ class PositionEncoding(Part):
         leave `write_qk` out of a decode step and have its attention kernel do the same work."""
         return None
 
+    def score_bias(self) -> Optional[torch.Tensor]:
+        """None, or float32 [H, L]: the score of head h for a key n positions behind its query is raised by
+        table[h, min(n, L - 1)].  Only a mixer that knows how to add it takes such an encoding."""
+        return None
+
     def write_qk(self, qkv: torch.Tensor, step, kv, num_heads: int, num_kv_heads: int, head_dim: int, write_kv: bool) -> None:
         from ..kernels import ops
 

@@ -9,7 +9,8 @@ import torch
 from ..kernels import ops
 from ..kernels.linear import STREAM_MAX_ROWS, linear, linear_to_stream
 from ..errors import ConfigError
-from .base import BLOCKS, Block, ParamInfo, ResidualStream
+from ..spec import PartSpec
+from .base import BLOCKS, NORMS, Block, ParamInfo, ResidualStream
 
 
 def _fold_enabled() -> bool:
@@ -103,6 +104,31 @@ class SandwichBlock(Block):
             return
         xn = self.norms["feed_forward"].forward(stream)
         stream.add(self.feed_forward.forward(xn, step), norm=self.norms["feed_forward_out"].rms_weight())
+
+
+@BLOCKS.register("postnorm")
+class PostNormBlock(Block):
+    """x += norm_m(mixer(x)); x += norm_f(feed_forward(x)): the sublayers read the stream as it is and only their results are normed
+    (a constant factor on a result is part of its norm's weight: `factor`).  norms: "mixer_out", and with a feed-forward
+    "feed_forward_out", both RMS norms.
+
+    A sublayer's result stays pending on the stream together with its norm; one pass then norms it, adds it and hands the sum on
+    in the activation type."""
+
+    def __init__(self, spec, runtime, mixer, feed_forward, norms):
+        super().__init__(spec, runtime, mixer, feed_forward, norms)
+        for name in ["mixer_out"] + (["feed_forward_out"] if feed_forward is not None else []):
+            if name not in self.norms or self.norms[name].rms_weight() is None:
+                raise ConfigError(f"postnorm block: no RMS norm '{name}'")
+        self.read = NORMS.build(PartSpec("identity"), runtime)
+
+    def forward(self, stream: ResidualStream, step, cache, shared_cache: bool = False) -> None:
+        x = self.read.forward(stream)
+        stream.add_result(self.mixer.forward(x, step, cache, shared_cache), norm=self.norms["mixer_out"].rms_weight(), bias=self.mixer.output_bias())
+        if self.feed_forward is None:
+            return
+        x = self.read.forward(stream)
+        stream.add(self.feed_forward.forward(x, step), norm=self.norms["feed_forward_out"].rms_weight())
 
 
 @BLOCKS.register("shared_norm")

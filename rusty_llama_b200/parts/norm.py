@@ -1,4 +1,4 @@
-"""RMSNorm, fused with the residual sum that precedes it."""
+"""RMSNorm, fused with the residual sum that precedes it, and the arrangement's way to have no norm there."""
 
 from __future__ import annotations
 
@@ -19,14 +19,16 @@ class RMSNorm(Norm):
     the stored tensor is the weight's distance from `offset`, y = ... * (offset + w); such a weight is kept in 32-bit whatever
     the run's type, since offset + w has more digits than w), float32 (optional bool: the weight is kept in 32-bit in every run,
     for designs whose norms are 32-bit arithmetic throughout), groups (optional, default 1: the row is cut into that many equal
-    consecutive parts and each is divided by its own root mean square).  tensor: <prefix>weight [size]."""
+    consecutive parts and each is divided by its own root mean square), factor (optional, default 1: a constant that the weight is
+    multiplied by at load; such a weight is kept in 32-bit too).  tensor: <prefix>weight [size]."""
 
     def __init__(self, spec, runtime):
         super().__init__(spec, runtime)
         self.size = int(self._param("size"))
         self.eps = float(self._param("eps"))
         self.offset = float(spec.params.get("offset", 0.0))
-        self.keep32 = bool(spec.params.get("float32", False))
+        self.factor = float(spec.params.get("factor", 1.0))
+        self.keep32 = bool(spec.params.get("float32", False)) or self.factor != 1.0
         self.tensor_name = self.prefix + str(spec.params.get("name", "weight"))
         self.groups = int(spec.params.get("groups", 1))
         if self.groups < 1 or self.size % self.groups:
@@ -44,6 +46,8 @@ class RMSNorm(Norm):
         self.weight = tensors[self.tensor_name]
         if self.offset:
             self.weight = (self.weight.to(torch.float32) + self.offset).contiguous()
+        if self.factor != 1.0:
+            self.weight = self.weight * self.factor
 
     def rms_weight(self):
         return (self.weight, self.eps) if self.groups == 1 else None
@@ -62,3 +66,20 @@ class RMSNorm(Norm):
         return ops.add_rmsnorm(
             stream.x, delta, self.weight, self.eps, stream.act_dtype, rows=rows, write_x=rows is None
         )
+
+
+@NORMS.register("identity")
+class NoNorm(Norm):
+    """y = x in the activation type: for sublayers that read the stream as it is.  What is pending on the stream is added (through its
+    own norm, if it has one) in the same pass.  No params, no tensors."""
+
+    def forward(self, stream: ResidualStream, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        delta, delta_norm, gate = stream.take_pending()
+        if gate is not None:
+            stream.add(delta, gate=gate)
+            stream.flush()
+            delta = None
+        if delta_norm is not None:
+            return ops.normed_add_rmsnorm(stream.x, delta, delta_norm[0], delta_norm[1], None, 0.0, stream.act_dtype, rows=rows,
+                                          write_x=rows is None, delta_bias=delta_norm[2], plain_out=True)
+        return ops.add_rmsnorm(stream.x, delta, None, 0.0, stream.act_dtype, rows=rows, write_x=rows is None and delta is not None, plain_out=True)

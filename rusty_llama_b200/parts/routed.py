@@ -1,4 +1,4 @@
-"""A feed-forward that sends each token to a few of many small gated feed-forwards."""
+"""A feed-forward that sends each token to a few of many small feed-forwards."""
 
 from __future__ import annotations
 
@@ -35,11 +35,16 @@ class RoutedExperts(FeedForward):
     activation "clamped_swish" (params `limit`, `alpha`): f_e(x) = W_down[e] (g s(alpha g) (u + 1)) with g = min(W_gate[e] x, limit),
     u = clamp(W_up[e] x, -limit, limit), s the logistic function, in the place of silu(g) * u.
 
+    activation "relu2": experts without a gate, f_e(x) = W_down[e] relu(W_up[e] x)^2 (no gate tensors).
+
+    identity (default 0): the router scores that many choices more, behind the E experts; such a choice has no tensors, and its
+    output is x itself (times its weight).
+
     params: hidden_size, n_experts, top, expert_ff, bias (bool), renormalize (bool),
             shared_ff (0: none), shared_gate (bool), router ("softmax", "sigmoid" or "table"; with "table" also vocab_size), renorm_eps,
             weight_scale, activation
-            ("silu" or "clamped_swish"), names (optional).
-    tensors: <prefix>e<i>.gate [ff, d], e<i>.up [ff, d], e<i>.down [d, ff], router [E, d] (or table [vocab, top]), correction [E],
+            ("silu", "clamped_swish" or "relu2"), identity, names (optional).
+    tensors: <prefix>e<i>.gate [ff, d], e<i>.up [ff, d], e<i>.down [d, ff], router [E + identity, d] (or table [vocab, top]), correction [E + identity],
              shared.gate / shared.up / shared.down, shared.sg [1, d]."""
 
     def __init__(self, spec, runtime):
@@ -63,11 +68,18 @@ class RoutedExperts(FeedForward):
             if self.has_bias or self.renormalize or self.shared_gate:
                 raise ConfigError("routed_experts: a table chooses without scores; bias, renormalize and a gated shared expert need a router")
         activation = spec.params.get("activation", "silu")
-        if activation not in ("silu", "clamped_swish"):
-            raise ConfigError(f"routed_experts: activation '{activation}' is not built (only 'silu' and 'clamped_swish')")
+        if activation not in ("silu", "clamped_swish", "relu2"):
+            raise ConfigError(f"routed_experts: activation '{activation}' is not built (only 'silu', 'clamped_swish' and 'relu2')")
+        self.gated = activation != "relu2"
         self.act = (float(self._param("alpha")), float(self._param("limit"))) if activation == "clamped_swish" else None
-        if not 0 < self.top <= self.E:
-            raise ConfigError(f"routed_experts: {self.top} of {self.E} experts per token")
+        self.identity = int(spec.params.get("identity", 0))
+        self.choices = self.E + self.identity  # what the router scores
+        if self.identity < 0 or (self.identity and self.router == "table"):
+            raise ConfigError(f"routed_experts: {self.identity} identity choices (a table names experts only)")
+        if not self.gated and self.shared_ff:
+            raise ConfigError("routed_experts: a shared expert beside experts without a gate is not built")
+        if not 0 < self.top <= self.choices:
+            raise ConfigError(f"routed_experts: {self.top} of {self.choices} experts per token")
         if self.ff <= 0:
             raise ConfigError(f"routed_experts: expert size {self.ff}")
 
@@ -80,15 +92,16 @@ class RoutedExperts(FeedForward):
     def param_infos(self) -> Dict[str, ParamInfo]:
         infos = {}
         for i in range(self.E):
-            infos[self._expert(i, "gate")] = ParamInfo((self.ff, self.d))
+            if self.gated:
+                infos[self._expert(i, "gate")] = ParamInfo((self.ff, self.d))
             infos[self._expert(i, "up")] = ParamInfo((self.ff, self.d))
             infos[self._expert(i, "down")] = ParamInfo((self.d, self.ff))
         if self.router == "table":
             infos[self.prefix + self.names["table"]] = ParamInfo((self.vocab, self.top), "table", upper=self.E)
         else:
-            infos[self.prefix + self.names["router"]] = ParamInfo((self.E, self.d), "scalars")
+            infos[self.prefix + self.names["router"]] = ParamInfo((self.choices, self.d), "scalars")
         if self.has_bias:
-            infos[self.prefix + self.names["bias"]] = ParamInfo((self.E,), "scalars")
+            infos[self.prefix + self.names["bias"]] = ParamInfo((self.choices,), "scalars")
         if self.shared_ff:
             infos[self._shared("gate")] = ParamInfo((self.shared_ff, self.d))
             infos[self._shared("up")] = ParamInfo((self.shared_ff, self.d))
@@ -99,7 +112,8 @@ class RoutedExperts(FeedForward):
 
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
         stack = lambda which: torch.stack([tensors[self._expert(i, which)] for i in range(self.E)], dim=0).contiguous()  # noqa: E731
-        self.w_gate, self.w_up, self.w_down = stack("gate"), stack("up"), stack("down")
+        self.w_gate = stack("gate") if self.gated else None
+        self.w_up, self.w_down = stack("up"), stack("down")
         if self.router == "table":
             self.table = tensors[self.prefix + self.names["table"]].contiguous()
             if self.table.numel() and (int(self.table.min()) < 0 or int(self.table.max()) >= self.E):
@@ -125,7 +139,7 @@ class RoutedExperts(FeedForward):
             ids, weights = ops.moe_table_lookup(step.tokens, self.table, self.E)
             gate = None
         else:
-            ids, weights, gate = ops.moe_router(xn, self.w_router, self.bias, self.E, self.top, self.renormalize,
+            ids, weights, gate = ops.moe_router(xn, self.w_router, self.bias, self.choices, self.top, self.renormalize,
                                                 logistic=self.router == "sigmoid", renorm_eps=self.renorm_eps, weight_scale=self.weight_scale)
         # the height of a row tile: 128 once the experts get that many rows on average (a prompt step), else 32; the plain
         # kernels of a 32-bit run have their own
@@ -133,7 +147,10 @@ class RoutedExperts(FeedForward):
         if xn.dtype == torch.bfloat16 and self.d % 8 == 0 and self.ff % 8 == 0:  # (else the plain products, 16-byte rows or not)
             tile_rows = 128 if T * self.top >= 64 * self.E else 32
         order, place, tiles, max_tiles = ops.moe_plan(ids, self.E, tile_rows)
-        h = ops.moe_gemm(xn, self.w_gate, tiles, max_tiles, T * self.top, order=order, gather_div=self.top, w2=self.w_up, tile_rows=tile_rows, act=self.act)
+        if self.gated:
+            h = ops.moe_gemm(xn, self.w_gate, tiles, max_tiles, T * self.top, order=order, gather_div=self.top, w2=self.w_up, tile_rows=tile_rows, act=self.act)
+        else:
+            h = ops.moe_gemm(xn, self.w_up, tiles, max_tiles, T * self.top, order=order, gather_div=self.top, tile_rows=tile_rows, act="relu2")
         y = ops.moe_gemm(h, self.w_down, tiles, max_tiles, T * self.top, out_dtype=torch.float32, tile_rows=tile_rows)
         shared = None
         if self.shared_ff:
@@ -144,4 +161,4 @@ class RoutedExperts(FeedForward):
             else:
                 hs = ops.swiglu(linear(xn, self.ws_gate_up))
             shared = linear(hs, self.ws_down)
-        return ops.moe_combine(y, place, weights, shared, gate)
+        return ops.moe_combine(y, place, weights, shared, gate, x=xn if self.identity else None)
