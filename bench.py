@@ -2,7 +2,7 @@
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference] [--reps R]
     python bench.py --sizes 1b|13b --workload
-    python bench.py --design vezatar|revirax|tefavik|namalix|fakelorn [--design-sizes small,lite,wide]
+    python bench.py --design vezatar|revirax|tefavik|namalix|fakelorn|damadra [--design-sizes small,lite,wide]
 
 The default run has the layer sizes of Llama-3.1-8B with random
 bfloat16 weights, a batch of 8 sequences and a context of 4096.  A step is one decode step of the
@@ -474,7 +474,7 @@ def main() -> int:
     ap.add_argument("--reps", type=int, default=5, help="repetitions of the timed steps (mean and standard deviation are reported)")
     ap.add_argument("--no-kernels", action="store_true", help="leave out the kernel-by-kernel table")
     ap.add_argument("--workload", action="store_true", help="with --sizes 1b or 13b: BASELINE.json's workload of unequal prompts through LLM.generate, instead of the contract line")
-    ap.add_argument("--design", default="", choices=["", "vezatar", "revirax", "tefavik", "namalix", "fakelorn"], help="instead of the default line: this design beside Llama (Tefavik and Namalix: beside Revirax; Fakelorn: beside Vezatar) at equal sizes (prompt and decode steps through the engine, and its kernels alone)")
+    ap.add_argument("--design", default="", choices=["", "vezatar", "revirax", "tefavik", "namalix", "fakelorn", "damadra"], help="instead of the default line: this design beside Llama (Tefavik and Namalix: beside Revirax; Fakelorn: beside Vezatar; Damadra: beside both) at equal sizes (prompt and decode steps through the engine, and its kernels alone)")
     ap.add_argument("--design-sizes", default="small,lite", help="with --design: which of the sizes small, lite, wide")
     ap.add_argument("--design-tokens", type=int, default=2048, help="with --design: tokens of the prompt step, and the context of the decode steps")
     args = ap.parse_args()
@@ -487,6 +487,8 @@ def main() -> int:
             from rusty_llama_b200.kernels import namalix_bench as design_bench
         elif args.design == "fakelorn":
             from rusty_llama_b200.kernels import fakelorn_bench as design_bench
+        elif args.design == "damadra":
+            from rusty_llama_b200.kernels import damadra_bench as design_bench
         else:
             from rusty_llama_b200.kernels import design_bench
 
