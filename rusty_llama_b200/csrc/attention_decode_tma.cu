@@ -25,8 +25,8 @@
 // eight product warps.  At head size 64 a page's keys and values are half as many bytes, so the ring
 // has six stages instead of three and the same bytes are in flight.
 //
-// A learned bias by head and distance (`rl_distance_bias`): a thread's four scores of a page need four numbers, asked for before
-// the page is waited for; beyond the last distance with a number of its own they are two registers.
+// A learned bias by head and distance (`rl_distance_bias`): a thread's four scores of a page need four numbers, asked for a page
+// ahead (the first page's before the kernel before this one has ended: a weight is not waited for); beyond the last distance with a number of its own they are two registers.
 //
 // Every mbarrier wait is bounded; on expiry a code goes to status[0] and the block drains.
 #include "tc_common.cuh"
@@ -206,9 +206,27 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
       bars.sn[j] = sn;
     }
   }
+  const int g = lane >> 2, t4 = lane & 3;
+  const float* bias_rows[2] = {bias, bias};
+  float far_bias[2] = {0.f, 0.f};
+  if (bias != nullptr) {  // (a column past the group's last head reads that head's numbers and is not stored)
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      bias_rows[j] += (size_t)(h0 + min(2 * t4 + j, n_heads - 1)) * bias_len;
+      far_bias[j] = bias_rows[j][bias_len - 1] * 1.4426950408889634f;
+    }
+  }
+  float score_bias[4];  // of the next page: (key g [+8], head 2*t4 [+1]), base-2 exponents
+  auto ask_bias = [&](int tile) {
+    const int at = pos - (tile * PAGE + warp * 16 + g);
+    const bool near = bias != nullptr && pos - (tile * PAGE + warp * 16 + 15) < bias_len - 1;
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+      score_bias[e] = near ? rl_distance_bias(bias_rows[e & 1], bias_len, at - 8 * (e >> 1)) * 1.4426950408889634f : far_bias[e & 1];
+  };
+  ask_bias(my_lo);
   pdl_wait();  // the queries are the previous kernel's output, and it may still read this one's scratch
   // ---------------- products
-  const int g = lane >> 2, t4 = lane & 3;
   {
     // this block's queries: HEADS rows of HD values, 16 bytes per thread
     constexpr int PIECES = HD / 8;
@@ -321,25 +339,10 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
       }
     }
   }
-  const float* bias_rows[2] = {bias, bias};
-  float far_bias[2] = {0.f, 0.f};
-  if (bias != nullptr) {  // (a column past the group's last head reads that head's numbers and is not stored)
-#pragma unroll
-    for (int j = 0; j < 2; ++j) {
-      bias_rows[j] += (size_t)(h0 + min(2 * t4 + j, n_heads - 1)) * bias_len;
-      far_bias[j] = bias_rows[j][bias_len - 1] * 1.4426950408889634f;
-    }
-  }
   bool ok = true;
   int done = 0;
   for (int tile = my_lo; tile <= my_hi && ok; ++tile, ++done) {
     const int st = done % STAGES;
-    float score_bias[4] = {far_bias[0], far_bias[1], far_bias[0], far_bias[1]};  // (key g [+8], head 2*t4 [+1]), base-2 exponents
-    if (bias != nullptr && pos - (tile * PAGE + warp * 16 + 15) < bias_len - 1) {
-#pragma unroll
-      for (int e = 0; e < 4; ++e)
-        score_bias[e] = rl_distance_bias(bias_rows[e & 1], bias_len, pos - (tile * PAGE + warp * 16 + g + 8 * (e >> 1))) * 1.4426950408889634f;
-    }
     if (!mbar_wait_role(&bars.full[st], (done / STAGES) & 1, ctl, 52)) {
       if (lane == 0) {
         give_up_code(status, 52);
@@ -426,6 +429,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
       s_acc[e] = v;
       tmax[e & 1] = fmaxf(tmax[e & 1], v);
     }
+    ask_bias(tile + 1);  // (a page past the range reads the smallest distance's number and is not used)
     float alpha[2], m_use[2];
 #pragma unroll
     for (int j = 0; j < 2; ++j) {

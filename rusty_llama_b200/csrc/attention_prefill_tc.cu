@@ -51,9 +51,11 @@
 // tokens has too few blocks for two per SM and pays for the short tiles: 12.3 us against 10.5.
 // Softmax statistics, the accumulator and the final division are 32-bit.
 //
-// A learned bias by head and distance (`rl_distance_bias`): the head's numbers lie in shared memory (times log2 e; in global
-// memory where they do not fit beside the tiles), neighbouring rows of a tile read neighbouring ones.  A tile that lies wholly
-// beyond the last distance with a number of its own adds one number to every score, which goes into the exponent's constant.
+// A learned bias by head and distance (`rl_distance_bias`): the head's numbers lie in shared memory, in units of the raw scores and
+// with room on both sides for every distance of a tile that is not far, so that a thread's 64 loads have constant offsets and
+// neighbouring rows read neighbouring numbers (a table that does not fit beside the tiles is read from global memory instead).  A
+// tile that lies wholly beyond the last distance with a number of its own adds one number to every score, which goes into the
+// exponent's constant.
 //
 // Every mbarrier wait is bounded; on expiry a code goes to status[0] and the block drains.
 #include "tc_common.cuh"
@@ -72,7 +74,12 @@ RL_DEFINE_ERROR_TEXT()
 #define O_COL 128
 #define RESCALE_THRESHOLD 8.0f          // in base-2 exponents
 #define SMALL_BYTES 512
-#define BIAS_SMEM_FLOATS(HD) ((113 * 1024 - SMEM_NEEDED(HD)) / 4)  // what is left of half an SM's shared memory
+// Distances in a tile that is not far lie between -(BMQ + BNK) and bias_len + BMQ + BNK: that much room on both sides of the table.
+#define BIAS_PAD (BMQ + BNK)
+#define BIAS_SMEM_FLOATS(HD) ((113 * 1024 - SMEM_NEEDED(HD)) / 4 - 2 * BIAS_PAD)  // what is left of half an SM's shared memory
+#define BIAS_NONE 0
+#define BIAS_SMEM 1
+#define BIAS_GLOBAL 2
 // Q is HD / 64 sub-tiles of 16 KB; a K or V tile HD / 64 sub-tiles of 8 KB.  Two blocks must fit an SM and
 // no more (a third would wait for tensor memory): at head size 64 the request is padded to that end.
 #define SMEM_NEEDED(HD) ((HD) / 64 * SUBQ_BYTES + 2 * KV_STAGES * ((HD) / 64) * SUBK_BYTES + SMALL_BYTES)
@@ -221,14 +228,14 @@ __device__ __forceinline__ uint32_t pv_block(uint32_t tmem_o, uint32_t tmem_p, u
 
 // MAPS 2: query heads 2h and 2h + 1 are the two halves of the HD numbers of row h (the values are the same for both); the row's
 // tile is loaded whole and a block's scores use its half of it and of the keys.
-template <int HD, int MAPS, bool BIAS>
+template <int HD, int MAPS, int BIAS>
 __global__ void __launch_bounds__(NUM_THREADS, 2)
 flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                         const __grid_constant__ CUtensorMap map_v, const int* __restrict__ block_table, int table_width,
                         const int* __restrict__ seq_start, const int* __restrict__ seq_pos0, bf16* __restrict__ out,
                         int out_stride, int H, int K, int window, float scale_log2, int* __restrict__ status,
                         int test_role, uint32_t test_ns, const float* __restrict__ sink, int chunk, float softcap,
-                        const float* __restrict__ bias, int bias_len, int bias_in_smem) {
+                        const float* __restrict__ bias, int bias_len) {
   // All shared memory is dynamic, so that the tiles start at the block's first byte (1024-byte
   // aligned, as the 128-byte swizzle needs) and the small items fit behind them.
   constexpr int SUBS = HD / 64, Q_BYTES = SUBS * SUBQ_BYTES, KV_BYTES = SUBS * SUBK_BYTES;
@@ -269,12 +276,14 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   const int lowest_key = rl_first_key(first_pos, window, chunk);
   const int tile_lo = lowest_key / BNK, tile_hi = last_pos / BNK;
   const int n_tiles = tile_hi - tile_lo + 1;
-  const float* bias_row = BIAS ? bias + (size_t)h * bias_len : nullptr;
-  if (BIAS && bias_in_smem) {
-    float* b = reinterpret_cast<float*>(smem_dyn + SMEM_NEEDED(HD));
-    for (int i = threadIdx.x; i < bias_len; i += NUM_THREADS) b[i] = bias_row[i];
-    bias_row = b;
-  }
+  const float* bias_row = BIAS != BIAS_NONE ? bias + (size_t)h * bias_len : nullptr;
+  float* bias_s = reinterpret_cast<float*>(smem_dyn + SMEM_NEEDED(HD));
+  // with a cap c the scores become tanh(raw * scale / c) first, and c log2(e) takes the scale's place from there on
+  const float exp_scale = softcap != 0.f ? softcap * 1.4426950408889634f : scale_log2;
+  const float bias_unit = BIAS != BIAS_NONE ? 1.4426950408889634f / exp_scale : 0.f;  // the bias in units of the scores before exp_scale
+  if (BIAS == BIAS_SMEM)  // (a weight: no kernel writes it)
+    for (int i = threadIdx.x; i < bias_len + 2 * BIAS_PAD; i += NUM_THREADS)
+      bias_s[i] = rl_distance_bias(bias_row, bias_len, i - BIAS_PAD) * bias_unit;
 
   if (threadIdx.x == 0) {
     mbar_init(&q_full, 1);
@@ -415,10 +424,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     const int qpos = first_pos + r;
     const int qlow = rl_first_key(qpos, window, chunk);
     const int last_low = rl_first_key(last_pos, window, chunk);
-    // with a cap c the scores become tanh(raw * scale / c) first, and c log2(e) takes the scale's place from there on
-    const float exp_scale = softcap != 0.f ? softcap * 1.4426950408889634f : scale_log2;
-    const float far_bias = BIAS ? bias_row[bias_len - 1] * 1.4426950408889634f : 0.f;
-    const float bias_unit = BIAS ? 1.4426950408889634f / exp_scale : 0.f;  // the bias in units of the scores before exp_scale
+    const float far_bias = BIAS != BIAS_NONE ? bias_row[bias_len - 1] * 1.4426950408889634f : 0.f;
     const float cap_in = softcap != 0.f ? scale_log2 / exp_scale : 0.f;
     const uint32_t lane_addr = tmem_base + ((uint32_t)(warp * 32) << 16);
     const uint32_t o_addr = lane_addr + O_COL;
@@ -461,14 +467,20 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         for (int i = 0; i < BNK; ++i) v[i] = __float_as_uint(rl_tanh_sfu(__uint_as_float(v[i]) * cap_in));
       }
       float add = 0.f;  // what every score of the tile is raised by, in base-2 exponents
-      if (BIAS) {
+      if (BIAS != BIAS_NONE) {
         if (first_pos - (key0 + BNK - 1) >= bias_len - 1) {
           add = far_bias;
         } else {
           const int gap = qpos - key0;
+          if (BIAS == BIAS_SMEM) {
+            const float* at = bias_s + (gap + BIAS_PAD - (BNK - 1));
 #pragma unroll
-          for (int i = 0; i < BNK; ++i)
-            v[i] = __float_as_uint(fmaf(rl_distance_bias(bias_row, bias_len, gap - i), bias_unit, __uint_as_float(v[i])));
+            for (int i = 0; i < BNK; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) + at[BNK - 1 - i]);
+          } else {
+#pragma unroll
+            for (int i = 0; i < BNK; ++i)
+              v[i] = __float_as_uint(fmaf(rl_distance_bias(bias_row, bias_len, gap - i), bias_unit, __uint_as_float(v[i])));
+          }
         }
       }
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
@@ -573,7 +585,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
 // Head sizes this kernel is built for: 64 and 128 (1 if `hd` is one of them).
 RL_API int rl_flash_prefill_tc_takes(int hd) { return hd == 64 || hd == 128; }
 
-template <int HD, int MAPS, bool BIAS>
+template <int HD, int MAPS, int BIAS>
 static int launch_flash_tc(const void* q, int q_stride, int n_tokens, const void* k_pages, const void* v_pages, int n_pages,
                            const int* block_table, int table_width, const int* seq_start, const int* seq_pos0, void* out,
                            int out_stride, int n_seqs, int max_q_len, int H, int K, int window, float scale, int* status,
@@ -583,16 +595,16 @@ static int launch_flash_tc(const void* q, int q_stride, int n_tokens, const void
     RL_REFUSE(10, "flash_prefill_tc: cannot describe the query tensor to TMA");
   if (make_page_map(&map_k, k_pages, n_pages, K, PAGE, HD, PAGE) || make_page_map(&map_v, v_pages, n_pages, K, PAGE, HD, PAGE))
     RL_REFUSE(11, "flash_prefill_tc: cannot describe the cache pages to TMA");
-  const int bias_in_smem = BIAS && bias_len <= BIAS_SMEM_FLOATS(HD);
   size_t smem = SMEM_BYTES_OF(HD);
-  if (bias_in_smem && SMEM_NEEDED(HD) + (size_t)bias_len * 4 > smem) smem = SMEM_NEEDED(HD) + (size_t)bias_len * 4;
+  const size_t with_bias = SMEM_NEEDED(HD) + (size_t)(bias_len + 2 * BIAS_PAD) * 4;
+  if (BIAS == BIAS_SMEM && with_bias > smem) smem = with_bias;
   auto kern = flash_prefill_tc_kernel<HD, MAPS, BIAS>;
   if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
     RL_REFUSE(12, "flash_prefill_tc: cannot get %zu bytes of shared memory", smem);
   dim3 grid(H * n_seqs, (max_q_len + BMQ - 1) / BMQ);
   RL_LAUNCH_CHECK(rl_launch(kern, grid, NUM_THREADS, smem, stream, map_q, map_k, map_v, block_table, table_width, seq_start, seq_pos0,
                             (bf16*)out, out_stride, H, K, window, scale * 1.4426950408889634f, status, wait_test_role,
-                            (uint32_t)wait_test_ns, sink, chunk, softcap, bias, bias_len, bias_in_smem));
+                            (uint32_t)wait_test_ns, sink, chunk, softcap, bias, bias_len));
   return 0;
 }
 
@@ -625,11 +637,13 @@ RL_API int rl_flash_prefill_tc(const void* q, int q_stride, int n_tokens, const 
   return launch_flash_tc<HDV, MAPSV, BIASV>(q, q_stride, n_tokens, k_pages, v_pages, n_pages, block_table, table_width, seq_start, seq_pos0, out,  \
                                      out_stride, n_seqs, max_q_len, H, K, window, scale, status, wait_test_role, wait_test_ns, sink, chunk, \
                                      softcap, bias, bias_len, stream)
-  if (bias != nullptr && hd == 64) RL_FTC(64, 1, true);
-  if (bias != nullptr) RL_FTC(128, 1, true);
-  if (hd == 64 && maps == 2) RL_FTC(64, 2, false);
-  if (hd == 64) RL_FTC(64, 1, false);
-  if (maps == 2) RL_FTC(128, 2, false);
-  RL_FTC(128, 1, false);
+  if (bias != nullptr && hd == 64 && bias_len <= BIAS_SMEM_FLOATS(64)) RL_FTC(64, 1, BIAS_SMEM);
+  if (bias != nullptr && hd == 64) RL_FTC(64, 1, BIAS_GLOBAL);
+  if (bias != nullptr && bias_len <= BIAS_SMEM_FLOATS(128)) RL_FTC(128, 1, BIAS_SMEM);
+  if (bias != nullptr) RL_FTC(128, 1, BIAS_GLOBAL);
+  if (hd == 64 && maps == 2) RL_FTC(64, 2, BIAS_NONE);
+  if (hd == 64) RL_FTC(64, 1, BIAS_NONE);
+  if (maps == 2) RL_FTC(128, 2, BIAS_NONE);
+  RL_FTC(128, 1, BIAS_NONE);
 #undef RL_FTC
 }

@@ -184,6 +184,18 @@ RL_API int rl_moe_router(const void* x, int ldx, int dtype, const float* w, cons
   return 0;
 }
 
+// The choice alone, from logits that another product made (float32 [n_tokens, E + has_gate]).
+RL_API int rl_moe_choose(const float* logits, const float* bias, int n_tokens, int E, int top, int renorm, int has_gate, int* ids, float* weights,
+                         float* gate, int logistic, float renorm_eps, float weight_scale, cudaStream_t stream) {
+  if (n_tokens <= 0 || E <= 0 || top <= 0 || top > E) RL_REFUSE(1, "moe_choose: T=%d E=%d top=%d", n_tokens, E, top);
+  if (has_gate && gate == nullptr) RL_REFUSE(2, "moe_choose: a gate column but nowhere to write the gate");
+  const size_t smem = (size_t)4 * 2 * E * sizeof(float);
+  if (smem > 48 * 1024) RL_REFUSE(3, "moe_choose: %d experts exceed the kernel's shared memory", E);
+  RL_LAUNCH_CHECK(rl_launch<false>(moe_router_choose_kernel, (n_tokens + 3) / 4, 128, smem, stream, logits, bias, E, E + (has_gate ? 1 : 0), top,
+                                   renorm, n_tokens, ids, weights, gate, logistic, renorm_eps, weight_scale));
+  return 0;
+}
+
 // ---------------------------------------------------------------- plan
 // ids[n] (n = T * top pairs) -> order[n] (pairs laid out expert after expert, each expert's pairs in ascending
 // pair index), place[pair] (its row in that layout), tiles[1 + 3 * max_tiles]: the number of tiles, then
@@ -402,18 +414,68 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
   }
 }
 
+// The same sums, four neighbouring columns a thread and everything a thread needs of eight choices in flight at once.
+#define COMBINE_AHEAD 8
+template <typename TS, typename TO>
+__global__ void __launch_bounds__(256)
+moe_combine_vec_kernel(const float* __restrict__ y, const int* __restrict__ place, const float* __restrict__ weights, int top,
+                       const TS* __restrict__ shared, const float* __restrict__ gate, TO* __restrict__ out, int d,
+                       const TS* __restrict__ x, int ldx) {
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x, i = (blockIdx.y * blockDim.x + threadIdx.x) * 4;
+  if (i >= d) return;
+  float v[4] = {0.f, 0.f, 0.f, 0.f};
+  for (int j0 = 0; j0 < top; j0 += COMBINE_AHEAD) {
+    int p[COMBINE_AHEAD];
+    float w[COMBINE_AHEAD], f[COMBINE_AHEAD][4];
+#pragma unroll
+    for (int u = 0; u < COMBINE_AHEAD; ++u) {
+      const bool in = j0 + u < top;
+      p[u] = in ? __ldcg(place + (size_t)t * top + j0 + u) : -1;
+      w[u] = in ? __ldcg(weights + (size_t)t * top + j0 + u) : 0.f;
+    }
+#pragma unroll
+    for (int u = 0; u < COMBINE_AHEAD; ++u) {
+      if (j0 + u >= top || (p[u] < 0 && x == nullptr)) f[u][0] = f[u][1] = f[u][2] = f[u][3] = 0.f;
+      else if (p[u] >= 0) load4_g<float>(y + (size_t)p[u] * d + i, f[u]);
+      else load4_g<TS>(x + (size_t)t * ldx + i, f[u]);
+    }
+#pragma unroll
+    for (int u = 0; u < COMBINE_AHEAD; ++u)
+      if (j0 + u < top)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) v[e] += w[u] * f[u][e];
+  }
+  if (shared) {
+    float s[4];
+    load4_g<TS>(shared + (size_t)t * d + i, s);
+    const float g = gate ? __ldcg(gate + t) : 1.f;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[e] += g * s[e];
+  }
+  store4<TO>(out + (size_t)t * d + i, v);
+}
+
 RL_API int rl_moe_combine(const float* y, const int* place, const float* weights, int top, const void* shared, int shared_dtype,
                           const float* gate, void* out, int out_dtype, int n_tokens, int d, const void* x, int x_dtype, int ldx,
                           cudaStream_t stream) {
   if (n_tokens <= 0 || d <= 0 || top <= 0) RL_REFUSE(1, "moe_combine: T=%d d=%d top=%d", n_tokens, d, top);
   if (shared == nullptr && x != nullptr) shared_dtype = x_dtype;
   if (x != nullptr && shared_dtype != x_dtype) RL_REFUSE(3, "moe_combine: shared result of type %d beside an input of type %d", shared_dtype, x_dtype);
+  // (which kernel runs depends on sizes and addresses only; both add in the same order)
+  const bool vec = d % 4 == 0 && ldx % 4 == 0 && (((uintptr_t)y | (uintptr_t)shared | (uintptr_t)out | (uintptr_t)x) & 15) == 0;
+  dim3 grid(n_tokens, (d / 4 + 255) / 256);
 #define RL_MC(TS, TO)                                                                                                          \
+  if (vec)                                                                                                                     \
+    RL_LAUNCH_CHECK(rl_launch(moe_combine_vec_kernel<TS, TO>, grid, 256, 0, stream, y, place, weights, top, (const TS*)shared, gate, \
+                              (TO*)out, d, (const TS*)x, ldx));                                                                \
+  else                                                                                                                         \
   RL_LAUNCH_CHECK(rl_launch<false>(moe_combine_kernel<TS, TO>, n_tokens, 256, 0, stream, y, place, weights, top, (const TS*)shared, \
                                    gate, (TO*)out, d, (const TS*)x, ldx))
-  if (shared_dtype == RL_BF16 && out_dtype == RL_F32) RL_MC(bf16, float);
-  else if (shared_dtype == RL_F32 && out_dtype == RL_F32) RL_MC(float, float);
-  else if (shared_dtype == RL_BF16 && out_dtype == RL_BF16) RL_MC(bf16, bf16);
+  if (shared_dtype == RL_BF16 && out_dtype == RL_F32) { RL_MC(bf16, float); }
+  else if (shared_dtype == RL_F32 && out_dtype == RL_F32) { RL_MC(float, float); }
+  else if (shared_dtype == RL_BF16 && out_dtype == RL_BF16) { RL_MC(bf16, bf16); }
   else RL_REFUSE(2, "moe_combine: unsupported types shared=%d out=%d", shared_dtype, out_dtype);
 #undef RL_MC
   return 0;

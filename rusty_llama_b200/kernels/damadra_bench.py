@@ -23,6 +23,7 @@ import torch
 
 from . import microbench as mb
 from . import ops
+from .linear import linear
 from .design_bench import SIZES as VEZATAR_SIZES
 from .design_bench import _frac, llama_config, step_times, vezatar_config
 
@@ -131,9 +132,10 @@ def kernel_table(z: dict, T: int, batch: int, ctx: int, peaks: dict) -> Dict[str
         E, I, top, eff = z["experts"], z["identity"], z["top"], z["eff"]
         x = torch.randn(rows, d, device=dev, dtype=bf)
         wr, corr = torch.randn(E + I, d, device=dev) / math.sqrt(d), torch.zeros(E + I, device=dev)
-        us = timed(lambda: ops.moe_router(x, wr, corr, E + I, top))
+        wr16 = wr.to(bf)
+        us = timed(lambda: ops.moe_choose(linear(x, wr16, out_dtype=torch.float32), corr, E + I, top))
         us_like = timed(lambda: ops.moe_router(x, wr[:E], corr[:E], E, top))
-        note(f"{tag}_router", us, (E + I) * d * 4 + rows * d * 2, 0, ("moe_router of Vezatar", us_like, E * d * 4 + rows * d * 2, 0))
+        note(f"{tag}_router", us, (E + I) * d * 2 + rows * d * 2, 0, ("moe_router (32-bit rows)", us_like, E * d * 4 + rows * d * 2, 0))
         tile_rows = 128 if rows * top >= 64 * E else 32
         ids, wts, _ = ops.moe_router(x, wr, corr, E + I, top)
         ids_l, wts_l, _ = ops.moe_router(x, wr[:E], corr[:E], E, top)

@@ -1230,6 +1230,26 @@ def moe_router(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], n
     return ids, weights, gate
 
 
+def moe_choose(logits: torch.Tensor, bias: Optional[torch.Tensor], n_experts: int, top: int, renormalize: bool = False,
+               logistic: bool = False, renorm_eps: float = 0.0, weight_scale: float = 1.0):
+    """`moe_router` behind its product: logits float32 [T, E (+1)] that another product made."""
+    _cuda(logits, "moe_choose logits", torch.float32)
+    _need(logits.dim() == 2 and logits.shape[1] in (n_experts, n_experts + 1), f"moe_choose: logits {tuple(logits.shape)} for {n_experts} experts")
+    T = logits.shape[0]
+    has_gate = logits.shape[1] == n_experts + 1
+    if bias is not None:
+        _cuda(bias, "moe_choose bias", torch.float32)
+        _need(bias.numel() == n_experts, "moe_choose: one bias per expert")
+    ids = torch.empty((T, top), dtype=torch.int32, device=logits.device)
+    weights = torch.empty((T, top), dtype=torch.float32, device=logits.device)
+    gate = torch.empty((T,), dtype=torch.float32, device=logits.device) if has_gate else None
+    lib = build.load("moe")
+    rc = lib.rl_moe_choose(_p(logits), _p(bias), c_int(T), c_int(n_experts), c_int(top), c_int(1 if renormalize else 0), c_int(1 if has_gate else 0),
+                           _p(ids), _p(weights), _p(gate), c_int(1 if logistic else 0), c_float(renorm_eps), c_float(weight_scale), _stream())
+    _check(lib, rc, "moe_choose")
+    return ids, weights, gate
+
+
 def moe_table_lookup(tokens: torch.Tensor, table: torch.Tensor, n_experts: int):
     """tokens int32 [T], table int32 [vocab, top] -> (ids int32 [T, top] = table[tokens], weights float32 [T, top] = 1 / top)."""
     _cuda(tokens, "moe_table_lookup tokens", torch.int32)

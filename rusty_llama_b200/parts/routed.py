@@ -123,6 +123,11 @@ class RoutedExperts(FeedForward):
             if self.shared_gate:
                 rows.append(tensors[self.prefix + self.names["shared_gate"]])  # one more row of the router's product
             self.w_router = torch.cat(rows, dim=0).contiguous()
+            # A bfloat16 run whose router rows are bfloat16 numbers (as checkpoints store them) gets the same logits from the library's
+            # products, whose sums are 32-bit: every term is the exact product of two bfloat16 numbers either way.
+            narrow = self.w_router.to(torch.bfloat16)
+            exact = self.rt.dtype == torch.bfloat16 and self.d % 8 == 0 and torch.equal(narrow.to(torch.float32), self.w_router)
+            self.w_router16 = narrow if exact else None
         self.bias = tensors[self.prefix + self.names["bias"]].contiguous() if self.has_bias else None
         if self.shared_ff:
             gate, up = tensors[self._shared("gate")], tensors[self._shared("up")]
@@ -139,8 +144,11 @@ class RoutedExperts(FeedForward):
             ids, weights = ops.moe_table_lookup(step.tokens, self.table, self.E)
             gate = None
         else:
-            ids, weights, gate = ops.moe_router(xn, self.w_router, self.bias, self.choices, self.top, self.renormalize,
-                                                logistic=self.router == "sigmoid", renorm_eps=self.renorm_eps, weight_scale=self.weight_scale)
+            how = dict(renormalize=self.renormalize, logistic=self.router == "sigmoid", renorm_eps=self.renorm_eps, weight_scale=self.weight_scale)
+            if self.w_router16 is not None:
+                ids, weights, gate = ops.moe_choose(linear(xn, self.w_router16, out_dtype=torch.float32), self.bias, self.choices, self.top, **how)
+            else:
+                ids, weights, gate = ops.moe_router(xn, self.w_router, self.bias, self.choices, self.top, **how)
         # the height of a row tile: 128 once the experts get that many rows on average (a prompt step), else 32; the plain
         # kernels of a 32-bit run have their own
         tile_rows = 0
