@@ -1,4 +1,5 @@
-// Decode attention over the paged cache in bfloat16 for head sizes 64 and 128, the form for small batches
+// Decode attention over the paged cache in bfloat16 for key and value sizes in multiples of 8 up to 128 (each padded to 64 or 128:
+// TMA fills what lies past a key's or a value's size with zeros, the queries' padding is zero too), the form for small batches
 // whose key range is cut into splits: the same mathematics and the same scratch layout as
 // `attn_decode` (attention_decode.cu; the reference runs its scalar kernel with a single row here,
 // src/backend/cuda.rs:1189-1192), another way of feeding it.
@@ -23,7 +24,7 @@
 // reads the row) and, for the next steps, into the cache.  Same formulas as rope.cu.
 // Two blocks share an SM (99 KB of shared memory each): 192 KB of keys and values in flight per SM,
 // eight product warps.  At head size 64 a page's keys and values are half as many bytes, so the ring
-// has six stages instead of three and the same bytes are in flight.
+// has six stages instead of three (four where only one of the two is 64) and the same bytes are in flight.
 //
 // A learned bias by head and distance (`rl_distance_bias`): a thread's four scores of a page need four numbers, asked for a page
 // ahead (the first page's before the kernel before this one has ended: a weight is not waited for); beyond the last distance with a number of its own they are two registers.
@@ -41,17 +42,17 @@ RL_DEFINE_ERROR_TEXT()
 #define HALF_BYTES (PAGE * 64 * 2)            // one [64 keys][64 dims] swizzled box: 8 KB
 #define MAX_STAGES 6
 
-// What follows from the head size HD (64 or 128): a stage holds a page's keys and then its values, each as
-// HD / 64 boxes of 64 dims; the ring has 96 KB whatever the head size.
-template <int HD>
+// What follows from the padded key and value sizes KD and VD (64 or 128): a stage holds a page's keys and then its values, as
+// KD / 64 and VD / 64 boxes of 64 dims; the ring has 96 KB whatever the sizes.
+template <int KD, int VD>
 struct Shape {
-  static constexpr int BOXES = HD / 64;                     // boxes per page of keys (and of values)
-  static constexpr int STAGE_BYTES = 2 * BOXES * HALF_BYTES;
-  static constexpr int STAGES = 3 * 128 / HD;               // 3 at head size 128, 6 at 64
-  static constexpr int Q_STRIDE = HD + 8;                   // bf16 elements per row of the query tile
-  static constexpr int O_STRIDE = HD + 4;                   // floats per head in the merge buffer
+  static constexpr int K_BOXES = KD / 64, V_BOXES = VD / 64;  // boxes per page of keys, of values
+  static constexpr int STAGE_BYTES = (K_BOXES + V_BOXES) * HALF_BYTES;
+  static constexpr int STAGES = 96 * 1024 / STAGE_BYTES;      // 3 at sizes of 128, 6 at 64, 4 where they differ
+  static constexpr int Q_STRIDE = KD + 8;                     // bf16 elements per row of the query tile
+  static constexpr int O_STRIDE = VD + 4;                     // floats per head in the merge buffer
   static constexpr int SMEM_BYTES = STAGES * STAGE_BYTES + HEADS * Q_STRIDE * 2 + 1024;
-  static constexpr int DPL = HD / 32;                       // dims of the new key and value per lane of the patching warp
+  static constexpr int DPL = KD / 32;                         // dims of the new key and value per lane of the patching warp
 };
 
 struct DecodeBarriers {
@@ -93,7 +94,8 @@ __device__ __forceinline__ void product_warps_sync() { asm volatile("bar.sync 1,
 // byte offset, inside a [64 keys][64 dims] box, of the 16-byte piece `piece` (0..7) of row `row`
 __device__ __forceinline__ uint32_t swz(int row, int piece) { return (uint32_t)(row * 128 + ((piece ^ (row & 7)) << 4)); }
 
-template <int HD>
+// kdim, vdim: the sizes themselves (fuse > 0 and two maps need kdim = vdim = KD = VD)
+template <int KD, int VD>
 __global__ void __launch_bounds__(NUM_THREADS, 2)
 attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                        const bf16* __restrict__ q, int q_stride, const int* __restrict__ block_table, int table_width,
@@ -104,11 +106,12 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
                        unsigned int* __restrict__ counters, bf16* __restrict__ out, int out_stride,
                        const float* __restrict__ q_parts, int n_parts, long long part_stride, int test_role,
                        uint32_t test_ns, const float* __restrict__ sink, int chunk, float softcap, int maps,
-                       const float* __restrict__ bias, int bias_len) {
+                       const float* __restrict__ bias, int bias_len, int kdim, int vdim) {
   // all shared memory is dynamic, so that the ring starts at the block's first byte (1024-byte
   // aligned, as the 128-byte swizzle needs)
-  constexpr int STAGES = Shape<HD>::STAGES, STAGE_BYTES = Shape<HD>::STAGE_BYTES, BOXES = Shape<HD>::BOXES;
-  constexpr int Q_STRIDE = Shape<HD>::Q_STRIDE, O_STRIDE = Shape<HD>::O_STRIDE, DPL = Shape<HD>::DPL;
+  using SH = Shape<KD, VD>;
+  constexpr int STAGES = SH::STAGES, STAGE_BYTES = SH::STAGE_BYTES, K_BOXES = SH::K_BOXES, V_BOXES = SH::V_BOXES;
+  constexpr int Q_STRIDE = SH::Q_STRIDE, O_STRIDE = SH::O_STRIDE, DPL = SH::DPL;
   extern __shared__ __align__(1024) unsigned char smem[];
   unsigned char* ring = smem;
   bf16* q_s = reinterpret_cast<bf16*>(ring + STAGES * STAGE_BYTES);  // [HEADS][Q_STRIDE]
@@ -178,10 +181,9 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
         unsigned char* dst = ring + (size_t)st * STAGE_BYTES;
         mbar_expect_tx(&bars.full[st], STAGE_BYTES);
 #pragma unroll
-        for (int b = 0; b < BOXES; ++b) {
-          tma_load_4d(dst + b * HALF_BYTES, &map_k, &bars.full[st], 64 * b, 0, kh, page);
-          tma_load_4d(dst + (BOXES + b) * HALF_BYTES, &map_v, &bars.full[st], 64 * b, 0, kh, page);
-        }
+        for (int b = 0; b < K_BOXES; ++b) tma_load_4d(dst + b * HALF_BYTES, &map_k, &bars.full[st], 64 * b, 0, kh, page);
+#pragma unroll
+        for (int b = 0; b < V_BOXES; ++b) tma_load_4d(dst + (K_BOXES + b) * HALF_BYTES, &map_v, &bars.full[st], 64 * b, 0, kh, page);
       }
     }
     // The copying warp stays until the product warps have left their loop over the pages (they arrive at
@@ -228,13 +230,13 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
   pdl_wait();  // the queries are the previous kernel's output, and it may still read this one's scratch
   // ---------------- products
   {
-    // this block's queries: HEADS rows of HD values, 16 bytes per thread
-    constexpr int PIECES = HD / 8;
+    // this block's queries: HEADS rows of kdim values, 16 bytes per thread
+    constexpr int PIECES = KD / 8;
     const int r = threadIdx.x / PIECES, piece = threadIdx.x % PIECES;  // 128 threads = 8 (or 16) rows x 16 (or 8) pieces
     // (with two maps per head, query heads 2h and 2h + 1 are the halves of row h; the rest of their rows here stays zero)
     const int qh = (h0 + r) / maps, q_half = (h0 + r) - qh * maps;
-    if (r < n_heads && (maps == 1 || piece / (PIECES / 2) == q_half)) {
-      const size_t at = (size_t)s * q_stride + (size_t)qh * HD + piece * 8;
+    if (r < n_heads && piece * 8 < kdim && (maps == 1 || piece / (PIECES / 2) == q_half)) {
+      const size_t at = (size_t)s * q_stride + (size_t)qh * kdim + piece * 8;
       if (n_parts == 0) {
         *reinterpret_cast<uint4*>(q_s + (size_t)r * Q_STRIDE + piece * 8) = __ldcg(reinterpret_cast<const uint4*>(q + at));
       } else {
@@ -267,9 +269,9 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     }
   }
   product_warps_sync();
-  uint32_t qf[HD / 16][2];  // Q^T as B fragments: (dims kk*16 + 2*t4 [+8], head g)
+  uint32_t qf[KD / 16][2];  // Q^T as B fragments: (dims kk*16 + 2*t4 [+8], head g)
 #pragma unroll
-  for (int k2 = 0; k2 < HD / 32; ++k2) {
+  for (int k2 = 0; k2 < KD / 32; ++k2) {
     uint32_t r[4];
     ldmatrix_x4(r, smem_u32(q_s + (size_t)(lane & 7) * Q_STRIDE + k2 * 32 + 8 * (lane >> 3)));
     qf[2 * k2][0] = r[0];
@@ -278,9 +280,9 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     qf[2 * k2 + 1][1] = r[3];
   }
 
-  float o_acc[HD / 16][4];  // (dim dt*16 + g [+8], head 2*t4 [+1])
+  float o_acc[VD / 16][4];  // (dim dt*16 + g [+8], head 2*t4 [+1])
 #pragma unroll
-  for (int i = 0; i < HD / 16; ++i) o_acc[i][0] = o_acc[i][1] = o_acc[i][2] = o_acc[i][3] = 0.f;
+  for (int i = 0; i < VD / 16; ++i) o_acc[i][0] = o_acc[i][1] = o_acc[i][2] = o_acc[i][3] = 0.f;
   float m_run[2] = {-INFINITY, -INFINITY};  // heads 2*t4, 2*t4+1
   float l_run[2] = {0.f, 0.f};              // per-thread partial sums over this thread's keys
   if (sink != nullptr && split == 0 && warp == 0) {
@@ -299,14 +301,14 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
   const int k_row = warp * 16 + (lane & 7) + 8 * ((lane >> 3) & 1), k_piece = lane >> 4;      // + 2 * kk
   const int v_row = warp * 16 + (lane & 7) + 8 * (lane >> 4), v_piece = (lane >> 3) & 1;      // + 2 * dt
   // The warp that owns the new position's row in the sequence's last page reads the new token's raw key
-  // and value now, so that the loads are long done when that page arrives: lane l takes DPL = HD / 32
+  // and value now, so that the loads are long done when that page arrives: lane l takes DPL = KD / 32
   // dimensions of both, from DPL l on, one load each (or one per partial sum, all independent).
-  const bool patch_here = fuse == 2 && my_lo <= my_hi && my_hi == tile_hi && warp == ((pos & (PAGE - 1)) >> 4);
+  const bool patch_here = KD == VD && fuse == 2 && my_lo <= my_hi && my_hi == tile_hi && warp == ((pos & (PAGE - 1)) >> 4);
   float new_k[DPL], new_v[DPL];
 #pragma unroll
   for (int e = 0; e < DPL; ++e) new_k[e] = new_v[e] = 0.f;
   if (patch_here) {
-    const size_t k_at = (size_t)s * q_stride + (size_t)(H / maps + kh) * HD + DPL * lane, v_at = k_at + (size_t)K * HD;
+    const size_t k_at = (size_t)s * q_stride + (size_t)(H / maps + kh) * KD + DPL * lane, v_at = k_at + (size_t)K * KD;
     if (n_parts == 0) {
       if (DPL == 4) {
         const uint2 kr = __ldcg(reinterpret_cast<const uint2*>(q + k_at)), vr = __ldcg(reinterpret_cast<const uint2*>(q + v_at));
@@ -355,7 +357,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
       ok = false;
       break;
     }
-    const uint32_t k_s = smem_u32(ring) + st * STAGE_BYTES, v_s = k_s + BOXES * HALF_BYTES;
+    const uint32_t k_s = smem_u32(ring) + st * STAGE_BYTES, v_s = k_s + K_BOXES * HALF_BYTES;
     if (patch_here && tile == tile_hi) {
       // the new token's key and value (read before the loop): the key turned by the position's angles,
       // both into this block's copy of the page and (one block per kv head) into the cache
@@ -384,12 +386,12 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
       const int d0 = DPL * lane;
       const uint32_t in_tile = (d0 >> 6) * HALF_BYTES + swz(row, (d0 & 63) >> 3) + (d0 & 7) * 2;
       unsigned char* k_tile = ring + (size_t)st * STAGE_BYTES;
-      const size_t cache_at = (((size_t)table[tile] * K + kh) * PAGE + row) * HD + d0;
+      const size_t cache_at = (((size_t)table[tile] * K + kh) * PAGE + row) * KD + d0;
       if (DPL == 4) {
         const uint2 k_packed = make_uint2(pack_bf16(o[0], o[1]), pack_bf16(o[DPL - 2], o[DPL - 1]));
         const uint2 v_packed = make_uint2(pack_bf16(new_v[0], new_v[1]), pack_bf16(new_v[DPL - 2], new_v[DPL - 1]));
         *reinterpret_cast<uint2*>(k_tile + in_tile) = k_packed;
-        *reinterpret_cast<uint2*>(k_tile + BOXES * HALF_BYTES + in_tile) = v_packed;
+        *reinterpret_cast<uint2*>(k_tile + K_BOXES * HALF_BYTES + in_tile) = v_packed;
         if (g0 == 0) {
           *reinterpret_cast<uint2*>(k_pages_w + cache_at) = k_packed;
           *reinterpret_cast<uint2*>(v_pages_w + cache_at) = v_packed;
@@ -397,7 +399,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
       } else {
         const uint32_t k_packed = pack_bf16(o[0], o[1]), v_packed = pack_bf16(new_v[0], new_v[1]);
         *reinterpret_cast<uint32_t*>(k_tile + in_tile) = k_packed;
-        *reinterpret_cast<uint32_t*>(k_tile + BOXES * HALF_BYTES + in_tile) = v_packed;
+        *reinterpret_cast<uint32_t*>(k_tile + K_BOXES * HALF_BYTES + in_tile) = v_packed;
         if (g0 == 0) {
           *reinterpret_cast<uint32_t*>(k_pages_w + cache_at) = k_packed;
           *reinterpret_cast<uint32_t*>(v_pages_w + cache_at) = v_packed;
@@ -409,7 +411,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     // ---- S^T = K Q^T: this warp's 16 keys x 8 heads
     float s_acc[4] = {0.f, 0.f, 0.f, 0.f};  // (key g [+8], head 2*t4 [+1])
 #pragma unroll
-    for (int kk = 0; kk < HD / 16; ++kk) {
+    for (int kk = 0; kk < KD / 16; ++kk) {
       uint32_t a[4];
       ldmatrix_x4(a, k_s + (kk >> 2) * HALF_BYTES + swz(k_row, ((kk & 3) << 1) | k_piece));
       mma_bf16(s_acc, a, qf[kk][0], qf[kk][1]);
@@ -452,7 +454,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     const uint32_t pb0 = movmatrix_trans(pack_bf16(p[0], p[1]));  // keys 0..7 of the warp's 16
     const uint32_t pb1 = movmatrix_trans(pack_bf16(p[2], p[3]));  // keys 8..15
 #pragma unroll
-    for (int i = 0; i < HD / 16; ++i) {
+    for (int i = 0; i < VD / 16; ++i) {
       o_acc[i][0] *= alpha[0];
       o_acc[i][1] *= alpha[1];
       o_acc[i][2] *= alpha[0];
@@ -461,7 +463,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
 
     // ---- O^T += V^T P^T: head size (16-row tiles) x 8 heads over the warp's 16 keys
 #pragma unroll
-    for (int dt = 0; dt < HD / 16; ++dt) {
+    for (int dt = 0; dt < VD / 16; ++dt) {
       uint32_t a[4];
       ldmatrix_x4_trans(a, v_s + (dt >> 2) * HALF_BYTES + swz(v_row, ((dt & 3) << 1) | v_piece));
       mma_bf16(o_acc[dt], a, pb0, pb1);
@@ -488,7 +490,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     }
     float* mo = merge_o + (size_t)(warp * HEADS + head) * O_STRIDE;
 #pragma unroll
-    for (int dt = 0; dt < HD / 16; ++dt) {
+    for (int dt = 0; dt < VD / 16; ++dt) {
       mo[dt * 16 + g] = o_acc[dt][j];
       mo[dt * 16 + g + 8] = o_acc[dt][2 + j];
     }
@@ -512,10 +514,11 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
       if (counters != nullptr && n_splits == 1) {
         // the only split: this is the result
         const float inv = 1.0f / l;
-        bf16* orow = out + (size_t)s * out_stride + (size_t)(h0 + head) * HD;
+        bf16* orow = out + (size_t)s * out_stride + (size_t)(h0 + head) * vdim;
 #pragma unroll
-        for (int j = 0; j < HD / 16; ++j) {
+        for (int j = 0; j < VD / 16; ++j) {
           const int d = d0 + 16 * j;
+          if (d >= vdim) break;
           float o = 0.f;
 #pragma unroll
           for (int w = 0; w < PRODUCT_WARPS; ++w) o += mw[w] * merge_o[(size_t)(w * HEADS + head) * O_STRIDE + d];
@@ -527,10 +530,11 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
           part_ml[slot * 2] = M;  // -inf when the split held no key at all (an empty split)
           part_ml[slot * 2 + 1] = l;
         }
-        float* po = part_o + slot * HD;
+        float* po = part_o + slot * vdim;
 #pragma unroll
-        for (int j = 0; j < HD / 16; ++j) {
+        for (int j = 0; j < VD / 16; ++j) {
           const int d = d0 + 16 * j;
+          if (d >= vdim) break;
           float o = 0.f;
 #pragma unroll
           for (int w = 0; w < PRODUCT_WARPS; ++w) o += mw[w] * merge_o[(size_t)(w * HEADS + head) * O_STRIDE + d];
@@ -556,7 +560,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     const int head = threadIdx.x >> 4, d0 = threadIdx.x & 15;
     if (head < n_heads) {
       const float* ml = part_ml + ((size_t)s * H + h0 + head) * n_splits * 2;
-      const float* po = part_o + ((size_t)s * H + h0 + head) * n_splits * HD;
+      const float* po = part_o + ((size_t)s * H + h0 + head) * n_splits * vdim;
       float M = -INFINITY;
       for (int i = 0; i < n_splits; ++i) M = fmaxf(M, __ldcg(ml + 2 * i));
       float denom = 0.f;
@@ -565,33 +569,35 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
         denom += ((v.x == -INFINITY) ? 0.f : exp2f(v.x - M)) * v.y;
       }
       const float inv = 1.0f / denom;
-      float o[HD / 16];
+      float o[VD / 16];
 #pragma unroll
-      for (int j = 0; j < HD / 16; ++j) o[j] = 0.f;
+      for (int j = 0; j < VD / 16; ++j) o[j] = 0.f;
       for (int i = 0; i < n_splits; ++i) {
         const float mi = __ldcg(ml + 2 * i);
         const float wi = ((mi == -INFINITY) ? 0.f : exp2f(mi - M)) * inv;
 #pragma unroll
-        for (int j = 0; j < HD / 16; ++j) o[j] += wi * __ldcg(po + (size_t)i * HD + d0 + 16 * j);
+        for (int j = 0; j < VD / 16; ++j)
+          if (d0 + 16 * j < vdim) o[j] += wi * __ldcg(po + (size_t)i * vdim + d0 + 16 * j);
       }
-      bf16* orow = out + (size_t)s * out_stride + (size_t)(h0 + head) * HD;
+      bf16* orow = out + (size_t)s * out_stride + (size_t)(h0 + head) * vdim;
 #pragma unroll
-      for (int j = 0; j < HD / 16; ++j) orow[d0 + 16 * j] = __float2bfloat16_rn(o[j]);
+      for (int j = 0; j < VD / 16; ++j)
+        if (d0 + 16 * j < vdim) orow[d0 + 16 * j] = __float2bfloat16_rn(o[j]);
     }
   }
   if (threadIdx.x == 0) *counter = 0u;  // ready for the next call
 }
 
 // ------------------------------------------------------------------ host side
-// Head sizes this kernel is built for: 64 and 128 (1 if `hd` is one of them).
-RL_API int rl_attn_decode_tma_takes(int hd) { return hd == 64 || hd == 128; }
+// Key and value sizes this kernel is built for (1 if it takes them): multiples of 8 up to 128.
+RL_API int rl_attn_decode_tma_takes(int kdim, int vdim) { return kdim > 0 && vdim > 0 && kdim <= 128 && vdim <= 128 && kdim % 8 == 0 && vdim % 8 == 0; }
 
-// Same arguments as rl_attn_decode (scratch: part_o of n_seqs*H*n_splits*hd floats, part_ml of
+// Same arguments as rl_attn_decode (scratch: part_o of n_seqs*H*n_splits*vdim floats, part_ml of
 // n_seqs*H*n_splits*2), plus the number of cache pages and a status word: one int in device memory,
 // 0 before the call; non-zero afterwards means that a bounded wait expired (51 the copying lane, 52 a
 // product warp; 56: shared memory not aligned) and the output is not valid.
 // fuse: 0 = the queries are already position-encoded and the new key and value already in the cache;
-// 1 = turn the queries here (the cache is another layer's and complete); 2 = turn the queries, and take
+// 1 = turn the queries here (the cache is another layer's and complete), with key and value sizes of 64 or of 128; 2 = turn the queries, and take
 // the new token's key and value from q's rows (keys at column H * hd, values at (H + K) * hd), turn the
 // key and store both (k_pages and v_pages are written).  inv_freq: rot / 2 angles per position; rot = 0
 // means no rotation at all (then fuse = 2 only stores).
@@ -604,19 +610,19 @@ RL_API int rl_attn_decode_tma_takes(int hd) { return hd == 64 || hd == 128; }
 // second kernel then combines the pair, out[s][h] = o / sqrt(mean(o^2) + pair_eps) * pair_factor with o = a_2h - pair_lambda a_(2h+1).
 // wait_test_role, wait_test_ns: 0, 0 in normal use; a test names 51 or 52 and a limit in nanoseconds, and
 // that role's waits give up after that long instead of a second.
-template <int HD>
+template <int KD, int VD>
 static int launch_decode_tma(const void* q, int q_stride, const void* k_pages, const void* v_pages, int n_pages,
                              const int* block_table, int table_width, const int* seq_len, float* part_o, float* part_ml,
-                             void* out, int out_stride, int n_seqs, int H, int K, int window, float scale, int n_splits,
+                             void* out, int out_stride, int n_seqs, int H, int K, int kdim, int vdim, int window, float scale, int n_splits,
                              int* status, int fuse, const float* inv_freq, int rot, int interleaved, unsigned int* counters,
                              const float* q_parts, int n_parts, long long part_stride, int wait_test_role,
                              unsigned int wait_test_ns, const float* sink, int chunk, float softcap, int maps, float pair_lambda, float pair_eps,
                              float pair_factor, const float* bias, int bias_len, cudaStream_t stream) {
   CUtensorMap map_k, map_v;
-  if (make_page_map(&map_k, k_pages, n_pages, K, PAGE, HD, PAGE) || make_page_map(&map_v, v_pages, n_pages, K, PAGE, HD, PAGE))
+  if (make_page_map(&map_k, k_pages, n_pages, K, PAGE, kdim, PAGE) || make_page_map(&map_v, v_pages, n_pages, K, PAGE, vdim, PAGE))
     RL_REFUSE(10, "attn_decode_tma: cannot describe the cache pages to TMA");
-  auto kern = attn_decode_tma_kernel<HD>;
-  constexpr int smem = Shape<HD>::SMEM_BYTES;
+  auto kern = attn_decode_tma_kernel<KD, VD>;
+  constexpr int smem = Shape<KD, VD>::SMEM_BYTES;
   if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
     RL_REFUSE(11, "attn_decode_tma: cannot get %d bytes of shared memory", smem);
   const int G = H / K;
@@ -625,23 +631,23 @@ static int launch_decode_tma(const void* q, int q_stride, const void* k_pages, c
                             table_width, seq_len, part_o, part_ml, H, K, window, scale * 1.4426950408889634f, n_splits, status,
                             fuse, (bf16*)const_cast<void*>(k_pages), (bf16*)const_cast<void*>(v_pages), inv_freq, fuse ? rot : 0,
                             interleaved, counters, (bf16*)out, out_stride, q_parts, n_parts, part_stride, wait_test_role,
-                            (uint32_t)wait_test_ns, sink, chunk, softcap, maps, bias, bias_len));
+                            (uint32_t)wait_test_ns, sink, chunk, softcap, maps, bias, bias_len, kdim, vdim));
   if (maps == 2) {
     dim3 grid1(H / 2, n_seqs);
-    RL_LAUNCH_CHECK(rl_launch(attn_decode_merge_pair_kernel, grid1, HD, 0, stream, (const float*)part_o, (const float*)part_ml, (bf16*)out,
-                              out_stride, H, HD, n_splits, pair_lambda, pair_eps, pair_factor));
+    RL_LAUNCH_CHECK(rl_launch(attn_decode_merge_pair_kernel, grid1, VD, 0, stream, (const float*)part_o, (const float*)part_ml, (bf16*)out,
+                              out_stride, H, vdim, n_splits, pair_lambda, pair_eps, pair_factor));
     return 0;
   }
   if (counters != nullptr) return 0;
   dim3 grid2(H, n_seqs);
   RL_LAUNCH_CHECK(rl_launch(attn_decode_merge_kernel, grid2, 128, 0, stream, (const float*)part_o, (const float*)part_ml,
-                            (bf16*)out, out_stride, H, HD, n_splits));
+                            (bf16*)out, out_stride, H, vdim, n_splits));
   return 0;
 }
 
 RL_API int rl_attn_decode_tma(const void* q, int q_stride, const void* k_pages, const void* v_pages, int n_pages,
                               const int* block_table, int table_width, const int* seq_len, float* part_o, float* part_ml,
-                              void* out, int out_stride, int n_seqs, int H, int K, int hd, int page_size, int window,
+                              void* out, int out_stride, int n_seqs, int H, int K, int kdim, int vdim, int page_size, int window,
                               float scale, int n_splits, int* status, int fuse, const float* inv_freq, int rot,
                               int interleaved, unsigned int* counters, const float* q_parts, int n_parts,
                               long long part_stride, int wait_test_role, unsigned int wait_test_ns, const float* sink,
@@ -651,7 +657,9 @@ RL_API int rl_attn_decode_tma(const void* q, int q_stride, const void* k_pages, 
   if (maps < 1 || maps > 2 || H % maps || (maps == 2 && (counters != nullptr || rot != 0)))
     RL_REFUSE(15, "attn_decode_tma: %d maps in %d heads (two maps: no rotation, no counters)", maps, H);
   if (n_seqs <= 0 || H <= 0 || K <= 0 || n_pages <= 0) RL_REFUSE(1, "attn_decode_tma: S=%d H=%d K=%d pages=%d", n_seqs, H, K, n_pages);
-  if (!rl_attn_decode_tma_takes(hd)) RL_REFUSE(2, "attn_decode_tma: head size %d, this kernel is built for 64 and 128", hd);
+  if (!rl_attn_decode_tma_takes(kdim, vdim)) RL_REFUSE(2, "attn_decode_tma: key and value sizes %d / %d, this kernel is built for multiples of 8 up to 128", kdim, vdim);
+  if ((fuse != 0 || maps == 2) && (kdim != vdim || kdim % 64))
+    RL_REFUSE(17, "attn_decode_tma: fuse=%d and %d maps with key and value sizes %d / %d (64 or 128 of both)", fuse, maps, kdim, vdim);
   if (H % K) RL_REFUSE(3, "attn_decode_tma: %d query heads are not a multiple of %d kv heads", H, K);
   if (page_size != PAGE) RL_REFUSE(4, "attn_decode_tma: page size %d, this kernel is built for %d", page_size, PAGE);
   if (q_stride % 8) RL_REFUSE(5, "attn_decode_tma: query row stride %d breaks 16-byte alignment", q_stride);
@@ -659,17 +667,19 @@ RL_API int rl_attn_decode_tma(const void* q, int q_stride, const void* k_pages, 
   if (n_splits <= 0 || n_splits > 64 || n_seqs > 65535) RL_REFUSE(7, "attn_decode_tma: splits=%d (1..64) seqs=%d", n_splits, n_seqs);
   if (window < 0 || chunk < 0 || softcap < 0.f || status == nullptr || !(scale > 0.f))
     RL_REFUSE(8, "attn_decode_tma: bad window, chunk, cap or scale, or no status word");
-  if (fuse < 0 || fuse > 2 || rot < 0 || rot > hd || (rot & 7) || (fuse && rot > 0 && inv_freq == nullptr))
+  if (fuse < 0 || fuse > 2 || rot < 0 || rot > kdim || (rot & 7) || (fuse && rot > 0 && inv_freq == nullptr))
     RL_REFUSE(12, "attn_decode_tma: fuse=%d with a rotary size of %d (a multiple of 8 up to the head size)%s", fuse, rot, inv_freq ? "" : " and no angles");
   if (n_parts < 0 || n_parts > 64 || (n_parts > 0 && (q_parts == nullptr || fuse == 0 || ((uintptr_t)q_parts & 15) || part_stride % 4 || q_stride % 4)))
     RL_REFUSE(14, "attn_decode_tma: %d partial sums need fuse > 0 and 16-byte aligned rows", n_parts);
-  if (fuse == 2 && q_stride < (H / maps + 2 * K) * hd) RL_REFUSE(13, "attn_decode_tma: rows of %d hold no key and value behind %d query heads", q_stride, H);
-#define RL_DECODE_TMA(HDV)                                                                                                  \
-  return launch_decode_tma<HDV>(q, q_stride, k_pages, v_pages, n_pages, block_table, table_width, seq_len, part_o, part_ml, out, \
-                                out_stride, n_seqs, H, K, window, scale, n_splits, status, fuse, inv_freq, rot, interleaved,      \
+  if (fuse == 2 && q_stride < (H / maps + 2 * K) * kdim) RL_REFUSE(13, "attn_decode_tma: rows of %d hold no key and value behind %d query heads", q_stride, H);
+#define RL_DECODE_TMA(KDV, VDV)                                                                                             \
+  return launch_decode_tma<KDV, VDV>(q, q_stride, k_pages, v_pages, n_pages, block_table, table_width, seq_len, part_o, part_ml, out, \
+                                out_stride, n_seqs, H, K, kdim, vdim, window, scale, n_splits, status, fuse, inv_freq, rot, interleaved,  \
                                 counters, q_parts, n_parts, part_stride, wait_test_role, wait_test_ns, sink, chunk, softcap, maps, pair_lambda,    \
                                 pair_eps, pair_factor, bias, bias_len, stream)
-  if (hd == 64) RL_DECODE_TMA(64);
-  RL_DECODE_TMA(128);
+  if (kdim <= 64 && vdim <= 64) RL_DECODE_TMA(64, 64);
+  if (kdim <= 64) RL_DECODE_TMA(64, 128);
+  if (vdim <= 64) RL_DECODE_TMA(128, 64);
+  RL_DECODE_TMA(128, 128);
 #undef RL_DECODE_TMA
 }

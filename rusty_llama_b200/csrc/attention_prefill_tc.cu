@@ -1,5 +1,6 @@
-// Causal flash attention for prompts on the 5th-generation tensor cores, head sizes 64 and 128, bfloat16,
-// reading keys and values from the paged cache.  Same contract as `flash_prefill` (ragged batch,
+// Causal flash attention for prompts on the 5th-generation tensor cores, bfloat16, key and value sizes in multiples of 8 up to 128
+// (each padded to 64 or 128: TMA fills what lies past a key's or a value's size with zeros, so whatever the queries' tile holds there
+// counts for nothing), reading keys and values from the paged cache.  Same contract as `flash_prefill` (ragged batch,
 // positions from seq_pos0, optional window); the reference's counterpart is its scalar
 // `attention_kernel` (src/backend/cuda.rs:157-232).
 //
@@ -76,14 +77,14 @@ RL_DEFINE_ERROR_TEXT()
 #define SMALL_BYTES 512
 // Distances in a tile that is not far lie between -(BMQ + BNK) and bias_len + BMQ + BNK: that much room on both sides of the table.
 #define BIAS_PAD (BMQ + BNK)
-#define BIAS_SMEM_FLOATS(HD) ((113 * 1024 - SMEM_NEEDED(HD)) / 4 - 2 * BIAS_PAD)  // what is left of half an SM's shared memory
+#define BIAS_SMEM_FLOATS(KD, VD) ((113 * 1024 - SMEM_NEEDED(KD, VD)) / 4 - 2 * BIAS_PAD)  // what is left of half an SM's shared memory
 #define BIAS_NONE 0
 #define BIAS_SMEM 1
 #define BIAS_GLOBAL 2
-// Q is HD / 64 sub-tiles of 16 KB; a K or V tile HD / 64 sub-tiles of 8 KB.  Two blocks must fit an SM and
-// no more (a third would wait for tensor memory): at head size 64 the request is padded to that end.
-#define SMEM_NEEDED(HD) ((HD) / 64 * SUBQ_BYTES + 2 * KV_STAGES * ((HD) / 64) * SUBK_BYTES + SMALL_BYTES)
-#define SMEM_BYTES_OF(HD) (SMEM_NEEDED(HD) > 80 * 1024 ? SMEM_NEEDED(HD) : 80 * 1024)
+// Q is KD / 64 sub-tiles of 16 KB; a K tile KD / 64 sub-tiles of 8 KB, a V tile VD / 64.  Two blocks must fit an SM and
+// no more (a third would wait for tensor memory): at small head sizes the request is padded to that end.
+#define SMEM_NEEDED(KD, VD) ((KD) / 64 * SUBQ_BYTES + KV_STAGES * ((KD) / 64 + (VD) / 64) * SUBK_BYTES + SMALL_BYTES)
+#define SMEM_BYTES_OF(KD, VD) (SMEM_NEEDED(KD, VD) > 80 * 1024 ? SMEM_NEEDED(KD, VD) : 80 * 1024)
 
 struct SmallItems {
   uint64_t q_full, k_full[KV_STAGES], v_full[KV_STAGES];
@@ -95,7 +96,7 @@ struct SmallItems {
 static_assert(sizeof(SmallItems) <= SMALL_BYTES, "the small items must fit behind the tiles");
 static_assert(KV_STAGES == 2, "tile j's key / value stage and its S buffer / product barrier share the index j & 1");
 static_assert(SOFTMAX_WARPS * ROW_STAGE_BYTES <= SUBQ_BYTES, "the output's way out uses the queries' buffer");
-static_assert(2 * (SMEM_BYTES_OF(128) + 1024) <= 228 * 1024, "two blocks must fit an SM's shared memory");
+static_assert(2 * (SMEM_BYTES_OF(128, 128) + 1024) <= 228 * 1024, "two blocks must fit an SM's shared memory");
 
 // 2^x for x <= 8 or so; -inf gives 0
 __device__ __forceinline__ float exp2_fast(float x) {
@@ -107,7 +108,7 @@ __device__ __forceinline__ float exp2_fast(float x) {
 // The MMAs of S = Q K^T for one key tile (a k step is 16 dims; Q and K lie in sub-tiles of 64 dims: 16 KB and 8 KB
 // apart, in the descriptors' units of 16 bytes 1024 and 512), their commit, and a question about another barrier asked
 // first and read last.  Returns 1 if that barrier's phase `peek_parity` is complete.
-// KD: how many dims take part (HD, or half of them where a head has two maps: the descriptors then start at the map's half).
+// KD: how many dims take part (all of the tile's, or half of them where a head has two maps: the descriptors then start at the map's half).
 template <int KD>
 __device__ __forceinline__ uint32_t qk_block(uint32_t tmem_s, uint64_t q_desc, uint64_t k_desc, uint32_t idesc, uint32_t commit_bar,
                                              uint32_t peek_bar, uint32_t peek_parity) {
@@ -195,7 +196,6 @@ __device__ __forceinline__ uint32_t qk_block(uint32_t tmem_s, uint64_t q_desc, u
 }
 // The same for O (+)= P V: four MMAs of 16 keys each, P from tensor memory (8 columns a step), V as the M/N-contiguous
 // operand (2048 bytes = 128 units a step).
-template <int HD>
 __device__ __forceinline__ uint32_t pv_block(uint32_t tmem_o, uint32_t tmem_p, uint64_t v_desc, uint32_t idesc, uint32_t accumulate_first,
                                              uint32_t commit_bar, uint32_t peek_bar, uint32_t peek_parity) {
   uint32_t ready;
@@ -226,24 +226,25 @@ __device__ __forceinline__ uint32_t pv_block(uint32_t tmem_o, uint32_t tmem_p, u
   return ready;
 }
 
-// MAPS 2: query heads 2h and 2h + 1 are the two halves of the HD numbers of row h (the values are the same for both); the row's
-// tile is loaded whole and a block's scores use its half of it and of the keys.
-template <int HD, int MAPS, int BIAS>
+// KD, VD: the padded sizes of a key and a value; kdim, vdim: the sizes themselves.
+// MAPS 2: query heads 2h and 2h + 1 are the two halves of the KD numbers of row h (the values are the same for both); the row's
+// tile is loaded whole and a block's scores use its half of it and of the keys (kdim is then KD).
+template <int KD, int VD, int MAPS, int BIAS>
 __global__ void __launch_bounds__(NUM_THREADS, 2)
 flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                         const __grid_constant__ CUtensorMap map_v, const int* __restrict__ block_table, int table_width,
                         const int* __restrict__ seq_start, const int* __restrict__ seq_pos0, bf16* __restrict__ out,
                         int out_stride, int H, int K, int window, float scale_log2, int* __restrict__ status,
                         int test_role, uint32_t test_ns, const float* __restrict__ sink, int chunk, float softcap,
-                        const float* __restrict__ bias, int bias_len) {
+                        const float* __restrict__ bias, int bias_len, int kdim, int vdim) {
   // All shared memory is dynamic, so that the tiles start at the block's first byte (1024-byte
   // aligned, as the 128-byte swizzle needs) and the small items fit behind them.
-  constexpr int SUBS = HD / 64, Q_BYTES = SUBS * SUBQ_BYTES, KV_BYTES = SUBS * SUBK_BYTES;
+  constexpr int K_SUBS = KD / 64, V_SUBS = VD / 64, Q_BYTES = K_SUBS * SUBQ_BYTES, K_BYTES = K_SUBS * SUBK_BYTES, V_BYTES = V_SUBS * SUBK_BYTES;
   extern __shared__ __align__(1024) unsigned char smem_dyn[];
-  unsigned char* q_s = smem_dyn;                           // 128 rows x HD
-  unsigned char* k_s = q_s + Q_BYTES;                      // KV_STAGES x (64 keys x HD)
-  unsigned char* v_s = k_s + KV_STAGES * KV_BYTES;         // KV_STAGES x (64 keys x HD)
-  SmallItems& sm = *reinterpret_cast<SmallItems*>(v_s + KV_STAGES * KV_BYTES);
+  unsigned char* q_s = smem_dyn;                          // 128 rows x KD
+  unsigned char* k_s = q_s + Q_BYTES;                     // KV_STAGES x (64 keys x KD)
+  unsigned char* v_s = k_s + KV_STAGES * K_BYTES;         // KV_STAGES x (64 keys x VD)
+  SmallItems& sm = *reinterpret_cast<SmallItems*>(v_s + KV_STAGES * V_BYTES);
   uint64_t& q_full = sm.q_full;
   uint64_t(&k_full)[KV_STAGES] = sm.k_full;
   uint64_t(&v_full)[KV_STAGES] = sm.v_full;
@@ -277,7 +278,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   const int tile_lo = lowest_key / BNK, tile_hi = last_pos / BNK;
   const int n_tiles = tile_hi - tile_lo + 1;
   const float* bias_row = BIAS != BIAS_NONE ? bias + (size_t)h * bias_len : nullptr;
-  float* bias_s = reinterpret_cast<float*>(smem_dyn + SMEM_NEEDED(HD));
+  float* bias_s = reinterpret_cast<float*>(smem_dyn + SMEM_NEEDED(KD, VD));
   // with a cap c the scores become tanh(raw * scale / c) first, and c log2(e) takes the scale's place from there on
   const float exp_scale = softcap != 0.f ? softcap * 1.4426950408889634f : scale_log2;
   const float bias_unit = BIAS != BIAS_NONE ? 1.4426950408889634f / exp_scale : 0.f;  // the bias in units of the scores before exp_scale
@@ -315,7 +316,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     if (lane == 0) {
       mbar_expect_tx(&q_full, Q_BYTES);
 #pragma unroll
-      for (int b = 0; b < SUBS; ++b) tma_load_2d(q_s + b * SUBQ_BYTES, &map_q, &q_full, (h / MAPS) * HD + 64 * b, tok0 + row0);
+      for (int b = 0; b < K_SUBS; ++b) tma_load_2d(q_s + b * SUBQ_BYTES, &map_q, &q_full, (h / MAPS) * kdim + 64 * b, tok0 + row0);
       const int* table = block_table + (size_t)s * table_width;
       for (int j = 0; j < n_tiles; ++j) {
         const int st = j % KV_STAGES;
@@ -331,9 +332,9 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
           break;
         }
         if (*(volatile int*)&abort_flag) break;
-        mbar_expect_tx(&k_full[st], KV_BYTES);
+        mbar_expect_tx(&k_full[st], K_BYTES);
 #pragma unroll
-        for (int b = 0; b < SUBS; ++b) tma_load_4d(k_s + (size_t)st * KV_BYTES + b * SUBK_BYTES, &map_k, &k_full[st], 64 * b, 0, kh, page);
+        for (int b = 0; b < K_SUBS; ++b) tma_load_4d(k_s + (size_t)st * K_BYTES + b * SUBK_BYTES, &map_k, &k_full[st], 64 * b, 0, kh, page);
         issued_k = j + 1;
         // V
         if (round > 0 && !mbar_wait_role(&pv_done[st], (round - 1) & 1, ctl, 12)) {
@@ -341,9 +342,9 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
           abort_flag = 1;
           break;
         }
-        mbar_expect_tx(&v_full[st], KV_BYTES);
+        mbar_expect_tx(&v_full[st], V_BYTES);
 #pragma unroll
-        for (int b = 0; b < SUBS; ++b) tma_load_4d(v_s + (size_t)st * KV_BYTES + b * SUBK_BYTES, &map_v, &v_full[st], 64 * b, 0, kh, page);
+        for (int b = 0; b < V_SUBS; ++b) tma_load_4d(v_s + (size_t)st * V_BYTES + b * SUBK_BYTES, &map_v, &v_full[st], 64 * b, 0, kh, page);
         issued_v = j + 1;
       }
     }
@@ -351,7 +352,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     // ---------------- tensor-core issuer
     if (lane == 0) {
       const uint32_t idesc_qk = make_idesc_bf16(BMQ, BNK, 0, 0);
-      const uint32_t idesc_pv = make_idesc_bf16(BMQ, HD, 0, 1);
+      const uint32_t idesc_pv = make_idesc_bf16(BMQ, VD, 0, 1);
       const uint32_t q_addr = smem_u32(q_s);
       bool ok = mbar_wait_role(&q_full, 0, ctl, 13);
       if (!ok) {
@@ -366,7 +367,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       // to skip the waits below: the tensor-core GEMM's issuer, built the same way, gave up on a stage about once in
       // 10^5 launches when it skipped its wait after a yes (before p_ready had two barriers), so every tile is waited for.
       // (a map's half starts at the second sub-tile of 64 dims, or 64 bytes into the only one)
-      constexpr uint64_t HALF_Q = HD == 128 ? SUBQ_BYTES / 16 : 4, HALF_K = HD == 128 ? SUBK_BYTES / 16 : 4;
+      constexpr uint64_t HALF_Q = KD == 128 ? SUBQ_BYTES / 16 : 4, HALF_K = KD == 128 ? SUBK_BYTES / 16 : 4;
       const uint64_t q_desc = make_smem_desc(q_addr) + (MAPS > 1 ? (h % MAPS) * HALF_Q : 0);
       const uint64_t k_half = MAPS > 1 ? (h % MAPS) * HALF_K : 0;
       uint32_t v_ready = 0, k_ready = 0;  // the answers: value tile j, key tile j + 2 (for the S after next) have landed
@@ -380,7 +381,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       auto issue_qk = [&](int j, int jv) {
         const int st = j % KV_STAGES;
         tc_fence_after();
-        v_ready = qk_block<HD / MAPS>(tmem_base + (uint32_t)((j & 1) * BNK), q_desc, make_smem_desc(smem_u32(k_s + (size_t)st * KV_BYTES)) + k_half, idesc_qk,
+        v_ready = qk_block<KD / MAPS>(tmem_base + (uint32_t)((j & 1) * BNK), q_desc, make_smem_desc(smem_u32(k_s + (size_t)st * K_BYTES)) + k_half, idesc_qk,
                                smem_u32(&s_full[j & 1]), smem_u32(&v_full[jv % KV_STAGES]), (uint32_t)((jv / KV_STAGES) & 1));
       };
       if (ok) ok = wait_for(&k_full[0], 0, 14);
@@ -400,8 +401,8 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         tc_fence_after();
         // O += P(j) V(j); asks for key tile j + 2
         const int jk = j + 2;
-        k_ready = pv_block<HD>(tmem_base + O_COL, tmem_base + (uint32_t)((j & 1) * BNK),
-                               make_smem_desc_mn(smem_u32(v_s + (size_t)st * KV_BYTES), SUBK_BYTES, 1024), idesc_pv, j > 0 ? 1u : 0u,
+        k_ready = pv_block(tmem_base + O_COL, tmem_base + (uint32_t)((j & 1) * BNK),
+                               make_smem_desc_mn(smem_u32(v_s + (size_t)st * V_BYTES), SUBK_BYTES, 1024), idesc_pv, j > 0 ? 1u : 0u,
                                smem_u32(&pv_done[j & 1]), smem_u32(&k_full[jk % KV_STAGES]), (uint32_t)((jk / KV_STAGES) & 1));
         if (jk < n_tiles) {
           // S of tile j + 2 goes into the buffer whose P this product has just been told to read
@@ -513,7 +514,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         }
         tc_fence_after();
 #pragma unroll 1
-        for (int c = 0; c < HD / 32; ++c) {
+        for (int c = 0; c < VD / 32; ++c) {
           uint32_t o[32];
           tmem_ld_32x32b_x32(o_addr + c * 32, o);
           tmem_ld_wait();
@@ -551,9 +552,9 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       // queries' buffer, which no product reads any more, and writes whole 128-byte rows (see tc_common.cuh).
       const uint32_t stage = smem_u32(q_s) + (uint32_t)(warp * ROW_STAGE_BYTES);
       const int rows_valid = rows_here - warp * 32;  // (may be <= 0: nothing is written then)
-      bf16* o = out + (size_t)(tok0 + row0 + warp * 32) * out_stride + (size_t)h * HD;
+      bf16* o = out + (size_t)(tok0 + row0 + warp * 32) * out_stride + (size_t)h * vdim;
 #pragma unroll 1
-      for (int c = 0; c < HD / 64; ++c) {
+      for (int c = 0; c < VD / 64; ++c) {
         uint32_t v0[32], v1[32];
         tmem_ld_32x32b_x32(o_addr + c * 64, v0);
         tmem_ld_32x32b_x32(o_addr + c * 64 + 32, v1);
@@ -563,7 +564,7 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
           v0[i] = __float_as_uint(__uint_as_float(v0[i]) * inv);
           v1[i] = __float_as_uint(__uint_as_float(v1[i]) * inv);
         }
-        store_rows64_bf16(o + c * 64, out_stride, rows_valid, v0, v1, stage, lane);
+        store_rows64_bf16(o + c * 64, out_stride, rows_valid, v0, v1, stage, lane, vdim - c * 64);
       }
     }
   }
@@ -582,29 +583,29 @@ flash_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
 }
 
 // ------------------------------------------------------------------ host side
-// Head sizes this kernel is built for: 64 and 128 (1 if `hd` is one of them).
-RL_API int rl_flash_prefill_tc_takes(int hd) { return hd == 64 || hd == 128; }
+// Key and value sizes this kernel is built for (1 if it takes them): multiples of 8 up to 128.
+RL_API int rl_flash_prefill_tc_takes(int kdim, int vdim) { return kdim > 0 && vdim > 0 && kdim <= 128 && vdim <= 128 && kdim % 8 == 0 && vdim % 8 == 0; }
 
-template <int HD, int MAPS, int BIAS>
+template <int KD, int VD, int MAPS, int BIAS>
 static int launch_flash_tc(const void* q, int q_stride, int n_tokens, const void* k_pages, const void* v_pages, int n_pages,
                            const int* block_table, int table_width, const int* seq_start, const int* seq_pos0, void* out,
-                           int out_stride, int n_seqs, int max_q_len, int H, int K, int window, float scale, int* status,
+                           int out_stride, int n_seqs, int max_q_len, int H, int K, int kdim, int vdim, int window, float scale, int* status,
                            int wait_test_role, unsigned int wait_test_ns, const float* sink, int chunk, float softcap, const float* bias, int bias_len, cudaStream_t stream) {
   CUtensorMap map_q, map_k, map_v;
   if (make_matrix_map(&map_q, q, n_tokens, q_stride, q_stride, BMQ))
     RL_REFUSE(10, "flash_prefill_tc: cannot describe the query tensor to TMA");
-  if (make_page_map(&map_k, k_pages, n_pages, K, PAGE, HD, PAGE) || make_page_map(&map_v, v_pages, n_pages, K, PAGE, HD, PAGE))
+  if (make_page_map(&map_k, k_pages, n_pages, K, PAGE, kdim, PAGE) || make_page_map(&map_v, v_pages, n_pages, K, PAGE, vdim, PAGE))
     RL_REFUSE(11, "flash_prefill_tc: cannot describe the cache pages to TMA");
-  size_t smem = SMEM_BYTES_OF(HD);
-  const size_t with_bias = SMEM_NEEDED(HD) + (size_t)(bias_len + 2 * BIAS_PAD) * 4;
+  size_t smem = SMEM_BYTES_OF(KD, VD);
+  const size_t with_bias = SMEM_NEEDED(KD, VD) + (size_t)(bias_len + 2 * BIAS_PAD) * 4;
   if (BIAS == BIAS_SMEM && with_bias > smem) smem = with_bias;
-  auto kern = flash_prefill_tc_kernel<HD, MAPS, BIAS>;
+  auto kern = flash_prefill_tc_kernel<KD, VD, MAPS, BIAS>;
   if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
     RL_REFUSE(12, "flash_prefill_tc: cannot get %zu bytes of shared memory", smem);
   dim3 grid(H * n_seqs, (max_q_len + BMQ - 1) / BMQ);
   RL_LAUNCH_CHECK(rl_launch(kern, grid, NUM_THREADS, smem, stream, map_q, map_k, map_v, block_table, table_width, seq_start, seq_pos0,
                             (bf16*)out, out_stride, H, K, window, scale * 1.4426950408889634f, status, wait_test_role,
-                            (uint32_t)wait_test_ns, sink, chunk, softcap, bias, bias_len));
+                            (uint32_t)wait_test_ns, sink, chunk, softcap, bias, bias_len, kdim, vdim));
   return 0;
 }
 
@@ -617,14 +618,15 @@ static int launch_flash_tc(const void* q, int q_stride, int n_tokens, const void
 RL_API int rl_flash_prefill_tc(const void* q, int q_stride, int n_tokens, const void* k_pages, const void* v_pages,
                                int n_pages, const int* block_table, int table_width, const int* seq_start,
                                const int* seq_pos0, void* out, int out_stride, int n_seqs, int max_q_len, int H, int K,
-                               int hd, int page_size, int window, float scale, int* status, int wait_test_role,
+                               int kdim, int vdim, int page_size, int window, float scale, int* status, int wait_test_role,
                                unsigned int wait_test_ns, const float* sink, int chunk, float softcap, int maps, const float* bias,
                                int bias_len, cudaStream_t stream) {
   if (bias != nullptr && (bias_len <= 0 || maps != 1)) RL_REFUSE(13, "flash_prefill_tc: a bias by distance of %d numbers a head, %d maps (one is built)", bias_len, maps);
   if (maps < 1 || maps > 2 || H % maps) RL_REFUSE(9, "flash_prefill_tc: %d maps in %d heads", maps, H);
   if (n_seqs <= 0 || max_q_len <= 0 || H <= 0 || K <= 0 || n_tokens <= 0 || n_pages <= 0)
     RL_REFUSE(1, "flash_prefill_tc: S=%d max_q=%d H=%d K=%d T=%d pages=%d", n_seqs, max_q_len, H, K, n_tokens, n_pages);
-  if (!rl_flash_prefill_tc_takes(hd)) RL_REFUSE(2, "flash_prefill_tc: head size %d, this kernel is built for 64 and 128", hd);
+  if (!rl_flash_prefill_tc_takes(kdim, vdim)) RL_REFUSE(2, "flash_prefill_tc: key and value sizes %d / %d, this kernel is built for multiples of 8 up to 128", kdim, vdim);
+  if (maps > 1 && (kdim != vdim || kdim % 64)) RL_REFUSE(14, "flash_prefill_tc: two maps in rows of %d numbers beside values of %d (64 or 128 of both)", kdim, vdim);
   if (H % K) RL_REFUSE(3, "flash_prefill_tc: %d query heads are not a multiple of %d kv heads", H, K);
   if (page_size != PAGE) RL_REFUSE(4, "flash_prefill_tc: page size %d, this kernel is built for %d", page_size, PAGE);
   if (q_stride % 8 || out_stride % 8) RL_REFUSE(5, "flash_prefill_tc: strides %d/%d break 16-byte alignment", q_stride, out_stride);
@@ -633,17 +635,22 @@ RL_API int rl_flash_prefill_tc(const void* q, int q_stride, int n_tokens, const 
     RL_REFUSE(7, "flash_prefill_tc: H=%d x S=%d blocks or %d query rows exceed the grid", H, n_seqs, max_q_len);
   if (window < 0 || chunk < 0 || softcap < 0.f || status == nullptr || !(scale > 0.f))
     RL_REFUSE(8, "flash_prefill_tc: bad window, chunk, cap or scale, or no status word");
-#define RL_FTC(HDV, MAPSV, BIASV)                                                                                                                  \
-  return launch_flash_tc<HDV, MAPSV, BIASV>(q, q_stride, n_tokens, k_pages, v_pages, n_pages, block_table, table_width, seq_start, seq_pos0, out,  \
-                                     out_stride, n_seqs, max_q_len, H, K, window, scale, status, wait_test_role, wait_test_ns, sink, chunk, \
-                                     softcap, bias, bias_len, stream)
-  if (bias != nullptr && hd == 64 && bias_len <= BIAS_SMEM_FLOATS(64)) RL_FTC(64, 1, BIAS_SMEM);
-  if (bias != nullptr && hd == 64) RL_FTC(64, 1, BIAS_GLOBAL);
-  if (bias != nullptr && bias_len <= BIAS_SMEM_FLOATS(128)) RL_FTC(128, 1, BIAS_SMEM);
-  if (bias != nullptr) RL_FTC(128, 1, BIAS_GLOBAL);
-  if (hd == 64 && maps == 2) RL_FTC(64, 2, BIAS_NONE);
-  if (hd == 64) RL_FTC(64, 1, BIAS_NONE);
-  if (maps == 2) RL_FTC(128, 2, BIAS_NONE);
-  RL_FTC(128, 1, BIAS_NONE);
+#define RL_FTC(KDV, VDV, MAPSV, BIASV)                                                                                                        \
+  return launch_flash_tc<KDV, VDV, MAPSV, BIASV>(q, q_stride, n_tokens, k_pages, v_pages, n_pages, block_table, table_width, seq_start,       \
+                                                 seq_pos0, out, out_stride, n_seqs, max_q_len, H, K, kdim, vdim, window, scale, status,       \
+                                                 wait_test_role, wait_test_ns, sink, chunk, softcap, bias, bias_len, stream)
+#define RL_FTC_BIAS(KDV, VDV)                                                        \
+  do {                                                                               \
+    if (bias == nullptr) RL_FTC(KDV, VDV, 1, BIAS_NONE);                             \
+    if (bias_len <= BIAS_SMEM_FLOATS(KDV, VDV)) RL_FTC(KDV, VDV, 1, BIAS_SMEM);      \
+    RL_FTC(KDV, VDV, 1, BIAS_GLOBAL);                                                \
+  } while (0)
+  if (maps == 2 && kdim == 64) RL_FTC(64, 64, 2, BIAS_NONE);
+  if (maps == 2) RL_FTC(128, 128, 2, BIAS_NONE);
+  if (kdim <= 64 && vdim <= 64) RL_FTC_BIAS(64, 64);
+  if (kdim <= 64) RL_FTC_BIAS(64, 128);
+  if (vdim <= 64) RL_FTC_BIAS(128, 64);
+  RL_FTC_BIAS(128, 128);
+#undef RL_FTC_BIAS
 #undef RL_FTC
 }

@@ -288,9 +288,10 @@ __device__ __forceinline__ uint32_t pack2(float a, float b) {
   __nv_bfloat162 p = __floats2bfloat162_rn(a, b);
   return *reinterpret_cast<uint32_t*>(&p);
 }
-// 64 columns of this lane's row (two tensor-memory loads) -> out[rows of the warp][col0 .. col0 + 63]
+// 64 columns of this lane's row (two tensor-memory loads) -> out[rows of the warp][col0 .. col0 + 63], the first `cols_valid` of them
+// (a multiple of 8)
 __device__ __forceinline__ void store_rows64_bf16(bf16* out_tile, int ldo, int rows_valid, const uint32_t (&r0)[32], const uint32_t (&r1)[32],
-                                                  uint32_t stage, int lane) {
+                                                  uint32_t stage, int lane, int cols_valid = 64) {
 #pragma unroll
   for (int p = 0; p < 8; ++p) {
     const uint32_t* r = p < 4 ? r0 : r1;
@@ -305,7 +306,7 @@ __device__ __forceinline__ void store_rows64_bf16(bf16* out_tile, int ldo, int r
     const int rr = it * 4 + (lane >> 3), pc = lane & 7;
     uint4 v;
     asm volatile("ld.shared.v4.u32 {%0, %1, %2, %3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "r"(stage + rr * 128 + ((pc ^ (rr & 7)) << 4)));
-    if (rr < rows_valid) *reinterpret_cast<uint4*>(out_tile + (size_t)rr * ldo + pc * 8) = v;
+    if (rr < rows_valid && pc * 8 < cols_valid) *reinterpret_cast<uint4*>(out_tile + (size_t)rr * ldo + pc * 8) = v;
   }
   __syncwarp();
 }
@@ -396,7 +397,7 @@ static int make_matrix_map(CUtensorMap* map, const void* base, int rows, int col
 }
 
 // The 4-D view of a group's cache pages that the attention kernels copy from: [page][kv head][position][dim],
-// boxes of 64 dims x `box_rows` positions of one head of one page, 128-byte swizzled.  0 on success.
+// boxes of 64 dims x `box_rows` positions of one head of one page, 128-byte swizzled (dims past the head's size read zero).  0 on success.
 static int make_page_map(CUtensorMap* map, const void* pages, int n_pages, int kv_heads, int page_size, int head_dim, int box_rows) {
   EncodeTiledFn enc = encode_tiled();
   if (!enc) return 1;

@@ -304,7 +304,12 @@ def attn_generic(
     return out
 
 
-ATTN_DECODE_TMA_HEAD_DIMS = (64, 128)  # head sizes the TMA-fed decode kernel is built for
+ATTN_DECODE_TMA_HEAD_DIMS = (64, 128)  # head sizes at which the TMA-fed decode kernel also takes raw projections (`fuse`) and two maps
+
+
+def attn_tma_takes(kdim: int, vdim: int) -> bool:
+    """Key and value sizes that the TMA-fed decode kernel and the tcgen05 prompt kernel are built for (each padded to 64 or 128)."""
+    return 0 < kdim <= 128 and 0 < vdim <= 128 and kdim % 8 == 0 and vdim % 8 == 0
 
 
 def _check_sink(sink, num_heads: int, what: str) -> None:
@@ -333,9 +338,12 @@ def attn_decode(
     out: Optional[torch.Tensor] = None, impl: str = "auto", fuse: int = 0,
     inv_freq: Optional[torch.Tensor] = None, rotary_dim: int = 0, interleaved: bool = False,
     counters: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0, pair=None,
-    bias: Optional[torch.Tensor] = None,
+    bias: Optional[torch.Tensor] = None, value_dim: int = 0,
 ) -> torch.Tensor:
     """One query token per sequence over keys 0..seq_len-1, the key range cut into `n_splits`.
+
+    value_dim (the "tma" kernel without fuse and pair): the size of a value where it differs from head_dim, a key's; the kernel then takes
+    multiples of 8 up to 128 of both.
 
     bias (the "tma" kernel only): None, or float32 [H, L], a learned bias of the scores by head and distance (`_bias_args`).
 
@@ -376,25 +384,26 @@ def attn_decode(
     _need(pair is None or (num_heads % 2 == 0 and rotary_dim == 0 and counters is None), "attn_decode: two maps per head take neither a rotation nor counters")
     _need(q_cols >= num_heads // maps * head_dim, "attn_decode: q rows too short")
     _need(q.data_ptr() % 16 == 0, "attn_decode: q is not 16-byte aligned")
-    _check_pages(k_pages, v_pages, act, num_kv_heads, head_dim, "attn_decode")
+    vdim = value_dim or head_dim
+    _check_kv_pages(k_pages, v_pages, act, num_kv_heads, head_dim, vdim, "attn_decode")
     _cuda(block_table, "attn_decode block_table", torch.int32)
     _cuda(seq_len, "attn_decode seq_len", torch.int32)
     _need(block_table.dim() == 2 and block_table.shape[0] >= S and seq_len.numel() == S, "attn_decode: metadata sizes")
     _cuda(scratch, "attn_decode scratch", torch.float32)
-    need = attn_decode_scratch_floats(S, num_heads, head_dim, n_splits)
+    need = attn_decode_scratch_floats(S, num_heads, vdim, n_splits)
     _need(scratch.numel() >= need, f"attn_decode: scratch holds {scratch.numel()} floats, {need} needed")
     if out is None:
-        out = torch.empty((S, num_heads // maps * head_dim), dtype=act, device=q.device)
+        out = torch.empty((S, num_heads // maps * vdim), dtype=act, device=q.device)
     _cuda(out, "attn_decode out", act, contiguous=False)
-    _need(_rows(out, "attn_decode out") >= out.shape[1] and tuple(out.shape) == (S, num_heads // maps * head_dim), "attn_decode: out must be [S, H head_dim] rows")
+    _need(_rows(out, "attn_decode out") >= out.shape[1] and tuple(out.shape) == (S, num_heads // maps * vdim), "attn_decode: out must be [S, H value_dim] rows")
     if scale is None:
         scale = 1.0 / math.sqrt(head_dim)
-    n_o = S * num_heads * n_splits * head_dim
+    n_o = S * num_heads * n_splits * vdim
     part_o = c_void_p(scratch.data_ptr())
     part_ml = c_void_p(scratch.data_ptr() + 4 * n_o)
     _need(impl in ("auto", "warp", "tma"), f"attn_decode: unknown impl {impl!r}")
     if impl == "auto":
-        impl = "tma" if (head_dim in ATTN_DECODE_TMA_HEAD_DIMS and act == torch.bfloat16) else "warp"
+        impl = "tma" if (act == torch.bfloat16 and (head_dim in ATTN_DECODE_TMA_HEAD_DIMS or vdim != head_dim)) else "warp"
     _need(fuse in (0, 1, 2), f"attn_decode: fuse={fuse}")
     if fuse:
         _need(impl == "tma", "attn_decode: only the TMA kernel fuses the position encoding")
@@ -417,7 +426,7 @@ def attn_decode(
         rc = lib.rl_attn_decode_tma(
             c_void_p(0) if q_parts is not None else _p(q), c_int(qs), _p(k_pages), _p(v_pages), c_int(k_pages.shape[0]), _p(block_table),
             c_int(block_table.shape[1]), _p(seq_len), part_o, part_ml, _p(out), c_int(out.stride(0)), c_int(S),
-            c_int(num_heads), c_int(num_kv_heads), c_int(head_dim), c_int(PAGE_SIZE), c_int(window), c_float(scale),
+            c_int(num_heads), c_int(num_kv_heads), c_int(head_dim), c_int(vdim), c_int(PAGE_SIZE), c_int(window), c_float(scale),
             c_int(n_splits), _p(status), c_int(fuse), _p(inv_freq) if (fuse and rotary_dim) else c_void_p(0), c_int(rotary_dim if fuse else 0),
             c_int(1 if interleaved else 0), _p(counters) if counters is not None else c_void_p(0),
             _p(q_parts) if q_parts is not None else c_void_p(0), c_int(0 if q_parts is None else q_parts.shape[0]),
@@ -426,7 +435,8 @@ def attn_decode(
         )
         _check(lib, rc, "attn_decode_tma", kernels=1 if counters is not None else 2)
         return out
-    _need(chunk == 0 and softcap == 0.0 and pair is None and bias is None, "attn_decode: only the TMA kernel takes chunks, capped scores, a bias and two maps per head")
+    _need(chunk == 0 and softcap == 0.0 and pair is None and bias is None and vdim == head_dim,
+          "attn_decode: only the TMA kernel takes chunks, capped scores, a bias, values of another size and two maps per head")
     lib = build.load("attention_decode")
     rc = lib.rl_attn_decode_sink(
         _p(q), c_int(_dt(q, "attn_decode")), c_int(qs), _p(k_pages), _p(v_pages), _p(block_table),
@@ -471,27 +481,29 @@ def flash_prefill(
     return out
 
 
-FLASH_TC_HEAD_DIMS = (64, 128)  # head sizes the tcgen05 prompt attention is built for
+FLASH_TC_HEAD_DIMS = (64, 128)  # head sizes at which the tcgen05 prompt attention needs no padding (and takes two maps)
 
 
 def flash_prefill_tc(
     q: torch.Tensor, k_pages, v_pages, block_table, seq_start, seq_pos0, max_q_len: int, num_heads: int,
     num_kv_heads: int, head_dim: int, window: int = 0, scale: Optional[float] = None,
     out: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None, chunk: int = 0, softcap: float = 0.0, maps: int = 1,
-    bias: Optional[torch.Tensor] = None,
+    bias: Optional[torch.Tensor] = None, value_dim: int = 0,
 ) -> torch.Tensor:
-    """`flash_prefill` on the tcgen05 tensor cores (TMA-fed, S and P V in tensor memory); head sizes 64 and 128.
+    """`flash_prefill` on the tcgen05 tensor cores (TMA-fed, S and P V in tensor memory); key sizes head_dim and value sizes value_dim
+    (0: the same) in multiples of 8 up to 128.
     chunk: 0, or the size of the chunks of positions (counted from 0) outside of which a query sees nothing; softcap: 0, or the
     cap c of s <- c tanh(s / c) on the scaled scores.
     maps: 1, or 2: query heads 2h and 2h + 1 are the two halves of row h's head_dim numbers, against the same halves of the keys.
     bias: None, or float32 [H, L], a learned bias of the scores by head and distance (`_bias_args`; one map only)."""
     _need(maps in (1, 2) and num_heads % maps == 0, f"flash_prefill_tc: {maps} maps in {num_heads} heads")
-    _need(head_dim in FLASH_TC_HEAD_DIMS, f"flash_prefill_tc: head size {head_dim}, this kernel is built for {FLASH_TC_HEAD_DIMS}")
+    vdim = value_dim or head_dim
+    _need(attn_tma_takes(head_dim, vdim), f"flash_prefill_tc: key and value sizes {head_dim} / {vdim}, this kernel is built for multiples of 8 up to 128")
     _cuda(q, "flash_prefill_tc q", torch.bfloat16, contiguous=False)
     qs = _rows(q, "flash_prefill_tc q")
     T = q.shape[0]
     _need(q.shape[1] >= num_heads // maps * head_dim, "flash_prefill_tc: q rows too short")
-    _check_pages(k_pages, v_pages, torch.bfloat16, num_kv_heads, head_dim, "flash_prefill_tc")
+    _check_kv_pages(k_pages, v_pages, torch.bfloat16, num_kv_heads, head_dim, vdim, "flash_prefill_tc")
     _need(k_pages.shape[0] == v_pages.shape[0], "flash_prefill_tc: k and v have different page counts")
     _cuda(block_table, "flash_prefill_tc block_table", torch.int32)
     _cuda(seq_start, "flash_prefill_tc seq_start", torch.int32)
@@ -499,9 +511,9 @@ def flash_prefill_tc(
     S = seq_pos0.numel()
     _need(seq_start.numel() == S + 1 and block_table.dim() == 2 and block_table.shape[0] >= S, "flash_prefill_tc: metadata sizes")
     if out is None:
-        out = torch.empty((T, num_heads * head_dim), dtype=torch.bfloat16, device=q.device)
+        out = torch.empty((T, num_heads * vdim), dtype=torch.bfloat16, device=q.device)
     _cuda(out, "flash_prefill_tc out", torch.bfloat16, contiguous=False)
-    _need(_rows(out, "flash_prefill_tc out") % 8 == 0 and tuple(out.shape) == (T, num_heads * head_dim), "flash_prefill_tc: out must be [T, H head_dim] rows at 16-byte steps")
+    _need(_rows(out, "flash_prefill_tc out") % 8 == 0 and tuple(out.shape) == (T, num_heads * vdim), "flash_prefill_tc: out must be [T, H value_dim] rows at 16-byte steps")
     if scale is None:
         scale = 1.0 / math.sqrt(head_dim)
     _check_sink(sink, num_heads, "flash_prefill_tc")
@@ -510,7 +522,7 @@ def flash_prefill_tc(
     rc = lib.rl_flash_prefill_tc(
         _p(q), c_int(qs), c_int(T), _p(k_pages), _p(v_pages), c_int(k_pages.shape[0]), _p(block_table),
         c_int(block_table.shape[1]), _p(seq_start), _p(seq_pos0), _p(out), c_int(out.stride(0)), c_int(S), c_int(max_q_len),
-        c_int(num_heads), c_int(num_kv_heads), c_int(head_dim), c_int(PAGE_SIZE), c_int(window), c_float(scale), _p(status), *_wt(), _p(sink),
+        c_int(num_heads), c_int(num_kv_heads), c_int(head_dim), c_int(vdim), c_int(PAGE_SIZE), c_int(window), c_float(scale), _p(status), *_wt(), _p(sink),
         c_int(chunk), c_float(softcap), c_int(maps), *_bias_args(bias, num_heads, "flash_prefill_tc"), _stream(),
     )
     _check(lib, rc, "flash_prefill_tc")

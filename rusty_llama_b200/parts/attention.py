@@ -27,14 +27,14 @@ _DECODE_TMA_BLOCKS_PER_SM = 2
 _DECODE_TMA_MIN_PAGES = 4
 
 
-def decode_splits(n_seqs: int, num_heads: int, num_kv_heads: int, kv_len: int, head_dim: int = 0, sms: int = 0) -> int:
-    """How many pieces to cut the key range into, from shapes only (head_dim tells which of the two
+def decode_splits(n_seqs: int, num_heads: int, num_kv_heads: int, kv_len: int, head_dim: int = 0, sms: int = 0, tma: bool = False) -> int:
+    """How many pieces to cut the key range into, from shapes only (head_dim, or tma, tells which of the two
     decode kernels will run; sms: the GPU's multiprocessors, asked from the current device if 0)."""
     sms = sms or sm_count()
     group = num_heads // num_kv_heads
     per_split = n_seqs * num_kv_heads * ((group + _DECODE_HEADS_PER_BLOCK - 1) // _DECODE_HEADS_PER_BLOCK)
     tiles = max(1, (kv_len + ops.PAGE_SIZE - 1) // ops.PAGE_SIZE)
-    if head_dim in ops.ATTN_DECODE_TMA_HEAD_DIMS:
+    if tma or head_dim in ops.ATTN_DECODE_TMA_HEAD_DIMS:
         want = _DECODE_TMA_BLOCKS_PER_SM * sms // per_split
         return max(1, min(want, (tiles + _DECODE_TMA_MIN_PAGES - 1) // _DECODE_TMA_MIN_PAGES, 64))
     want = _DECODE_BLOCKS_PER_SM * sms // per_split
@@ -86,8 +86,9 @@ class Attention(Mixer):
     A plain attention, with or without a sink, runs on the kernels built for it (tensor-core prompt attention, TMA-fed
     decode attention, the rotation fused with the cache write or with the decode kernel).  With any other option (and with a
     sink in a 32-bit run, or at a head size that is no multiple of 8) it runs on `qkv_prep` and then, in bfloat16 at sizes in
-    multiples of 8, on the tensor-core kernels of csrc/attention_mix_mma.cu (`flash_mix` for prompts, `flash_mix_decode` for
-    single tokens, mixed scores through `fold_queries`), else on `attn_ext` (csrc/attention_ext.cu), which takes every option,
+    multiples of 8, on tensor cores (up to 128 without mixed scores and gates the tcgen05 prompt kernel and the TMA-fed decode kernel,
+    else the kernels of csrc/attention_mix_mma.cu: `flash_mix` for prompts, `flash_mix_decode` for single tokens, mixed scores
+    through `fold_queries`), else on `attn_ext` (csrc/attention_ext.cu), which takes every option,
     every size and both element types."""
 
     takes_out = True
@@ -284,31 +285,32 @@ class Attention(Mixer):
 
     def _attend(self, proj: torch.Tensor, gate, step, cache, out):
         """The attention itself over rows whose queries are ready and whose keys and values are in the cache.  bfloat16 runs take
-        the tcgen05 prompt kernel and the TMA-fed decode kernel where the sizes are theirs (equal key and value sizes of 64 or
-        128, no mixed scores, no gate), else the tensor-core kernel for unequal sizes, mixed scores and gates; 32-bit runs and
+        the tcgen05 prompt kernel and the TMA-fed decode kernel where the sizes are theirs (multiples of 8 up to 128; two maps: 64
+        or 128; no mixed scores, no gate), else the tensor-core kernel for larger sizes, mixed scores and gates; 32-bit runs and
         the remaining sizes take the general kernel."""
         bf = self.rt.dtype == torch.bfloat16
         bias = self.position.score_bias()
         if self.logistic:
             return self._attend_logistic(proj, gate, step, cache, out)
-        if (bf and self.hd == self.vd and self.hd in ops.FLASH_TC_HEAD_DIMS and not self.has_mix and gate is None and self.out_scale == 1.0
+        sizes = ops.attn_tma_takes(self.hd, self.vd) if self.maps == 1 else (self.hd == self.vd and self.hd in ops.FLASH_TC_HEAD_DIMS)
+        if (bf and sizes and not self.has_mix and gate is None and self.out_scale == 1.0
                 and proj.stride(0) % 8 == 0 and proj.data_ptr() % 16 == 0):
             direct = out is not None and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0 and out.stride(1) == 1
-            if step.decode_only and self.hd in ops.ATTN_DECODE_TMA_HEAD_DIMS and self.maps == 1:
+            if step.decode_only and self.maps == 1:
                 keys = min(self.window, step.plan_kv_len) if self.window else step.plan_kv_len
                 keys = min(self.chunk, keys) if self.chunk else keys
-                n_splits = decode_splits(step.n_seqs, self.H, self.K, keys, self.hd)
-                scratch = self.rt.workspace.get("attn_decode", ops.attn_decode_scratch_floats(step.n_seqs, self.H, self.hd, n_splits), torch.float32)
+                n_splits = decode_splits(step.n_seqs, self.H, self.K, keys, tma=True)
+                scratch = self.rt.workspace.get("attn_decode", ops.attn_decode_scratch_floats(step.n_seqs, self.H, self.vd, n_splits), torch.float32)
                 a = ops.attn_decode(
                     proj, cache.k_pages, cache.v_pages, cache.block_table, step.seq_len, self.H, self.K, self.hd, n_splits, scratch,
                     window=self.window, scale=self.scale, sink=self.sink, chunk=self.chunk, softcap=self.softcap, impl="tma",
-                    out=out if direct else None, bias=bias,
+                    out=out if direct else None, bias=bias, value_dim=self.vd,
                 )
             else:
                 a = ops.flash_prefill_tc(
                     proj, cache.k_pages, cache.v_pages, cache.block_table, step.seq_start, step.seq_pos0, step.max_q_len, self.H, self.K,
                     self.hd, window=self.window, scale=self.scale, sink=self.sink, chunk=self.chunk, softcap=self.softcap,
-                    out=out if direct else None, maps=self.maps, bias=bias,
+                    out=out if direct else None, maps=self.maps, bias=bias, value_dim=self.vd,
                 )
             if out is not None and a is not out:
                 out.copy_(a)

@@ -75,16 +75,19 @@ def config_d():
     """Larger and odd sizes in another order: keys of 40, 96 and 72 beside values of 24, 64 and 72 (padded tiles), ten heads on five, windows
     of 130 and 200, tables of many rows, twelve experts and four identities of which three, four of four experts."""
     return _model(1000, 384, 1e-5, 5.0, 0.9, [
-        dict(_full(5, 5, 96, 64, 0.12, 300, 0.4, 64), mlp=_moe(12, 4, 3, 64)),
-        dict(_win(10, 5, 40, 0.2, 150, 130), mlp=_dense(512)),
+        dict(_full(5, 5, 96, 64, 0.12, 300, 0.4, 64), mlp=_dense(512)),
+        dict(_win(10, 5, 40, 0.2, 150, 130), mlp=None),
         dict(_full(6, 3, 40, 24, 0.2, 180, 0.3, 20), mlp=_moe(4, 0, 4, 72)),
-        dict(_full(10, 5, 96, 64, 0.15, 500, 0.2, 33, kv_from=0), mlp=None),
+        dict(_full(10, 5, 96, 64, 0.15, 500, 0.2, 33, kv_from=0), mlp=_moe(12, 4, 3, 64)),
         dict(_win(4, 4, 72, 0.18, 90, 200), mlp=_moe(6, 3, 2, 96)),
         dict(_full(9, 3, 40, 24, 0.2, 70, 0.3, 50, kv_from=2), mlp=_dense(200)),
     ])
 
 
 CONFIGS = {"a": config_a, "b": config_b, "c": config_c, "d": config_d}
+# seeds with which the tests' sequences bring no close call between two experts among their first tokens (a bfloat16 run may then choose
+# the other one, and with few keys to look at every later token sees the difference)
+SEEDS = {"a": 211, "b": 213, "c": 206, "d": 212}
 ROWS = {"a": [8, 12, 26, 6, 10, 20], "b": [4, 2, 6, 2], "c": [16, 16, 32, 24, 12], "d": [40, 64, 30, 48, 20, 32]}  # rows of each layer's table
 
 
@@ -130,7 +133,9 @@ def random_weights(cfg, rows, seed):
         elif last == "rel":
             t = 1.2 * rng.standard_normal(shape)
         elif last == "correction":
-            t = 0.1 * rng.standard_normal(shape)
+            t = 0.2 * rng.standard_normal(shape)
+        elif last == "router":
+            t = 2.0 * rng.standard_normal(shape) / np.sqrt(shape[-1])  # (the last expert chosen then has a small weight beside the first)
         elif name == "embed":
             t = rng.standard_normal(shape) / float(cfg["embedding"]["scale"])
         else:

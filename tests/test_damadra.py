@@ -11,7 +11,7 @@ import torch
 
 import plain_damadra as pd
 from helpers import check_logits
-from damadra_cases import CONFIGS, ROWS, as_float64, random_weights, write_model
+from damadra_cases import CONFIGS, ROWS, SEEDS, as_float64, random_weights, write_model
 
 pytestmark = pytest.mark.gpu
 
@@ -20,9 +20,9 @@ pytestmark = pytest.mark.gpu
 def models(tmp_path_factory):
     """name -> (config, folder, float64 weights)."""
     out = {}
-    for i, (name, make) in enumerate(CONFIGS.items()):
+    for name, make in CONFIGS.items():
         cfg = make()
-        w = random_weights(cfg, ROWS[name], seed=131 + i)
+        w = random_weights(cfg, ROWS[name], SEEDS[name])
         out[name] = (cfg, write_model(tmp_path_factory.mktemp(f"dam_{name}"), cfg, w), as_float64(w))
     return out
 

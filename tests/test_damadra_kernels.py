@@ -90,7 +90,7 @@ def check_cuts(mixer, rows, ref, dtype, cut_lists, tol_bf, what=""):
 
 # heads, kv heads, key size (and value size): sizes of the general kernel, of the padded tensor-core kernels, of the tcgen05 and TMA ones
 WINDOWED = [(6, 2, 12), (3, 1, 7), (4, 2, 48), (2, 2, 72), (4, 2, 64), (12, 1, 64), (3, 1, 128), (4, 4, 136)]
-FULL = [(3, 1, 10, 12), (4, 2, 48, 32), (5, 5, 96, 64), (6, 3, 40, 24), (4, 2, 64, 64), (9, 1, 64, 64), (2, 1, 128, 128), (2, 2, 24, 200)]
+FULL = [(3, 1, 10, 12), (4, 2, 48, 32), (5, 5, 96, 64), (6, 3, 40, 24), (4, 2, 64, 64), (9, 1, 64, 64), (2, 1, 128, 128), (2, 2, 24, 200), (3, 1, 32, 128), (8, 2, 128, 40)]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -208,6 +208,46 @@ def test_batches_of_unequal_sequences(windowed, shape, dtype):
                 assert torch.equal(g, mixer.run(rows, [n]))
         seqs = seqs[::-1]
         lens = lens[::-1]
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("shape", [(4, 2, 48, 32), (6, 2, 128, 128), (4, 1, 64, 96), (3, 3, 136, 40), (4, 2, 12, 10)])
+def test_a_bias_beside_caps_sinks_windows_and_chunks(shape, dtype):
+    """The bias is added after the cap; the other options of the attention keep their meaning beside it.  Prompts and single tokens."""
+    from rusty_llama_b200.parts.attention import chunked_attention_runner
+    from types import SimpleNamespace
+
+    H, G, kd, vd = shape
+    rng = np.random.default_rng(kd)
+    n, L = 200, 17
+    q, k, v = (_rounded(rng.standard_normal(s), dtype) for s in ((n, H, kd), (n, G, kd), (n, G, vd)))
+    table = _rounded(rng.standard_normal((H, L)), torch.float32)
+    sink = _rounded(rng.standard_normal(H), torch.float32)
+    pages = [3, 0, 2, 1]
+    kp, vp = (torch.zeros((4, G, 64, size), dtype=dtype, device="cuda") for size in (kd, vd))
+    for i in range(n):
+        kp[pages[i // 64], :, i % 64], vp[pages[i // 64], :, i % 64] = _dev(k[i], dtype), _dev(v[i], dtype)
+    gap = torch.arange(n)[:, None] - torch.arange(n)[None, :]
+    for window, chunk, cap, use_sink in ((0, 0, 2.0, True), (70, 0, 0.0, True), (0, 48, 1.5, False), (33, 96, 0.0, False)):
+        scale = 1.5 / np.sqrt(kd)
+        s = torch.einsum("ihd,jhd->hij", q, k.repeat_interleave(H // G, 1)) * scale
+        s = (cap * torch.tanh(s / cap) if cap else s) + table[:, gap.clamp(0, L - 1)]
+        vis = (gap >= 0) & ((gap < window) if window else True)
+        if chunk:
+            vis = vis & (torch.arange(n)[:, None] // chunk == torch.arange(n)[None, :] // chunk)
+        e = torch.exp(s.masked_fill(~vis[None], -np.inf))
+        den = e.sum(-1, keepdim=True) + (torch.exp(sink)[:, None, None] if use_sink else 0.0)
+        ref = torch.einsum("hij,jhv->ihv", e / den, v.repeat_interleave(H // G, 1)).reshape(n, -1)
+        for p0, m in ((0, n), (130, 70), (199, 1), (64, 1)):
+            step = SimpleNamespace(tok_seq=_i32(np.zeros(m)), tok_pos=_i32(np.arange(p0, p0 + m)), seq_start=_i32([0, m]), seq_pos0=_i32([p0]), max_q_len=m, n_seqs=1,
+                                   decode_only=m == 1)
+            rows = torch.zeros((m, H * kd + 8), dtype=dtype, device="cuda")
+            rows[:, : H * kd] = _dev(q[p0 : p0 + m].reshape(m, -1), dtype)
+            got = chunked_attention_runner(rows, kp, vp, _i32([pages]), step, H, G, kd, vd, scale, chunk, cap, _dev(sink, torch.float32) if use_sink else None,
+                                           window=window, bias=_dev(table, torch.float32))().to(F64).cpu()
+            tol = 1e-5 if dtype == torch.float32 else 2.5e-2
+            worst = (got - ref[p0 : p0 + m]).abs().max(1).values
+            assert float(worst.max()) <= tol * float(ref.abs().max()), f"window {window}, chunk {chunk}, cap {cap}, from {p0}: row {int(worst.argmax())}"
 
 
 # ------------------------------------------------------------------ norms, temperature, storing
