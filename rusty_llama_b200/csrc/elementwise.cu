@@ -535,6 +535,92 @@ __global__ void normed_add_rmsnorm_kernel(float* __restrict__ x, const TD* __res
   }
 }
 
+// The same with the row in registers, CHUNKS pieces of four values a thread.  One piece a thread (a row of up to four values a
+// thread of the block): everything is asked for before anything is used, and the sums above are added in the order above, so
+// which of the two runs does not show.  Several: fewer threads a row for the many rows of a prompt step, in bfloat16 runs only, whose
+// sums may be added in another order than a decode step's; the weights are asked for when they are needed, since the registers
+// that would hold them meanwhile are worth more as further rows in flight.
+template <typename TA, typename TW, typename TD, int CHUNKS>
+__global__ void __launch_bounds__(CHUNKS == 1 ? 1024 : 256, CHUNKS == 1 ? 1 : (CHUNKS == 2 ? 5 : 4))
+normed_add_rows_kernel(float* __restrict__ x, const TD* __restrict__ delta, int n_parts, long long part_stride,
+                       const float* __restrict__ bias, const TW* __restrict__ wd, float eps_d, const TW* __restrict__ w, float eps,
+                       TA* __restrict__ out, const int* __restrict__ rows, int d, int write_x) {
+  __shared__ float red[32];
+  pdl_trigger();
+  pdl_wait();
+  const int r = blockIdx.x;
+  const int t = rows ? rows[r] : r;
+  float* xr = x + (size_t)t * d;
+  constexpr bool AHEAD = CHUNKS == 1;
+  float v[CHUNKS][4], s[CHUNKS][4], wdv[4] = {0.f, 0.f, 0.f, 0.f}, wv[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+  for (int c = 0; c < CHUNKS; ++c) {
+    const int i = (threadIdx.x + c * blockDim.x) * 4;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[c][e] = s[c][e] = 0.f;
+    if (i < d) {
+      load4_g<float>(xr + i, v[c]);
+      load4_g<TD>(delta + (size_t)t * d + i, s[c]);
+      if (AHEAD) {
+        load4_g<TW>(wd + i, wdv);
+        if (w != nullptr) load4_g<TW>(w + i, wv);
+      }
+    }
+  }
+  for (int p = 1; p < n_parts; ++p) {
+#pragma unroll
+    for (int c = 0; c < CHUNKS; ++c) {
+      const int i = (threadIdx.x + c * blockDim.x) * 4;
+      if (i < d) {
+        float dv[4];
+        load4_g<TD>(delta + (size_t)p * part_stride + (size_t)t * d + i, dv);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[c][e] += dv[e];
+      }
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < CHUNKS; ++c) {
+    const int i = (threadIdx.x + c * blockDim.x) * 4;
+    if (bias != nullptr && i < d) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[c][e] += bias[i + e];
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) ss += s[c][e] * s[c][e];
+  }
+  const float inv_d = 1.0f / sqrtf(block_sum(ss, red) / (float)d + eps_d);
+  TA* o = out + (size_t)r * d;
+  ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < CHUNKS; ++c) {
+    const int i = (threadIdx.x + c * blockDim.x) * 4;
+    if (!AHEAD && i < d) load4_g<TW>(wd + i, wdv);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      v[c][e] += s[c][e] * inv_d * wdv[e];
+      ss += v[c][e] * v[c][e];
+    }
+    if (i < d) {
+      if (write_x) store4<float>(xr + i, v[c]);
+      if (w == nullptr && out != nullptr) store4<TA>(o + i, v[c]);
+    }
+  }
+  if (w == nullptr) return;
+  const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)d + eps);
+#pragma unroll
+  for (int c = 0; c < CHUNKS; ++c) {
+    const int i = (threadIdx.x + c * blockDim.x) * 4;
+    if (i < d) {
+      if (!AHEAD) load4_g<TW>(w + i, wv);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[c][e] = v[c][e] * inv * wv[e];
+      store4<TA>(o + i, v[c]);
+    }
+  }
+}
+
 RL_API int rl_normed_add_rmsnorm(float* x, const void* delta, int delta_dtype, int n_parts, long long part_stride, const float* bias, const void* wd,
                                  float eps_d, const void* w, int w_dtype, float eps, void* out, int act_dtype, const int* rows,
                                  int n_rows, int d, int write_x, cudaStream_t stream) {
@@ -547,9 +633,20 @@ RL_API int rl_normed_add_rmsnorm(float* x, const void* delta, int delta_dtype, i
   const bool vec = d % 4 == 0 && (((uintptr_t)x | (uintptr_t)delta | (uintptr_t)wd | (uintptr_t)w | (uintptr_t)out) % 16 == 0) &&
                    (part_stride % 4 == 0);
   const int th = vec ? row_threads(d) : (d >= 512 ? 512 : ((d + 31) / 32) * 32);
+  // (a row of at most 1024 values has its one piece a thread with 256 threads, too)
+  const bool many = vec && act_dtype == RL_BF16 && n_rows >= ROWS_KERNEL_MIN_ROWS && d > 1024 && d <= 4096;
 #define RL_NN(TA, TW, TD)                                                                                                       \
   do {                                                                                                                          \
-    if (vec)                                                                                                                    \
+    if (many && d <= 2048)                                                                                                      \
+      RL_LAUNCH_CHECK(rl_launch(normed_add_rows_kernel<TA, TW, TD, 2>, n_rows, 256, 0, stream, x, (const TD*)delta,             \
+                                n_parts, part_stride, bias, (const TW*)wd, eps_d, (const TW*)w, eps, (TA*)out, rows, d, write_x)); \
+    else if (many)                                                                                                              \
+      RL_LAUNCH_CHECK(rl_launch(normed_add_rows_kernel<TA, TW, TD, 4>, n_rows, 256, 0, stream, x, (const TD*)delta,             \
+                                n_parts, part_stride, bias, (const TW*)wd, eps_d, (const TW*)w, eps, (TA*)out, rows, d, write_x)); \
+    else if (vec && d <= th * 4)                                                                                                \
+      RL_LAUNCH_CHECK(rl_launch(normed_add_rows_kernel<TA, TW, TD, 1>, n_rows, th, 0, stream, x, (const TD*)delta,              \
+                                n_parts, part_stride, bias, (const TW*)wd, eps_d, (const TW*)w, eps, (TA*)out, rows, d, write_x)); \
+    else if (vec)                                                                                                               \
       RL_LAUNCH_CHECK(rl_launch(normed_add_rmsnorm_kernel<TA, TW, TD, true>, n_rows, th, smem, stream, x, (const TD*)delta,    \
                                 n_parts, part_stride, bias, (const TW*)wd, eps_d, (const TW*)w, eps, (TA*)out, rows, d, write_x)); \
     else                                                                                                                        \
