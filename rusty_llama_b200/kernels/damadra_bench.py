@@ -23,9 +23,9 @@ import torch
 
 from . import microbench as mb
 from . import ops
-from .linear import linear
 from .design_bench import SIZES as VEZATAR_SIZES
 from .design_bench import _frac, llama_config, step_times, vezatar_config
+from .linear import linear
 
 # Vezatar's sizes, and beside them: query heads, kv heads and their size, the window, the identities among the router's choices
 SIZES = {
@@ -118,7 +118,7 @@ def kernel_table(z: dict, T: int, batch: int, ctx: int, peaks: dict) -> Dict[str
                 us[b is not None] = timed(chunked_attention_runner(full_rows, kp, vp, table, step, H, K, hd, hd, scale, 0, 0.0, None, window=window, bias=b))
             nb, fl = (0, 4.0 * keys * H * hd) if prompt else (seen * K * 2 * hd * 2, 0)
             note(f"{tag}_{what}_attention", us[True], nb, fl, ("the same without a bias", us[False], nb, fl))
-        # ---- keys half as long again as the values, which the padded kernels take
+        # ---- keys half as long again as the values (sizes that the kernels pad)
         kd, vd = hd * 3 // 4, hd // 2
         kp2, vp2 = torch.randn(n_seqs * pages, K, 64, kd, device=dev, dtype=bf), torch.randn(n_seqs * pages, K, 64, vd, device=dev, dtype=bf)
         rows2 = torch.randn(rows, H * kd + K * (kd + vd), device=dev, dtype=bf)
@@ -127,7 +127,7 @@ def kernel_table(z: dict, T: int, batch: int, ctx: int, peaks: dict) -> Dict[str
             us[b is not None] = timed(chunked_attention_runner(rows2, kp2, vp2, table, step, H, K, kd, vd, scale, 0, 0.0, None, bias=b))
         keys = sum(p + 1 for p in range(pos0, pos0 + per)) * n_seqs
         nb, fl = (0, 2.0 * keys * H * (kd + vd)) if prompt else (ctx * n_seqs * K * (kd + vd) * 2, 0)
-        note(f"{tag}_unequal_attention", us[True], nb, fl, ("the same without a bias (Revirax)", us[False], nb, fl))
+        note(f"{tag}_unequal_attention", us[True], nb, fl, ("the same without a bias", us[False], nb, fl))
         # ---- experts
         E, I, top, eff = z["experts"], z["identity"], z["top"], z["eff"]
         x = torch.randn(rows, d, device=dev, dtype=bf)

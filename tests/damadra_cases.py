@@ -62,9 +62,9 @@ def config_b():
 def config_c():
     """Sizes that the tensor-core kernels take: heads of 64 and 128 on both kinds, windows of 64 and 70, a table whose borders are whole
     numbers (16 rows up to 128), a reader with another number of query heads."""
-    return _model(160, 128, 1e-6, 8.0, 0.5, [
+    return _model(160, 128, 1e-6, 8.0, 0.6, [
         dict(_win(4, 2, 64, 0.25, 128, 64), mlp=_dense(256)),
-        dict(_full(4, 2, 64, 64, 0.25, 128, 0.5, 32), mlp=_moe(8, 4, 3, 48)),
+        dict(_full(4, 2, 64, 64, 0.25, 128, 0.5, 32), mlp=_moe(9, 5, 3, 48)),
         dict(_win(3, 1, 128, 0.18, 100, 70), mlp=_moe(4, 1, 1, 128)),
         dict(_full(2, 1, 128, 128, 0.2, 128, 0.3, 50), mlp=_dense(128)),
         dict(_full(8, 2, 64, 64, 0.3, 40, 0.1, 9, kv_from=1), mlp=_dense(64)),
@@ -87,7 +87,7 @@ def config_d():
 CONFIGS = {"a": config_a, "b": config_b, "c": config_c, "d": config_d}
 # seeds with which the tests' sequences bring no close call between two experts among their first tokens (a bfloat16 run may then choose
 # the other one, and with few keys to look at every later token sees the difference)
-SEEDS = {"a": 211, "b": 213, "c": 206, "d": 212}
+SEEDS = {"a": 211, "b": 213, "c": 207, "d": 212}
 ROWS = {"a": [8, 12, 26, 6, 10, 20], "b": [4, 2, 6, 2], "c": [16, 16, 32, 24, 12], "d": [40, 64, 30, 48, 20, 32]}  # rows of each layer's table
 
 

@@ -89,8 +89,8 @@ def check_cuts(mixer, rows, ref, dtype, cut_lists, tol_bf, what=""):
 
 
 # heads, kv heads, key size (and value size): sizes of the general kernel, of the padded tensor-core kernels, of the tcgen05 and TMA ones
-WINDOWED = [(6, 2, 12), (3, 1, 7), (4, 2, 48), (2, 2, 72), (4, 2, 64), (12, 1, 64), (3, 1, 128), (4, 4, 136)]
-FULL = [(3, 1, 10, 12), (4, 2, 48, 32), (5, 5, 96, 64), (6, 3, 40, 24), (4, 2, 64, 64), (9, 1, 64, 64), (2, 1, 128, 128), (2, 2, 24, 200), (3, 1, 32, 128), (8, 2, 128, 40)]
+WINDOWED = [(6, 2, 12), (3, 1, 7), (4, 2, 56), (2, 2, 72), (4, 2, 64), (12, 1, 64), (3, 1, 128), (4, 4, 136)]
+FULL = [(3, 1, 10, 12), (4, 2, 56, 40), (5, 5, 96, 64), (6, 3, 40, 24), (4, 2, 64, 64), (9, 1, 64, 64), (2, 1, 128, 128), (2, 2, 24, 200), (3, 1, 32, 128), (8, 2, 128, 40)]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -211,7 +211,7 @@ def test_batches_of_unequal_sequences(windowed, shape, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("shape", [(4, 2, 48, 32), (6, 2, 128, 128), (4, 1, 64, 96), (3, 3, 136, 40), (4, 2, 12, 10)])
+@pytest.mark.parametrize("shape", [(4, 2, 56, 40), (6, 2, 128, 128), (4, 1, 64, 96), (3, 3, 136, 40), (4, 2, 12, 10)])
 def test_a_bias_beside_caps_sinks_windows_and_chunks(shape, dtype):
     """The bias is added after the cap; the other options of the attention keep their meaning beside it.  Prompts and single tokens."""
     from rusty_llama_b200.parts.attention import chunked_attention_runner
@@ -252,7 +252,7 @@ def test_a_bias_beside_caps_sinks_windows_and_chunks(shape, dtype):
 
 # ------------------------------------------------------------------ norms, temperature, storing
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("H,G,kd,vd", [(4, 2, 48, 32), (3, 1, 10, 6), (2, 2, 128, 128), (5, 1, 40, 8), (8, 4, 64, 64), (1, 1, 256, 16), (40, 8, 128, 128)])
+@pytest.mark.parametrize("H,G,kd,vd", [(4, 2, 56, 40), (3, 1, 10, 6), (2, 2, 128, 128), (5, 1, 40, 8), (8, 4, 64, 64), (1, 1, 256, 16), (40, 8, 128, 128)])
 def test_rows_normed_tempered_and_stored(H, G, kd, vd, dtype):
     """Norms over all heads at once and head by head, in rows whose heads differ by factors; values that are the raw keys; the
     temperature around its steps; rows of queries only leave the pages alone."""
@@ -291,7 +291,7 @@ def test_rows_normed_tempered_and_stored(H, G, kd, vd, dtype):
 
 # ------------------------------------------------------------------ experts and identities
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("E,identity,top,d,ff,T", [(5, 2, 3, 64, 48, 9), (4, 3, 2, 128, 72, 200), (1, 2, 3, 68, 30, 7), (3, 0, 1, 96, 24, 150), (12, 4, 3, 256, 96, 333), (2, 6, 4, 36, 17, 40)])
+@pytest.mark.parametrize("E,identity,top,d,ff,T", [(5, 2, 3, 64, 40, 9), (4, 3, 2, 128, 72, 200), (1, 2, 3, 68, 30, 7), (3, 0, 1, 96, 24, 150), (12, 5, 3, 192, 80, 333), (2, 6, 4, 36, 17, 40)])
 def test_experts_beside_choices_that_hand_the_input_on(E, identity, top, d, ff, T, dtype):
     from rusty_llama_b200.parts import FEED_FORWARDS, Runtime
     from rusty_llama_b200.spec import PartSpec
